@@ -10,7 +10,8 @@
 // result) whatever the dtype of x and out; one gate entry may cover `group` neighbouring columns (a gate per head).
 // Input and output rows may have strides of their own (the output may be a column block of a wider buffer).
 // Further: the gated hidden layer out[t][i] = act(gu[t][i]) * gu[t][I + i] of a feed-forward whose gate and up
-// projections are one product; out[t][c] = act(z[t][c]) * table[ids[t]][off + c], a gate on a slice of a row
+// projections are one product (also in the clamped form: gate and up limited to [-, c] and [-c, c], out = g sigmoid(1.702 g)
+// (u + 1)); out[t][c] = act(z[t][c]) * table[ids[t]][off + c], a gate on a slice of a row
 // gathered per token; and the soft cap x <- cap tanh(x / cap) of float32 rows in place.
 #include "common.cuh"
 #include "vec.cuh"
@@ -21,6 +22,7 @@
 #define PRISM_ACT_RELU 3
 #define PRISM_ACT_TANH 4
 #define PRISM_ACT_SIGMOID 5
+#define PRISM_ACT_CLAMPED 6      // gated layers only (common.cuh: clamped_glu)
 
 namespace prism {
 
@@ -92,8 +94,13 @@ __global__ void gated_product_kernel(const T* __restrict__ x_in, long long x_str
         o[i] = from_float<T>(to_float(x[i]) * activate<ACT>(g[i / group]) * c);
 }
 
+template <int ACT> __device__ __forceinline__ float gated(float g, float u, float limit) {
+    return ACT == PRISM_ACT_CLAMPED ? clamped_glu(g, u, limit) : activate<ACT>(g) * u;
+}
+
 template <typename T, int ACT>
-__global__ void glu_kernel(const T* __restrict__ gu_in, long long gs, T* __restrict__ out, long long os, int I, int vec) {
+__global__ void glu_kernel(const T* __restrict__ gu_in, long long gs, T* __restrict__ out, long long os, int I, int vec,
+                           float limit) {
     pdl_trigger();
     pdl_wait();
     const T* gu = pdl_fresh(gu_in) + (size_t)blockIdx.y * gs;
@@ -105,12 +112,12 @@ __global__ void glu_kernel(const T* __restrict__ gu_in, long long gs, T* __restr
         load8(gu + c, g);
         load8(gu + I + c, u);
 #pragma unroll
-        for (int k = 0; k < 8; ++k) g[k] = activate<ACT>(g[k]) * u[k];
+        for (int k = 0; k < 8; ++k) g[k] = gated<ACT>(g[k], u[k], limit);
         store8(o + c, g);
         return;
     }
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < I; i += gridDim.x * blockDim.x)
-        o[i] = from_float<T>(activate<ACT>(to_float(gu[i])) * to_float(gu[I + i]));
+        o[i] = from_float<T>(gated<ACT>(to_float(gu[i]), to_float(gu[I + i]), limit));
 }
 
 template <typename T, typename W, int ACT>
@@ -170,23 +177,25 @@ PRISM_EXPORT int prism_activation(const void* x, long long x_stride, void* out, 
 }
 
 // gu [rows, 2 I] of `dtype` (gate columns first, row stride gu_stride) -> out [rows, I] = act(gate) * up.
-// act: PRISM_ACT_SILU or PRISM_ACT_GELU_TANH.
+// act: PRISM_ACT_SILU, PRISM_ACT_GELU_TANH or PRISM_ACT_CLAMPED (with `limit`).
 PRISM_EXPORT int prism_glu(const void* gu, long long gu_stride, void* out, long long out_stride, int dtype, int rows, int I,
-                           int act, cudaStream_t stream) {
+                           int act, float limit, cudaStream_t stream) {
     if (rows <= 0 || I <= 0) return 0;
-    if (rows > 65535 || (act != PRISM_ACT_SILU && act != PRISM_ACT_GELU_TANH)) return (int)cudaErrorInvalidValue;
+    if (rows > 65535 || (act != PRISM_ACT_SILU && act != PRISM_ACT_GELU_TANH && act != PRISM_ACT_CLAMPED)) return (int)cudaErrorInvalidValue;
     const int esz = dtype == PRISM_DTYPE_BF16 ? 2 : 4;
     const bool vec = I % 8 == 0 && gu_stride % 8 == 0 && out_stride % 8 == 0 && (uintptr_t)gu % (8 * esz) == 0 &&
                      (uintptr_t)out % (8 * esz) == 0;
     dim3 grid(((vec ? I / 8 : I) + 255) / 256, rows);
 #define PRISM_GLU(TT, A)                                                                                          \
     return (int)prism::launch_kernel(prism::glu_kernel<TT, A>, grid, dim3(256), 0, stream, (const TT*)gu, gu_stride, \
-                                     (TT*)out, out_stride, I, vec ? 1 : 0)
+                                     (TT*)out, out_stride, I, vec ? 1 : 0, limit)
     if (dtype == PRISM_DTYPE_BF16) {
         if (act == PRISM_ACT_SILU) PRISM_GLU(__nv_bfloat16, PRISM_ACT_SILU);
+        if (act == PRISM_ACT_CLAMPED) PRISM_GLU(__nv_bfloat16, PRISM_ACT_CLAMPED);
         PRISM_GLU(__nv_bfloat16, PRISM_ACT_GELU_TANH);
     }
     if (act == PRISM_ACT_SILU) PRISM_GLU(float, PRISM_ACT_SILU);
+    if (act == PRISM_ACT_CLAMPED) PRISM_GLU(float, PRISM_ACT_CLAMPED);
     PRISM_GLU(float, PRISM_ACT_GELU_TANH);
 #undef PRISM_GLU
 }

@@ -111,6 +111,13 @@ __device__ __forceinline__ float load_param(const void* p, int is_bf16, size_t i
                    : reinterpret_cast<const float*>(p)[i];
 }
 
+// gate and up of a clamped gated feed-forward: g limited from above, u from both sides, g sigmoid(1.702 g) (u + 1)
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

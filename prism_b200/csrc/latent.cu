@@ -3,12 +3,14 @@
 //  * latent_kv_store: the row a token leaves in the cache.  From the down projection x [T, R + r] (float32):
 //    the first R entries divided by their root mean square (eps inside the root) and multiplied by a weight
 //    are the latent; the last r entries are the key part that carries the position and is shared by all
-//    heads: its first `rot_dims` entries are rotated (entry i paired with i + rot_dims / 2, angle
-//    position * inv_freq[i]), the others pass.  Norm, angles and rotation in float32, one rounding at the
+//    heads: its first `rot_dims` entries are rotated (entry i paired with i + rot_dims / 2, or entry 2i with
+//    2i + 1; angle position * inv_freq[i], cosine and sine times a constant `amp`), the others pass.  Norm, angles
+//    and rotation in float32, one rounding at the
 //    store into the paged plane [slots, R + r].  The same launch can norm the query latent of the token, which
 //    is another column block of the same down projection.
 //  * rotate_slice: the same rotation for a slice of `width` entries of every head of a [T, nh, ...] tensor,
-//    written to a slice of another tensor (the queries' rotated part, next to their absorbed part).
+//    written to a slice of another tensor (the queries' rotated part, next to their absorbed part) or in place, all
+//    entries times a constant.
 //  * rms_rows: x / sqrt(mean(x^2) + eps) * weight for rows of a float32 matrix with a row stride of its own
 //    (a column block of a fused projection's output), stored in the compute dtype.
 #include "common.cuh"
@@ -23,7 +25,7 @@ __global__ void latent_kv_store_kernel(const float* __restrict__ x_in, long long
                                        const int* __restrict__ positions, const int* __restrict__ tok_seg,
                                        int page_size, int num_pages, int max_pos, int* err,
                                        const float* __restrict__ xq_in, int q_rank, const void* __restrict__ q_weight,
-                                       int q_weight_bf16, T* __restrict__ q_out, long long q_out_stride) {
+                                       int q_weight_bf16, T* __restrict__ q_out, long long q_out_stride, int pairs, float amp) {
     pdl_trigger();
     pdl_wait();
     __shared__ float scratch[33];
@@ -58,19 +60,22 @@ __global__ void latent_kv_store_kernel(const float* __restrict__ x_in, long long
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float sn, cs;
         sincosf((float)pos * inv_freq[i], &sn, &cs);
-        const float u = x[R + i], v = x[R + i + half];
-        dst[R + i] = from_float<T>(u * cs - v * sn);
-        dst[R + i + half] = from_float<T>(v * cs + u * sn);
+        sn *= amp;
+        cs *= amp;
+        const int a = pairs ? 2 * i : i, b = pairs ? 2 * i + 1 : i + half;
+        const float u = x[R + a], v = x[R + b];
+        dst[R + a] = from_float<T>(u * cs - v * sn);
+        dst[R + b] = from_float<T>(v * cs + u * sn);
     }
     for (int c = rot_dims + threadIdx.x; c < r; c += blockDim.x) dst[R + c] = from_float<T>(x[R + c]);
 }
 
 // one warp per (token, head)
 template <typename T>
-__global__ void rotate_slice_kernel(const T* __restrict__ in_, long long in_tok_stride, int in_head_stride,
-                                    T* __restrict__ out, long long out_tok_stride, int out_head_stride, int width,
+__global__ void rotate_slice_kernel(const T* in_, long long in_tok_stride, int in_head_stride,
+                                    T* out, long long out_tok_stride, int out_head_stride, int width,
                                     int rot_dims, const float* __restrict__ inv_freq,
-                                    const int* __restrict__ positions, int Ttot, int nh) {
+                                    const int* __restrict__ positions, int Ttot, int nh, int pairs, float amp, float mul) {
     pdl_trigger();
     pdl_wait();
     const T* in = pdl_fresh(in_);
@@ -85,11 +90,14 @@ __global__ void rotate_slice_kernel(const T* __restrict__ in_, long long in_tok_
     for (int i = lane; i < half; i += 32) {
         float sn, cs;
         sincosf(pos * inv_freq[i], &sn, &cs);
-        const float u = to_float(src[i]), v = to_float(src[i + half]);
-        dst[i] = from_float<T>(u * cs - v * sn);
-        dst[i + half] = from_float<T>(v * cs + u * sn);
+        sn *= amp;
+        cs *= amp;
+        const int a = pairs ? 2 * i : i, b = pairs ? 2 * i + 1 : i + half;
+        const float u = to_float(src[a]), v = to_float(src[b]);
+        dst[a] = from_float<T>((u * cs - v * sn) * mul);
+        dst[b] = from_float<T>((v * cs + u * sn) * mul);
     }
-    for (int c = rot_dims + lane; c < width; c += 32) dst[c] = src[c];
+    for (int c = rot_dims + lane; c < width; c += 32) dst[c] = from_float<T>(to_float(src[c]) * mul);
 }
 
 template <typename T>
@@ -124,13 +132,14 @@ PRISM_EXPORT int prism_rms_rows(const float* x, long long x_stride, const void* 
 
 // x: float32 [T, R + r] with row stride x_stride; cache: plane [slots, R + r] of `dtype`.  xq (null: none):
 // float32 [T, q_rank] with the same row stride (another column block of the same product), RMS-normed with
-// q_weight into q_out [T, q_rank] of `dtype` by the same launch.
+// q_weight into q_out [T, q_rank] of `dtype` by the same launch.  pairs: rotate entries (2i, 2i + 1) instead of halves;
+// amp: a factor on cosine and sine.
 PRISM_EXPORT int prism_latent_kv_store(const float* x, long long x_stride, const void* weight, int weight_dtype,
                                        float eps, int R, int r, int rot_dims, const float* inv_freq, void* cache,
                                        int dtype, const int* block_table, int bt_width, const int* positions,
                                        const int* tok_seg, int T, int page_size, int num_pages, int max_pos, int* err,
                                        const float* xq, int q_rank, const void* q_weight, int q_weight_dtype,
-                                       void* q_out, long long q_out_stride, cudaStream_t stream) {
+                                       void* q_out, long long q_out_stride, int pairs, float amp, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (R <= 0 || r < 0 || rot_dims < 0 || rot_dims > r || rot_dims % 2) return (int)cudaErrorInvalidValue;
     if (q_out != nullptr && (xq == nullptr || q_weight == nullptr || q_rank <= 0)) return (int)cudaErrorInvalidValue;
@@ -140,17 +149,19 @@ PRISM_EXPORT int prism_latent_kv_store(const float* x, long long x_stride, const
         return (int)prism::launch_kernel(prism::latent_kv_store_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, x,
                                          x_stride, weight, wb, eps, R, r, rot_dims, inv_freq, (__nv_bfloat16*)cache,
                                          block_table, bt_width, positions, tok_seg, page_size, num_pages, max_pos, err, xq,
-                                         q_rank, q_weight, qwb, (__nv_bfloat16*)q_out, q_out_stride);
+                                         q_rank, q_weight, qwb, (__nv_bfloat16*)q_out, q_out_stride, pairs, amp);
     return (int)prism::launch_kernel(prism::latent_kv_store_kernel<float>, dim3(T), dim3(threads), 0, stream, x, x_stride,
                                      weight, wb, eps, R, r, rot_dims, inv_freq, (float*)cache, block_table, bt_width,
                                      positions, tok_seg, page_size, num_pages, max_pos, err, xq, q_rank, q_weight, qwb,
-                                     (float*)q_out, q_out_stride);
+                                     (float*)q_out, q_out_stride, pairs, amp);
 }
 
-// in/out point at the slice's first entry of head 0 of token 0; strides in elements.
+// in/out point at the slice's first entry of head 0 of token 0 (they may be the same); strides in elements; pairs and amp
+// as above, mul: a factor on every entry of the slice.
 PRISM_EXPORT int prism_rotate_slice(const void* in, long long in_tok_stride, int in_head_stride, void* out,
                                     long long out_tok_stride, int out_head_stride, int dtype, int width, int rot_dims,
-                                    const float* inv_freq, const int* positions, int T, int nh, cudaStream_t stream) {
+                                    const float* inv_freq, const int* positions, int T, int nh, int pairs, float amp,
+                                    float mul, cudaStream_t stream) {
     if (T <= 0 || nh <= 0 || width <= 0) return 0;
     if (rot_dims < 0 || rot_dims > width || rot_dims % 2) return (int)cudaErrorInvalidValue;
     const int warps = 4;
@@ -159,8 +170,8 @@ PRISM_EXPORT int prism_rotate_slice(const void* in, long long in_tok_stride, int
     if (dtype == PRISM_DTYPE_BF16)
         return (int)prism::launch_kernel(prism::rotate_slice_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), 0, stream,
                                          (const __nv_bfloat16*)in, in_tok_stride, in_head_stride, (__nv_bfloat16*)out,
-                                         out_tok_stride, out_head_stride, width, rot_dims, inv_freq, positions, T, nh);
+                                         out_tok_stride, out_head_stride, width, rot_dims, inv_freq, positions, T, nh, pairs, amp, mul);
     return (int)prism::launch_kernel(prism::rotate_slice_kernel<float>, dim3(blocks), dim3(warps * 32), 0, stream,
                                      (const float*)in, in_tok_stride, in_head_stride, (float*)out, out_tok_stride,
-                                     out_head_stride, width, rot_dims, inv_freq, positions, T, nh);
+                                     out_head_stride, width, rot_dims, inv_freq, positions, T, nh, pairs, amp, mul);
 }

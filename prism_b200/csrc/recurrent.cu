@@ -1,5 +1,5 @@
 // Recurrent mixers: layers whose memory of a sequence is a matrix of fixed size per head instead of a cache of
-// keys.  Two recurrences share one scan kernel; S is [dk, dv] per head, float32, one per request slot:
+// keys.  The recurrences share one scan kernel; S is [dk, dv] per head, float32, one per request slot:
 //
 //   delta rule with a scalar decay (SCAN_DELTA), per token with unit-length q, k and g, beta in (0, 1):
 //       S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q          (the read-out sees this token's write)
@@ -10,6 +10,8 @@
 //   generalized delta rule (SCAN_GENERAL), w, e, c vectors over the key channels (e the unit key, c = a * e a removal
 //   rate per channel times it):
 //       S <- diag(w) S - c (e^T S) + k v^T;   o = S^T r         (decay and removal both read the state before the token)
+//   decayed sum with one constant decay per head (SCAN_RETAIN):
+//       S <- g S + k v^T;   o = S^T q                           (the read-out sees this token's write)
 //
 // Everything that enters the recurrence is float32: the kernels here read the float32 results of the input
 // projections, and the state never leaves float32.  A request's state lives in its slot between steps, so
@@ -31,6 +33,7 @@
 #define PRISM_SCAN_BONUS 1
 #define PRISM_SCAN_CHANNEL 2
 #define PRISM_SCAN_GENERAL 3
+#define PRISM_SCAN_RETAIN 4
 
 namespace prism {
 
@@ -269,6 +272,7 @@ __global__ void headnorm_gate_kernel(const float* __restrict__ o_in, const float
 //                with w = exp(-exp(ww + w0)) formed in shared memory, w0 [H dk], bonus u [H dk].
 //   SCAN_CHANNEL: q, k, v as for SCAN_DELTA; the decay itself in ww [T, H dk] (row stride ws); bg [T, H]: beta.
 //   SCAN_GENERAL: r, k, v as for SCAN_BONUS; the decay itself in ww; ex [T, 2 H dk]: the unit key e at h dk, c at (H + h) dk.
+//   SCAN_RETAIN: q, k, v as for SCAN_BONUS; the decay of head h in w0[h].
 // ---------------------------------------------------------------------------------------------------------
 struct ScanArgs {
     const float* x;          // q | k | v (or r | k | v) rows
@@ -308,12 +312,17 @@ template <int L> __device__ __forceinline__ float column_sum(float v) {
     return v;
 }
 
+// vectors over the key channels that a token brings: q (or r) and k, a decay per channel, a unit key and what it removes
+__host__ __device__ constexpr int scan_vectors(int mode) {
+    return (mode == PRISM_SCAN_DELTA || mode == PRISM_SCAN_RETAIN) ? 2 : (mode == PRISM_SCAN_GENERAL ? 5 : 3);
+}
+
 template <int MODE, int R, int L>
 __global__ void scan_kernel(const ScanArgs a) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float sm[];
-    constexpr int NV = MODE == PRISM_SCAN_DELTA ? 2 : (MODE == PRISM_SCAN_GENERAL ? 5 : 3);       // vectors over the key channels per token
+    constexpr int NV = scan_vectors(MODE);       // vectors over the key channels per token
     constexpr int Q = R / 4;                                   // quads of rows a thread owns
     const int h = blockIdx.x, seg = blockIdx.y, col0 = blockIdx.z * a.cols;
     const int s0 = a.seg_start[seg], qlen = a.seg_start[seg + 1] - s0;
@@ -361,7 +370,7 @@ __global__ void scan_kernel(const ScanArgs a) {
         float* dst0 = sm + (size_t)buf * TB * per_tok;
         const int unit = a.vec ? 4 : 1;
         const int nk = (dk + unit - 1) / unit, nc = (ncols + unit - 1) / unit;     // pieces per vector
-        const size_t head_q = (size_t)((MODE == PRISM_SCAN_BONUS || MODE == PRISM_SCAN_GENERAL) ? h : kvh) * dk;
+        const size_t head_q = (size_t)((MODE == PRISM_SCAN_DELTA || MODE == PRISM_SCAN_CHANNEL) ? kvh : h) * dk;
         for (int tt = 0; tt < nb; ++tt) {
             const size_t t = (size_t)(s0 + b0 + tt);
             const float* xr = x + t * a.xs;
@@ -369,7 +378,7 @@ __global__ void scan_kernel(const ScanArgs a) {
             for (int c = lane; c < nk; c += 32) {
                 cp_async_f(dst + c * unit, xr + a.qo + head_q + c * unit, unit);
                 cp_async_f(dst + dkp + c * unit, xr + a.ko + head_q + c * unit, unit);
-                if (MODE != PRISM_SCAN_DELTA) cp_async_f(dst + 2 * dkp + c * unit, ww + t * a.ws + (size_t)h * dk + c * unit, unit);
+                if (NV > 2) cp_async_f(dst + 2 * dkp + c * unit, ww + t * a.ws + (size_t)h * dk + c * unit, unit);
                 if (MODE == PRISM_SCAN_GENERAL) {
                     cp_async_f(dst + 3 * dkp + c * unit, ex + t * a.es + (size_t)h * dk + c * unit, unit);
                     cp_async_f(dst + 4 * dkp + c * unit, ex + t * a.es + (size_t)(a.H + h) * dk + c * unit, unit);
@@ -421,6 +430,7 @@ __global__ void scan_kernel(const ScanArgs a) {
         }
     }
     __syncthreads();
+    const float keep = MODE == PRISM_SCAN_RETAIN ? load_param(a.w0, a.w0_bf16, h) : 0.f;      // the head's constant decay
 
     int buf = 0;
     for (int b0 = 0; b0 < qlen; b0 += TB, buf = buf + 1 == NBUF ? 0 : buf + 1) {
@@ -534,6 +544,21 @@ __global__ void scan_kernel(const ScanArgs a) {
                     o2 += S[4 * m + 2] * rr.z;
                     o3 += S[4 * m + 3] * rr.w;
                 }
+            } else if (MODE == PRISM_SCAN_RETAIN) {
+                const float v = f2[dkp + lc];
+#pragma unroll
+                for (int m = 0; m < Q; ++m) {
+                    const int i = 4 * (part + L * m);
+                    const float4 qq = *reinterpret_cast<const float4*>(f1 + i), kk = *reinterpret_cast<const float4*>(f2 + i);
+                    S[4 * m] = keep * S[4 * m] + kk.x * v;
+                    S[4 * m + 1] = keep * S[4 * m + 1] + kk.y * v;
+                    S[4 * m + 2] = keep * S[4 * m + 2] + kk.z * v;
+                    S[4 * m + 3] = keep * S[4 * m + 3] + kk.w * v;
+                    o0 += S[4 * m] * qq.x;
+                    o1 += S[4 * m + 1] * qq.y;
+                    o2 += S[4 * m + 2] * qq.z;
+                    o3 += S[4 * m + 3] * qq.w;
+                }
             } else {
                 const float* wd = f2 + dkp;
                 const float v = wd[dkp + lc];
@@ -576,7 +601,7 @@ __global__ void scan_kernel(const ScanArgs a) {
 
 template <int MODE, int R, int L>
 static int launch_scan(const ScanArgs& a, int S, cudaStream_t stream) {
-    const int per_tok = (MODE == PRISM_SCAN_DELTA ? 2 : (MODE == PRISM_SCAN_GENERAL ? 5 : 3)) * a.dkp + a.colsp + 4;
+    const int per_tok = scan_vectors(MODE) * a.dkp + a.colsp + 4;
     const size_t smem = ((size_t)3 * a.TB * per_tok + (MODE == PRISM_SCAN_BONUS ? a.dkp : 0)) * sizeof(float);
     auto kern = scan_kernel<MODE, R, L>;
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
@@ -693,6 +718,7 @@ PRISM_EXPORT int prism_recurrent_scan(int mode, const float* x, long long x_stri
     a.state = state; a.seg_start = seg_start; a.slots = slots; a.out = out; a.H = H; a.rep = rep; a.dk = dk; a.dv = dv;
     a.w_ready = w_ready;
     a.ex = ex; a.es = ex_stride;
+    if (mode == PRISM_SCAN_RETAIN && (w0 == nullptr || rep != 1)) return (int)cudaErrorInvalidValue;
     if (mode == PRISM_SCAN_GENERAL && (ex == nullptr || ww == nullptr || rep != 1)) return (int)cudaErrorInvalidValue;
     // A token's work is one chain (dot product, shuffles, update, dot product, shuffles), so a CTA is latency
     // bound: eight threads a column, four warps of them side by side, and as many CTAs as there are column blocks.
@@ -712,9 +738,9 @@ PRISM_EXPORT int prism_recurrent_scan(int mode, const float* x, long long x_stri
     a.colsp = (cols + 3) / 4 * 4;
     a.vec = dk % 4 == 0 && dv % 4 == 0 && cols % 4 == 0 && x_stride % 4 == 0 && qo % 4 == 0 && ko % 4 == 0 && vo % 4 == 0 &&
             (uintptr_t)x % 16 == 0 && (uintptr_t)state % 16 == 0 &&
-            (mode == PRISM_SCAN_DELTA || (ww_stride % 4 == 0 && (uintptr_t)ww % 16 == 0)) &&
+            (scan_vectors(mode) == 2 || (ww_stride % 4 == 0 && (uintptr_t)ww % 16 == 0)) &&
             (mode != PRISM_SCAN_GENERAL || (ex_stride % 4 == 0 && (uintptr_t)ex % 16 == 0 && ((long long)H * dk) % 4 == 0));
-    const int per_tok = (mode == PRISM_SCAN_DELTA ? 2 : (mode == PRISM_SCAN_GENERAL ? 5 : 3)) * a.dkp + a.colsp + 4;
+    const int per_tok = scan_vectors(mode) * a.dkp + a.colsp + 4;
     int tb = (24 * 1024 / 4) / per_tok;
     tb = tb < 1 ? 1 : (tb > 16 ? 16 : tb);
     a.TB = tb > max_q_len ? (max_q_len < 1 ? 1 : max_q_len) : tb;      // a decode step stages one token, and CTAs are small
@@ -732,6 +758,7 @@ PRISM_EXPORT int prism_recurrent_scan(int mode, const float* x, long long x_stri
     if (mode == PRISM_SCAN_BONUS) PRISM_SCAN(PRISM_SCAN_BONUS);
     if (mode == PRISM_SCAN_CHANNEL) PRISM_SCAN(PRISM_SCAN_CHANNEL);
     if (mode == PRISM_SCAN_GENERAL) PRISM_SCAN(PRISM_SCAN_GENERAL);
+    if (mode == PRISM_SCAN_RETAIN) PRISM_SCAN(PRISM_SCAN_RETAIN);
 #undef PRISM_SCAN
     return (int)cudaErrorInvalidValue;
 }

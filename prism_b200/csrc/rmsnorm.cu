@@ -215,7 +215,156 @@ __global__ void add_rows_kernel(float* __restrict__ residual, const TD* __restri
     }
 }
 
+// A sublayer between two norms: its result is normed before it joins the residual stream, and the next sublayer's norm
+// follows at once.  Per row, one block, one launch:
+//   d = sum_s delta[s, r, :];   x = residual[r, :] + d * rsqrt(mean(d^2) + eps_d) * wd;   residual[r, :] = x  (float32)
+//   out[i, :] = x * rsqrt(mean(x^2) + eps) * w
+// rows (optional): only these rows, and the residual rows are then left alone (nothing reads them afterwards).
+template <typename TD, typename TO>
+__global__ void add_normed_rmsnorm_kernel(float* __restrict__ residual, const TD* __restrict__ delta_in, int nsplit,
+                                          size_t split_stride, const void* __restrict__ wd, int wd_bf16, float eps_d,
+                                          const void* __restrict__ weight, int weight_bf16, float eps, TO* __restrict__ out,
+                                          const int* __restrict__ rows, int H) {
+    pdl_trigger();
+    pdl_wait();
+    const TD* delta = pdl_fresh(delta_in);
+    extern __shared__ float row[];                 // [H]: the summed delta, then the new residual row
+    __shared__ float scratch[33];
+    const int i = blockIdx.x;
+    const int r = rows ? rows[i] : i;
+    float* res = pdl_fresh(residual) + (size_t)r * H;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        float v = 0.f;
+        for (int s = 0; s < nsplit; ++s) v += to_float(delta[(size_t)s * split_stride + (size_t)r * H + c]);
+        row[c] = v;
+        ss += v * v;
+    }
+    ss = block_sum(ss, scratch);
+    const float inv_d = 1.f / sqrtf(ss / (float)H + eps_d);
+    ss = 0.f;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        const float v = res[c] + row[c] * inv_d * load_param(wd, wd_bf16, c);
+        row[c] = v;
+        if (rows == nullptr) res[c] = v;
+        ss += v * v;
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.f / sqrtf(ss / (float)H + eps);
+    TO* o = out + (size_t)i * H;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_float<TO>(row[c] * inv * load_param(weight, weight_bf16, c));
+}
+
+// Vector version for H % 8 == 0 and H <= 8 * 1024 * ITERS: everything in registers, both weights read before the wait.
+template <typename TD, typename TO, int ITERS>
+__global__ void __launch_bounds__(1024) add_normed_rmsnorm_vec_kernel(float* __restrict__ residual, const TD* __restrict__ delta_in,
+                                                                      int nsplit, size_t split_stride, const void* __restrict__ wd,
+                                                                      int wd_bf16, float eps_d, const void* __restrict__ weight,
+                                                                      int weight_bf16, float eps, TO* __restrict__ out,
+                                                                      const int* __restrict__ rows, int H) {
+    pdl_trigger();
+    float a[ITERS][8], w[ITERS][8];
+#pragma unroll
+    for (int it = 0; it < ITERS; ++it) {
+        const int c = (threadIdx.x + it * blockDim.x) * 8;
+        if (c < H) {
+            load_param8(wd, wd_bf16, c, a[it]);
+            load_param8(weight, weight_bf16, c, w[it]);
+        }
+    }
+    pdl_wait();
+    const TD* delta = pdl_fresh(delta_in);
+    __shared__ float scratch[33];
+    const int i = blockIdx.x;
+    const int r = rows ? rows[i] : i;
+    float* res = pdl_fresh(residual) + (size_t)r * H;
+    float x[ITERS][8], d[ITERS][8];
+    float ss = 0.f;
+#pragma unroll
+    for (int it = 0; it < ITERS; ++it) {
+        const int c = (threadIdx.x + it * blockDim.x) * 8;
+        if (c < H) {
+            load8(res + c, x[it]);                 // on its way while the delta is summed
+            const TD* d0 = delta + (size_t)r * H + c;
+            load8(d0, d[it]);
+            for (int s = 1; s < nsplit; ++s) {
+                float e[8];
+                load8(d0 + (size_t)s * split_stride, e);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) d[it][k] += e[k];
+            }
+#pragma unroll
+            for (int k = 0; k < 8; ++k) ss += d[it][k] * d[it][k];
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float inv_d = 1.f / sqrtf(ss / (float)H + eps_d);
+    ss = 0.f;
+#pragma unroll
+    for (int it = 0; it < ITERS; ++it) {
+        const int c = (threadIdx.x + it * blockDim.x) * 8;
+        if (c < H) {
+#pragma unroll
+            for (int k = 0; k < 8; ++k) {
+                x[it][k] += d[it][k] * inv_d * a[it][k];
+                ss += x[it][k] * x[it][k];
+            }
+            if (rows == nullptr) store8(res + c, x[it]);
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.f / sqrtf(ss / (float)H + eps);
+    TO* o = out + (size_t)i * H;
+#pragma unroll
+    for (int it = 0; it < ITERS; ++it) {
+        const int c = (threadIdx.x + it * blockDim.x) * 8;
+        if (c < H) {
+#pragma unroll
+            for (int k = 0; k < 8; ++k) w[it][k] *= x[it][k] * inv;
+            store8(o + c, w[it]);
+        }
+    }
+}
+
 }  // namespace prism
+
+// residual float32 [T, H] in place; delta [nsplit, T, H] of delta_dtype, normed with wd and eps_d before it is added; out
+// [nrows, H] of out_dtype: the norm (weight, eps) of the new rows, for all of them or for `rows` (the residual is then
+// not written).
+PRISM_EXPORT int prism_add_normed_rmsnorm(float* residual, const void* delta, int delta_dtype, int nsplit, long long split_stride,
+                                          const void* wd, int wd_dtype, float eps_d, const void* weight, int weight_dtype,
+                                          float eps, void* out, int out_dtype, const int* rows, int nrows, int H,
+                                          cudaStream_t stream) {
+    if (nrows <= 0) return 0;
+    if (nsplit < 1 || delta == nullptr || wd == nullptr || H < 1 || H > 50000) return (int)cudaErrorInvalidValue;
+    const int db = wd_dtype == PRISM_DTYPE_BF16, wb = weight_dtype == PRISM_DTYPE_BF16;
+    const int chunks = H / 8;
+    const bool vec = H % 8 == 0 && chunks <= 2048 && split_stride % 8 == 0 && (uintptr_t)residual % 32 == 0 &&
+                     (uintptr_t)delta % 32 == 0 && (uintptr_t)out % 32 == 0 && (uintptr_t)weight % 32 == 0 && (uintptr_t)wd % 32 == 0;
+    const int iters = chunks > 1024 ? 2 : 1;
+    const int threads = vec ? ((chunks + iters - 1) / iters + 31) / 32 * 32 : (H >= 4096 ? 512 : (H >= 1024 ? 256 : 128));
+    const size_t smem = vec ? 0 : (size_t)H * sizeof(float);
+#define ARGS residual, (const TD*)delta, nsplit, (size_t)split_stride, wd, db, eps_d, weight, wb, eps, (TO*)out, rows, H
+#define LAUNCH(TDx, TOx)                                                                                                  \
+    do {                                                                                                                  \
+        using TD = TDx; using TO = TOx;                                                                                   \
+        auto plain = prism::add_normed_rmsnorm_kernel<TD, TO>;                                                            \
+        if (smem > 40 * 1024) cudaFuncSetAttribute(plain, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);        \
+        if (vec && iters == 1)                                                                                            \
+            return (int)prism::launch_kernel(prism::add_normed_rmsnorm_vec_kernel<TD, TO, 1>, dim3(nrows), dim3(threads), 0, stream, ARGS); \
+        if (vec)                                                                                                          \
+            return (int)prism::launch_kernel(prism::add_normed_rmsnorm_vec_kernel<TD, TO, 2>, dim3(nrows), dim3(threads), 0, stream, ARGS); \
+        return (int)prism::launch_kernel(plain, dim3(nrows), dim3(threads), smem, stream, ARGS);                          \
+    } while (0)
+    if (delta_dtype == PRISM_DTYPE_BF16) {
+        if (out_dtype == PRISM_DTYPE_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
+        LAUNCH(__nv_bfloat16, float);
+    }
+    if (out_dtype == PRISM_DTYPE_BF16) LAUNCH(float, __nv_bfloat16);
+    LAUNCH(float, float);
+#undef LAUNCH
+#undef ARGS
+}
 
 // x float32 [rows, H] in place; delta (null: none) [nsplit, rows, H] of delta_dtype; copy (null: none) [rows, H] of
 // copy_dtype.

@@ -95,6 +95,7 @@ class _Sig:
     prism_attention_masked_supported = [_i, _i, _i, _i]
     prism_attention_masked_bf16 = [_p, _ll, _i, _p, _ll, _p, _ll, _i, _p, _ll, _i, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i,
                                    _i, _i, _i, _i, _i, _f, _p, _i, _i, _i, _p, _p, _p, _p, _i, _p]
+    prism_add_normed_rmsnorm = [_p, _p, _i, _i, _ll, _p, _i, _f, _p, _i, _f, _p, _i, _p, _i, _i, _p]
     prism_scale_add_rmsnorm = [_p, _f, _p, _i, _i, _ll, _p, _i, _f, _p, _i, _i, _i, _p]
     prism_gated_product = [_p, _ll, _p, _ll, _p, _ll, _i, _i, _i, _i, _f, _i, _p]
     prism_qk_norm_rope_store = [_p, _p, _p, _ll, _p, _i, _p, _i, _f, _p, _i, _p, _p, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i,
@@ -121,10 +122,10 @@ class _Sig:
     prism_rglru_scan = [_p, _p, _ll, _p, _ll, _p, _p, _p, _i, _i, _i, _p, _i, _ll, _p]
     prism_cache_store = [_p, _ll, _p, _i, _i, _p, _ll, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i, _p, _p]
     prism_latent_kv_store = [_p, _ll, _p, _i, _f, _i, _i, _i, _p, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i, _p, _p, _i, _p, _i,
-                             _p, _ll, _p]
-    prism_rotate_slice = [_p, _ll, _i, _p, _ll, _i, _i, _i, _i, _p, _p, _i, _i, _p]
+                             _p, _ll, _i, _f, _p]
+    prism_rotate_slice = [_p, _ll, _i, _p, _ll, _i, _i, _i, _i, _p, _p, _i, _i, _i, _f, _f, _p]
     prism_activation = [_p, _ll, _p, _ll, _i, _i, _i, _i, _p]
-    prism_glu = [_p, _ll, _p, _ll, _i, _i, _i, _i, _p]
+    prism_glu = [_p, _ll, _p, _ll, _i, _i, _i, _i, _f, _p]
     prism_gather_gate = [_p, _ll, _p, _p, _i, _ll, _i, _i, _p, _i, _ll, _i, _i, _i, _p, _p]
     prism_softcap = [_p, _ll, _f, _p]
     prism_add_rows = [_p, _p, _i, _i, _ll, _p, _i, _i, _i, _p]
@@ -146,7 +147,7 @@ class _Sig:
     prism_argmax_split = [_p, _i, _i, _i, _i, _p, _p, _p, _p, _p]
     prism_set_pdl = [_i]
     prism_gemm_tcgen05_supported = [_i, _i, _i]
-    prism_gemm_tcgen05 = [_p, _i, _p, _i, _p, _i, _p, _i, _i, _i, _i, _i, _i, _p, _p, _p, _i, _i, _p]
+    prism_gemm_tcgen05 = [_p, _i, _p, _i, _p, _i, _p, _i, _i, _i, _i, _i, _i, _p, _p, _p, _i, _i, _f, _p]
     prism_gemv_bf16_supported = [_i, _i, _i]
     prism_gemv_bf16 = [_p, _i, _p, _i, _p, _i, _p, _i, _i, _i, _i, _i, _p]
 
@@ -216,6 +217,23 @@ def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: t
                                    _dt(out), _ptr(rows), n, H, _stream()), "add_rmsnorm")
 
 
+def add_normed_rmsnorm(residual: torch.Tensor, delta: torch.Tensor, delta_weight: torch.Tensor, delta_eps: float,
+                       weight: torch.Tensor, eps: float, out: torch.Tensor, rows: Optional[torch.Tensor] = None):
+    """``x = residual + rmsnorm(delta) * delta_weight`` (float32, in place; ``delta [T, H]`` or a stack ``[k, T, H]`` of
+    partial sums, normed as their sum), then ``out = rmsnorm(x) * weight``: the norm behind one sublayer, the residual sum
+    and the norm before the next in one launch.  ``rows`` (int32): only these rows, and the residual is not written."""
+    _cuda(residual, delta, delta_weight, weight, out, rows)
+    assert residual.dtype == torch.float32 and residual.is_contiguous() and out.is_contiguous() and delta.is_contiguous()
+    T, H = residual.shape
+    assert delta.shape[-2:] == (T, H) and delta_weight.shape == weight.shape == (H,)
+    n = T if rows is None else rows.shape[0]
+    assert out.shape == (n, H)
+    _check(lib().prism_add_normed_rmsnorm(_ptr(residual), _ptr(delta), _dt(delta), 1 if delta.dim() == 2 else delta.shape[0],
+                                          T * H, _ptr(delta_weight), _dt(delta_weight), float(delta_eps), _ptr(weight),
+                                          _dt(weight), float(eps), _ptr(out), _dt(out), _ptr(rows), n, H, _stream()),
+           "add_normed_rmsnorm")
+
+
 def sgemm(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor):
     """True float32 ``out = x @ w.T + bias`` on CUDA cores."""
     _cuda(x, w, bias, out)
@@ -257,6 +275,8 @@ def gemv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: to
 
 EPI_PARTIAL = 3
 EPI_GEGLU = 4          # the paired epilogue with the gate through gelu_tanh instead of silu
+EPI_CLAMPED = 5        # the paired epilogue in the clamped form (``glu``), with a limit
+_PAIRED = (EPI_SWIGLU, EPI_GEGLU, EPI_CLAMPED)
 _tc_err = {}
 
 
@@ -292,7 +312,7 @@ def _tc_workspace(device, floats: int, tiles: int):
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
-            epi: int = EPI_BF16, ksplit: int = 1, err: Optional[torch.Tensor] = None, group_rows: int = 0):
+            epi: int = EPI_BF16, ksplit: int = 1, err: Optional[torch.Tensor] = None, group_rows: int = 0, limit: float = 0.0):
     """tcgen05 + TMA weight-streaming product for up to 64 tokens.  ``epi``:
     ``EPI_BF16`` / ``EPI_F32`` (``out [M, N]``, + bias), ``EPI_SWIGLU`` (``w`` is
     the fused ``[2N, K]`` gate/up weight), ``EPI_PARTIAL`` (``out`` float32
@@ -308,11 +328,11 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out:
     N = out.shape[-1]
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[1] == K
     assert x.stride(1) == 1 and w.stride(1) == 1 and out.is_contiguous()
-    assert w.shape[0] == (2 * N if epi in (EPI_SWIGLU, EPI_GEGLU) else N)
+    assert w.shape[0] == (2 * N if epi in _PAIRED else N)
     if epi == EPI_PARTIAL:
         assert out.dtype == torch.float32 and out.shape == (ksplit, M, N) and bias is None
     else:
-        assert out.shape == (M, N) and (ksplit == 1 or epi not in (EPI_SWIGLU, EPI_GEGLU))
+        assert out.shape == (M, N) and (ksplit == 1 or epi not in _PAIRED)
         assert out.dtype == (torch.float32 if epi == EPI_F32 else torch.bfloat16)
     err = err if err is not None else _tc_err_word(x.device)
     ws = cnt = None
@@ -320,7 +340,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out:
         ws, cnt = _tc_workspace(x.device, ksplit * M * N, (N + 127) // 128)
     _check(lib().prism_gemm_tcgen05(_ptr(w), w.stride(0), _ptr(x), x.stride(0) if M > 1 else K, _ptr(bias),
                                     F32 if bias is None else _dt(bias), _ptr(out), N, M, N, K, epi, ksplit,
-                                    _ptr(ws), _ptr(cnt), _ptr(err), int(group_rows), int(group_tokens), _stream()),
+                                    _ptr(ws), _ptr(cnt), _ptr(err), int(group_rows), int(group_tokens), float(limit), _stream()),
            "gemm_tcgen05")
 
 
@@ -1309,12 +1329,12 @@ def latent_kv_store(x: torch.Tensor, weight: torch.Tensor, eps: float, rank: int
                     inv_freq: Optional[torch.Tensor], plane: torch.Tensor, block_table: torch.Tensor,
                     positions: torch.Tensor, tok_seg: torch.Tensor, num_pages: int, max_pos: int, err: torch.Tensor,
                     xq: Optional[torch.Tensor] = None, q_weight: Optional[torch.Tensor] = None,
-                    q_out: Optional[torch.Tensor] = None):
+                    q_out: Optional[torch.Tensor] = None, interleaved: bool = False, amplitude: float = 1.0):
     """The cache row of latent attention from its down projection ``x [T, rank + r]`` (float32): the first
     ``rank`` entries RMS-normed with ``weight``, the last ``r`` with their first ``rot_dims`` entries rotated
     by the token's position; stored at the token's slot of ``plane [pages, P, 1, rank + r]``.  ``xq [T, q_rank]``
     (float32, another column block of the same matrix as ``x``): RMS-normed with ``q_weight`` into ``q_out`` by the
-    same launch."""
+    same launch.  ``interleaved``: pairs (2i, 2i + 1) instead of halves; ``amplitude``: a factor on cosine and sine."""
     _cuda(x, weight, inv_freq, plane, block_table, positions, tok_seg, xq, q_weight, q_out)
     T, width = x.shape
     r = width - rank
@@ -1333,19 +1353,21 @@ def latent_kv_store(x: torch.Tensor, weight: torch.Tensor, eps: float, rank: int
                                        block_table.shape[1], _ptr(positions), _ptr(tok_seg), T, plane.shape[1], num_pages,
                                        int(max_pos), _ptr(err), _ptr(xq), q_rank, _ptr(q_weight),
                                        F32 if q_weight is None else _dt(q_weight), _ptr(q_out),
-                                       0 if q_out is None else q_out.stride(0), _stream()), "latent_kv_store")
+                                       0 if q_out is None else q_out.stride(0), 1 if interleaved else 0, float(amplitude), _stream()),
+           "latent_kv_store")
 
 
 def rotate_slice(src: torch.Tensor, dst: torch.Tensor, rot_dims: int, inv_freq: Optional[torch.Tensor],
-                 positions: torch.Tensor):
-    """``dst[t, h, :] = src[t, h, :]`` with the first ``rot_dims`` entries rotated by token t's position (entry
-    i paired with i + rot_dims / 2).  ``src`` and ``dst`` are ``[T, nh, width]`` views with token and head
-    strides of their own."""
+                 positions: torch.Tensor, interleaved: bool = False, amplitude: float = 1.0, scale: float = 1.0):
+    """``dst[t, h, :] = scale * src[t, h, :]`` with the first ``rot_dims`` entries rotated by token t's position (entry
+    i paired with i + rot_dims / 2; ``interleaved``: 2i with 2i + 1; ``amplitude``: a factor on cosine and sine).  ``src``
+    and ``dst`` (they may be the same) are ``[T, nh, width]`` views with token and head strides of their own."""
     _cuda(src, dst, inv_freq, positions)
     T, nh, width = src.shape
     assert dst.shape == src.shape and dst.dtype == src.dtype and src.stride(2) == 1 and dst.stride(2) == 1
     _check(lib().prism_rotate_slice(_ptr(src), src.stride(0), src.stride(1), _ptr(dst), dst.stride(0), dst.stride(1),
-                                    _dt(src), width, int(rot_dims), _ptr(inv_freq), _ptr(positions), T, nh, _stream()),
+                                    _dt(src), width, int(rot_dims), _ptr(inv_freq), _ptr(positions), T, nh, 1 if interleaved else 0,
+                                    float(amplitude), float(scale), _stream()),
            "rotate_slice")
 
 
@@ -1361,14 +1383,18 @@ def activation(x: torch.Tensor, out: torch.Tensor, kind: str):
                                   ACTIVATIONS[kind], _stream()), "activation")
 
 
-def glu(gu: torch.Tensor, out: torch.Tensor, kind: str):
+GATED = ("silu", "gelu_tanh", "clamped")      # hidden layers of a gated feed-forward
+
+
+def glu(gu: torch.Tensor, out: torch.Tensor, kind: str, limit: float = 0.0):
     """``out[t, i] = act(gu[t, i]) * gu[t, I + i]``: the hidden layer of a gated feed-forward whose gate and up
-    projections are one product (gate columns first).  ``kind``: ``silu`` or ``gelu_tanh``."""
+    projections are one product (gate columns first).  ``kind``: ``silu``, ``gelu_tanh`` or ``clamped``: with ``g =
+    min(gate, limit)`` and ``u`` the up part clamped to ``[-limit, limit]``, ``g sigmoid(1.702 g) (u + 1)``."""
     _cuda(gu, out)
     rows, I = out.shape
     assert gu.shape == (rows, 2 * I) and gu.dtype == out.dtype and gu.stride(1) == 1 and out.stride(1) == 1
-    _check(lib().prism_glu(_ptr(gu), gu.stride(0), _ptr(out), out.stride(0), _dt(gu), rows, I, ACTIVATIONS[kind], _stream()),
-           "glu")
+    _check(lib().prism_glu(_ptr(gu), gu.stride(0), _ptr(out), out.stride(0), _dt(gu), rows, I,
+                           6 if kind == "clamped" else ACTIVATIONS[kind], float(limit), _stream()), "glu")
 
 
 def gather_gate(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, offset: int, out: torch.Tensor, kind: str,
@@ -1409,19 +1435,22 @@ def add_rows(residual: torch.Tensor, delta: Optional[torch.Tensor], copy: Option
                                 F32 if copy is None else _dt(copy), T, H, _stream()), "add_rows")
 
 
-def feed_forward_glu(ctx, x: torch.Tensor, gate_up_w: torch.Tensor, down_w: torch.Tensor, kind: str):
-    """``down(act(gate(x)) * up(x))`` with the fused gate/up weight and ``act`` one of ``silu``, ``gelu_tanh``; silu
-    takes the path with the activation in the product's epilogue (``feed_forward_swiglu``)."""
+def glu_hidden(ctx, x: torch.Tensor, gate_up_w: torch.Tensor, kind: str, limit: float = 0.0) -> torch.Tensor:
+    """The hidden layer of a gated feed-forward (``glu`` of the product with the fused gate/up weight); for a few tokens
+    the gated activation is the product's epilogue."""
+    act = ctx.alloc((x.shape[0], gate_up_w.shape[0] // 2), x.dtype)
+    if tc_gemm_ok(x, gate_up_w, TC_GEMM_MAX_M_SWIGLU):
+        gemm_tc(x, gate_up_w, None, act, {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU, "clamped": EPI_CLAMPED}[kind], limit=limit)
+    else:
+        glu(linear(x, gate_up_w), act, kind, limit)
+    return act
+
+
+def feed_forward_glu(ctx, x: torch.Tensor, gate_up_w: torch.Tensor, down_w: torch.Tensor, kind: str, limit: float = 0.0):
+    """``down(glu(x))`` with the fused gate/up weight; ``kind`` and ``limit`` as in ``glu``."""
     if kind == "silu":
         return feed_forward_swiglu(ctx, x, gate_up_w, down_w)
-    if tc_gemm_ok(x, gate_up_w, TC_GEMM_MAX_M_SWIGLU):
-        act = ctx.alloc((x.shape[0], gate_up_w.shape[0] // 2), x.dtype)
-        gemm_tc(x, gate_up_w, None, act, EPI_GEGLU)        # gate/up product with the gated activation in its epilogue
-        return linear_delta(act, down_w)
-    gu = linear(x, gate_up_w)
-    act = ctx.alloc((x.shape[0], gate_up_w.shape[0] // 2), x.dtype)
-    glu(gu, act, kind)
-    return linear_delta(act, down_w)
+    return linear_delta(glu_hidden(ctx, x, gate_up_w, kind, limit), down_w)
 
 
 def masked_attention(ctx, q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor,
@@ -1715,7 +1744,7 @@ def headnorm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps
                                      {"silu": 0, "sigmoid": 1, "none": 2}[gate_act], _stream()), "headnorm_gate")
 
 
-SCAN_DELTA, SCAN_BONUS, SCAN_CHANNEL, SCAN_GENERAL = 0, 1, 2, 3      # csrc/recurrent.cu: PRISM_SCAN_*
+SCAN_DELTA, SCAN_BONUS, SCAN_CHANNEL, SCAN_GENERAL, SCAN_RETAIN = 0, 1, 2, 3, 4      # csrc/recurrent.cu: PRISM_SCAN_*
 
 
 def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, ctx, H: int,
@@ -1730,7 +1759,8 @@ def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
     itself (``lowrank_decay``, ``decay_from_exponent``).  ``SCAN_CHANNEL``: delta rule whose decay is a vector over the
     key channels, ``ww [T, H * dk]`` (the decay itself), with ``bg [T, H]`` (beta).  ``SCAN_GENERAL``: the generalized
     delta rule ``S <- diag(w) S - c (e^T S) + k v^T; o = S^T r`` with the decay ``ww [T, H * dk]`` and ``ex [T, 2 H dk]``
-    = unit key e | removal rate times e (``unit_removal``); every head has its own r and k.  ``out [T, H, dv]`` float32."""
+    = unit key e | removal rate times e (``unit_removal``); every head has its own r and k.  ``SCAN_RETAIN``: ``S <- w0[h] S
+    + k v^T; o = S^T q`` with one constant decay per head, ``w0 [H]``.  ``out [T, H, dv]`` float32."""
     _cuda(q, k, v, state, out, bg, ww, w0, u, ex)
     T = q.shape[0]
     for t in (q, k, v):
@@ -1747,6 +1777,8 @@ def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
     elif mode == SCAN_GENERAL:
         assert rep == 1 and ww.dtype == torch.float32 and ww.shape == (T, H * dk) and ww.stride(1) == 1
         assert ex is not None and ex.dtype == torch.float32 and ex.shape == (T, 2 * H * dk) and ex.is_contiguous()
+    elif mode == SCAN_RETAIN:
+        assert rep == 1 and w0.numel() == H and w0.is_contiguous()
     else:
         assert ww.dtype == torch.float32 and ww.shape == (T, H * dk) and ww.stride(1) == 1
         assert w0.numel() == H * dk and u.numel() == H * dk and w0.is_contiguous() and u.is_contiguous()
@@ -1759,6 +1791,24 @@ def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
         _ptr(state), _ptr(ctx.seg_start), _ptr(ctx.state_slots), ctx.S, int(getattr(ctx, "max_q_len", None) or T), H, rep, dk, dv,
         _ptr(out), 1 if decay_ready else 0, _ptr(ex), 0 if ex is None else ex.stride(0), _stream()),
         "recurrent_scan")
+
+
+def retention(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, rot, decay: torch.Tensor, state: torch.Tensor, eps: float,
+              ones: torch.Tensor, out: torch.Tensor):
+    """Retention between its input and its output projection, for the step's tokens: from the float32 product ``proj [T,
+    H (2 dk + 2 dv)]`` (columns q | k | v | gate; q and k are rotated in place by ``rot``, a ``RotaryParams`` or None, and k
+    multiplied by ``dk^-1/2``), ``S <- decay[h] S + k v^T; o = S^T q`` from and into ``state [slots, H, dv, dk]``, ``out = o /
+    rms(o) * silu(gate)`` in the compute dtype."""
+    T, A, B = proj.shape[0], H * dk, H * dv
+    q, k = proj[:, :A].view(T, H, dk), proj[:, A:2 * A].view(T, H, dk)
+    rd, freq = (rot.rotary_dim, rot.inv_freq) if rot is not None else (0, None)
+    il, amp = (rot.interleaved, rot.amplitude) if rot is not None else (False, 1.0)
+    if rd:
+        rotate_slice(q, q, rd, freq, ctx.positions, il, amp)
+    rotate_slice(k, k, rd, freq, ctx.positions, il, amp, dk ** -0.5)
+    o = ctx.alloc((T, H, dv), torch.float32)
+    recurrent_scan(SCAN_RETAIN, proj[:, :A], proj[:, A:2 * A], proj[:, 2 * A:2 * A + B], state, ctx, H, 1, dk, dv, o, w0=decay)
+    headnorm_gate(o, proj[:, 2 * A + B:], ones, eps, 1.0, out)
 
 
 def unit_removal(k: torch.Tensor, a: torch.Tensor, a_bias: Optional[torch.Tensor], unit_eps: float, H: int, dk: int,

@@ -18,7 +18,7 @@ from typing import Optional
 import torch
 
 from ..config.model_config import ConfigError
-from .base import CacheNeed, DetachedProjection, Mixer, ParamSpec, PartSpec, WeightSource, build_part, register_part
+from .base import CacheNeed, DetachedProjection, Mixer, ParamSpec, PartSpec, RotaryParams, WeightSource, build_part, register_part
 from .. import ops
 
 
@@ -351,16 +351,22 @@ class LatentAttention(Mixer):
     key/value head whose values are the first ``kv_rank`` entries of its key rows.
 
     ``window``: sliding window (None: all keys).  ``rope_dims`` (default ``rot_dim``): how many entries of the
-    rotated part really turn.  ``names``: the tensors' names in the model file.
+    rotated part really turn (in halves).  ``position``: a rotary part that says how it turns instead (pairs, frequency
+    scaling, a factor on cosine and sine; ``rope_base`` and ``rope_dims`` are then not used).  ``sink``: a learned number
+    per head whose exponential joins the softmax's denominator, unscaled and without a value.  ``gate``: the
+    concatenated heads are multiplied by ``sigmoid(W_g h)`` before the output projection; its rows ride in the down
+    projections' product.  ``names``: the tensors' names in the model file.
     """
 
     NAMES = dict(dq="q_a_proj.weight", dq_norm="q_a_layernorm.weight", uq="q_b_proj.weight",
                  dkv="kv_a_proj_with_mqa.weight", dkv_norm="kv_a_layernorm.weight", uk="k_b_proj.weight",
-                 uv="v_b_proj.weight", o="o_proj.weight")
+                 uv="v_b_proj.weight", o="o_proj.weight", sink="sinks", g="g_proj.weight")
+    graph_safe = True
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, q_rank: int,
                  kv_rank: int, eps: float, rope_base: float = 10000.0, rope_dims: Optional[int] = None,
-                 window: Optional[int] = None, scale: Optional[float] = None, names: Optional[dict] = None):
+                 window: Optional[int] = None, scale: Optional[float] = None, names: Optional[dict] = None,
+                 position: Optional[PartSpec] = None, sink: bool = False, gate: bool = False):
         self.hidden_size, self.nh, self.hd = int(hidden_size), int(num_heads), int(head_dim)
         self.rd, self.vhd, self.q_rank, self.kv_rank = int(rot_dim), int(v_head_dim), int(q_rank), int(kv_rank)
         self.eps, self.rope_base = float(eps), float(rope_base)
@@ -375,6 +381,8 @@ class LatentAttention(Mixer):
         self.scale = float(scale) if scale is not None else (self.hd + self.rd) ** -0.5
         self.names = dict(self.NAMES, **(names or {}))
         self.mask = ops.KeyMask.window(self.window)
+        self.position = self.add_child("position", build_part("position", position)) if position else None
+        self.sink, self.gate = bool(sink), bool(gate)
         self._own_out = True
 
     def cache_need(self):
@@ -384,13 +392,15 @@ class LatentAttention(Mixer):
         H, nh, n = self.hidden_size, self.nh, self.names
         return [
             ParamSpec("down_w", (WeightSource(n["dq"], (self.q_rank, H)),
-                                 WeightSource(n["dkv"], (self.kv_rank + self.rd, H)))),
+                                 WeightSource(n["dkv"], (self.kv_rank + self.rd, H)))
+                      + ((WeightSource(n["g"], (nh * self.vhd, H)),) if self.gate else ())),
             ParamSpec("dq_norm", (WeightSource(n["dq_norm"], (self.q_rank,), "norm"),)),
             ParamSpec("dkv_norm", (WeightSource(n["dkv_norm"], (self.kv_rank,), "norm"),)),
             ParamSpec("uq_w", (WeightSource(n["uq"], (nh * (self.hd + self.rd), self.q_rank)),)),
             ParamSpec("uk_w", (WeightSource(n["uk"], (nh * self.hd, self.kv_rank)),)),
             ParamSpec("uv_w", (WeightSource(n["uv"], (nh * self.vhd, self.kv_rank)),)),
-        ] + ([ParamSpec("o_w", (self._o_source(),))] if self._own_out else [])
+        ] + ([ParamSpec("sink", (WeightSource(n["sink"], (nh,), "bias"),))] if self.sink else []) \
+          + ([ParamSpec("o_w", (self._o_source(),))] if self._own_out else [])
 
     detachable_out = True        # the down projections feed norms and stay float32: they are not handed over
 
@@ -402,9 +412,14 @@ class LatentAttention(Mixer):
         return DetachedProjection(self.handed_over(self._o_source()), (), self.nh * self.vhd)
 
     def on_bound(self):
-        half = self.rope_dims // 2
-        i = torch.arange(half, dtype=torch.float64)
-        self.inv_freq = (self.rope_base ** (-2.0 * i / max(self.rope_dims, 1))).to(torch.float32).to(self.device)
+        if self.position is not None:
+            self.rot = self.position.rotary()
+            if self.rot is None or self.rot.rotary_dim > self.rd:
+                raise ConfigError(f"latent attention takes a rotary position encoding of at most rot_dim {self.rd} entries")
+        else:
+            i = torch.arange(self.rope_dims // 2, dtype=torch.float64)
+            inv = (self.rope_base ** (-2.0 * i / max(self.rope_dims, 1))).to(torch.float32).to(self.device)
+            self.rot = RotaryParams(inv, self.rope_dims)
         # W_uk per head, turned so that a head's plain query part is projected into the latent space
         self.uk_t = self.w["uk_w"].view(self.nh, self.hd, self.kv_rank).transpose(1, 2).contiguous()     # [nh, R, hd]
         self.uv = self.w["uv_w"].view(self.nh, self.vhd, self.kv_rank)                                  # [nh, vhd, R]
@@ -415,20 +430,26 @@ class LatentAttention(Mixer):
         return ops.linear_delta(attn, self.w["o_w"])
 
     def forward_inner(self, ctx, x, cache, out, proj=None):
-        T, nh, hd, rd, R = x.shape[0], self.nh, self.hd, self.rd, self.kv_rank
-        # both down projections in one product; float32, because each feeds a norm
+        T, nh, hd, rd, R, rot = x.shape[0], self.nh, self.hd, self.rd, self.kv_rank, self.rot
+        # both down projections (and the gate) in one product; float32, because each feeds a norm
         down = ops.linear(x, self.w["down_w"], None, out_dtype=torch.float32)
         cq = ctx.alloc((T, self.q_rank), x.dtype)
         # one launch: the query latent normed, the key/value latent normed, the shared key part rotated, the row stored
-        ops.latent_kv_store(down[:, self.q_rank:], self.w["dkv_norm"], self.eps, R, self.rope_dims, self.inv_freq,
+        g0 = self.q_rank + R + rd                                  # first column of the gate
+        ops.latent_kv_store(down[:, self.q_rank:g0], self.w["dkv_norm"], self.eps, R, rot.rotary_dim, rot.inv_freq,
                             cache.k, cache.block_table, ctx.positions, ctx.tok_seg, cache.num_pages, ctx.max_positions,
-                            ctx.err, xq=down[:, :self.q_rank], q_weight=self.w["dq_norm"], q_out=cq)
+                            ctx.err, xq=down[:, :self.q_rank], q_weight=self.w["dq_norm"], q_out=cq,
+                            interleaved=rot.interleaved, amplitude=rot.amplitude)
         q = ops.linear(cq, self.w["uq_w"]).view(T, nh, hd + rd)
         qf = ctx.alloc((T, nh, R + rd), x.dtype)                   # per head [plain part in latent space | rotated part]
         ops.matmul_heads(q[:, :, :hd], self.uk_t, qf[:, :, :R])
         if rd:
-            ops.rotate_slice(q[:, :, hd:], qf[:, :, R:], self.rope_dims, self.inv_freq, ctx.positions)
+            ops.rotate_slice(q[:, :, hd:], qf[:, :, R:], rot.rotary_dim, rot.inv_freq, ctx.positions, rot.interleaved,
+                             rot.amplitude)
         lat = ctx.alloc((T, nh * R), x.dtype)
         ops.masked_attention(ctx, qf, lat, cache.k, cache.k[..., :R], cache.block_table, cache.num_pages, self.mask,
-                             self.scale, None)
-        ops.matmul_heads(lat.view(T, nh, R), self.uv, out.view(T, nh, self.vhd))
+                             self.scale, self.w["sink"] if self.sink else None)
+        heads = ctx.alloc((T, nh * self.vhd), x.dtype) if self.gate else out
+        ops.matmul_heads(lat.view(T, nh, R), self.uv, heads.view(T, nh, self.vhd))
+        if self.gate:
+            ops.gated_product(heads, down[:, g0:], out, "sigmoid")

@@ -125,6 +125,7 @@ class RotaryParams:
     inv_freq: object          # torch.Tensor [rotary_dim // 2] float32
     rotary_dim: int
     interleaved: bool = False # pairs (2i, 2i + 1) instead of (i, i + rotary_dim / 2)
+    amplitude: float = 1.0    # a factor on cosine and sine
 
 
 @dataclass
@@ -135,6 +136,15 @@ class StreamUpdate:
     delta: object
     mix: object
     out: object
+
+
+@dataclass
+class NormedDelta:
+    """A sublayer's result that is normed before it joins the residual stream, left open: ``x <- x + rmsnorm(delta) *
+    weight`` (``delta``: ``[T, W]`` or a stack of partial sums).  The next norm carries it out in its own launch."""
+    delta: object
+    weight: object
+    eps: float
 
 
 @dataclass(frozen=True)

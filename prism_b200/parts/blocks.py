@@ -6,6 +6,7 @@ a short causal convolution beside a skip path on what the mixer reads, no
 feed-forward, a per-layer token input after the feed-forward.
 ``parallel``: one norm whose output both the mixer and the feed-forward read;
 their two results are added to the residual stream together.
+``sandwich``: a norm before and after every sublayer.
 ``postnorm``: the residual stream itself is normed after every sum,
 ``x <- norm(alpha x + sublayer(x))``, and the sublayers read x as it is.
 ``hyper``: pre-norm sublayers around a residual stream kept in several
@@ -134,6 +135,34 @@ class PreNormBlock(Block):
             d = self.feed_forward.forward(ctx, h)
         if self.side is not None:
             d = self._token_side(ctx, residual, d)
+        return residual, d
+
+
+@register_part("block", "sandwich")
+class SandwichBlock(Block):
+    """``x += mixer_post(mixer(mixer_norm(x)))``, then ``x += ff_post(feed_forward(ff_norm(x)))``: a norm before and
+    after each sublayer.  The norm after a sublayer, the residual sum and the norm before the next sublayer (the next
+    block's, or the final norm) are one launch: each result is left open as a ``NormedDelta``.  ``feed_forward`` None: the
+    layer ends after its mixer (a file that still holds the two norms' weights may: nothing reads them)."""
+
+    def __init__(self, mixer: PartSpec, mixer_norm: PartSpec, mixer_post: PartSpec, feed_forward: Optional[PartSpec] = None,
+                 ff_norm: Optional[PartSpec] = None, ff_post: Optional[PartSpec] = None):
+        self.mixer_norm = self.add_child("mixer_norm", build_part("norm", mixer_norm))
+        self.mixer = self.add_child("mixer", build_part("mixer", mixer))
+        self.mixer_post = self.add_child("mixer_post", build_part("norm", mixer_post))
+        self.feed_forward = (self.add_child("feed_forward", build_part("feed_forward", feed_forward))
+                             if feed_forward is not None else None)
+        if self.feed_forward is not None and (ff_norm is None or ff_post is None):
+            raise ValueError("a sandwich block with a feed-forward needs the norms around it")
+        self.ff_norm = self.add_child("ff_norm", build_part("norm", ff_norm)) if ff_norm is not None else None
+        self.ff_post = self.add_child("ff_post", build_part("norm", ff_post)) if ff_post is not None else None
+
+    def forward(self, ctx, residual, delta, cache):
+        h = self.mixer_norm.forward(ctx, residual, delta)
+        d = self.mixer_post.leave_open(self.mixer.forward(ctx, h, cache))
+        if self.feed_forward is not None:
+            h = self.ff_norm.forward(ctx, residual, d)
+            d = self.ff_post.leave_open(self.feed_forward.forward(ctx, h))
         return residual, d
 
 

@@ -15,16 +15,20 @@ from .. import ops
 @register_part("feed_forward", "swiglu")
 class SwiGLU(FeedForward):
     """``names``: the gate, up and down tensors' names in the model file.  ``activation``: what the gate goes
-    through, ``silu`` or ``gelu_tanh``."""
+    through, ``silu`` or ``gelu_tanh``; or ``clamped``, the form with both projections limited by ``limit``
+    (``ops.glu``)."""
 
     def __init__(self, hidden_size: int, intermediate_size: int,
-                 names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), activation: str = "silu"):
+                 names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), activation: str = "silu",
+                 limit: Optional[float] = None):
         self.hidden_size = int(hidden_size)
         self.intermediate_size = int(intermediate_size)
         self.names = tuple(names)
-        if activation not in ("silu", "gelu_tanh"):
-            raise ValueError(f"a gated feed-forward's activation is silu or gelu_tanh, got {activation!r}")
-        self.activation = activation
+        if activation not in ops.GATED:
+            raise ValueError(f"a gated feed-forward's activation is one of {ops.GATED}, got {activation!r}")
+        if activation == "clamped" and limit is None:
+            raise ValueError("the clamped feed-forward needs its limit")
+        self.activation, self.limit = activation, float(limit or 0.0)
 
     def params(self):
         H, I = self.hidden_size, self.intermediate_size
@@ -35,7 +39,12 @@ class SwiGLU(FeedForward):
         ]
 
     def forward(self, ctx, x):
-        return ops.feed_forward_glu(ctx, x, self.w["gate_up_w"], self.w["down_w"], self.activation)
+        return ops.feed_forward_glu(ctx, x, self.w["gate_up_w"], self.w["down_w"], self.activation, self.limit)
+
+    def forward_to(self, ctx, x, out):
+        """The layer's result into ``out [T, hidden]`` (float32, contiguous): a plane of a stack that the next norm adds up."""
+        act = ops.glu_hidden(ctx, x, self.w["gate_up_w"], self.activation, self.limit)
+        ops.linear(act, self.w["down_w"], None, out=out)
 
 
 @register_part("feed_forward", "mlp")
@@ -97,14 +106,15 @@ class MixtureOfExperts(FeedForward):
     that is added to the scores for the choice only (the weights use the scores without it).  ``groups`` / ``keep``:
     the experts form ``groups`` equal groups of neighbours, a group's score is its largest choice score, and only
     experts of the best ``keep`` groups can be chosen.  ``weight_scale``: a constant on the weights; ``sum_eps``: added
-    to the sum that ``renorm`` divides by.  ``shared``: a feed-forward part with ``forward_to`` (``mlp``) that every token
-    goes through and whose result is added (its tensors under this part's prefix)."""
+    to the sum that ``renorm`` divides by.  ``shared``: a feed-forward part with ``forward_to`` (``mlp``, ``swiglu``) that
+    every token goes through and whose result is added (its tensors under this part's prefix).  ``router_bias``: the name
+    of a tensor ``[experts]`` added to the router's logits."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int, softmax: bool = False,
                  renorm: bool = False, scale_input: bool = True, activation: str = "silu",
                  names=("router", "e{e}.", "gate", "up", "down"), gated: bool = True, correction: Optional[str] = None,
                  groups: int = 1, keep: Optional[int] = None, weight_scale: float = 1.0, sum_eps: float = 0.0,
-                 shared: Optional[PartSpec] = None):
+                 shared: Optional[PartSpec] = None, router_bias: Optional[str] = None):
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.experts, self.top = int(experts), int(top)
         if not 1 <= self.top <= self.experts:
@@ -113,7 +123,7 @@ class MixtureOfExperts(FeedForward):
             raise ValueError(f"activation {activation!r}: one of {sorted(ops.MOE_ACTS)}")
         self.softmax, self.renorm, self.scale_input, self.activation = bool(softmax), bool(renorm), bool(scale_input), activation
         self.names = tuple(names)
-        self.gated, self.correction = bool(gated), correction
+        self.gated, self.correction, self.router_bias = bool(gated), correction, router_bias
         self.groups, self.keep = int(groups), int(groups if keep is None else keep)
         if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups:
             raise ValueError(f"{self.experts} experts in {self.groups} groups of which {self.keep} are kept: the groups must "
@@ -133,6 +143,8 @@ class MixtureOfExperts(FeedForward):
             dn.append(WeightSource(p + down, (H, I)))
         ps = [ParamSpec("router_w", (WeightSource(router, (self.experts, H)),)),
               ParamSpec("gate_up_w", tuple(gu)), ParamSpec("down_w", tuple(dn))]
+        if self.router_bias is not None:
+            ps.append(ParamSpec("router_b", (WeightSource(self.router_bias, (self.experts,), "bias"),)))
         if self.correction is not None:
             ps.append(ParamSpec("correction", (WeightSource(self.correction, (self.experts,), "bias"),)))
         return ps
@@ -142,7 +154,7 @@ class MixtureOfExperts(FeedForward):
 
     def forward(self, ctx, x):
         H, I, E = self.hidden_size, self.intermediate_size, self.experts
-        logits = ops.linear(x, self.w["router_w"], None, out_dtype=ops.torch.float32)
+        logits = ops.linear(x, self.w["router_w"], self.w.get("router_b"), out_dtype=ops.torch.float32)
         y = ops.moe_feed_forward(ctx, x, logits, self.w["gate_up_w"].view(E, (2 if self.gated else 1) * I, H),
                                  self.w["down_w"].view(E, H, I), self.top, self.softmax, self.renorm, self.scale_input,
                                  self.activation, self.gated, self.choice, extra_planes=0 if self.shared is None else 1)

@@ -7,37 +7,51 @@ that precedes it is the streams' update and its input their weighted sum."""
 
 from __future__ import annotations
 
-from .base import Norm, ParamSpec, StreamUpdate, WeightSource, register_part
+from .base import NormedDelta, Norm, ParamSpec, StreamUpdate, WeightSource, register_part
 from .. import ops
 
 
 @register_part("norm", "rmsnorm")
 class RMSNorm(Norm):
     """``x * rsqrt(mean(x^2) + eps) * weight``: the weight multiplies (no
-    ``1 + w``), no bias, no mean subtraction (fused_kernels.py:41-49)."""
+    ``1 + w``), no bias, no mean subtraction (fused_kernels.py:41-49).  ``centred``: the file stores the weight around
+    zero and ``1 + w`` multiplies (the sum is formed once, in float32, when the part is bound)."""
 
-    def __init__(self, width: int, eps: float, tensor: str = "weight", optional: bool = False):
+    def __init__(self, width: int, eps: float, tensor: str = "weight", optional: bool = False, centred: bool = False):
         self.width = int(width)
         self.eps = float(eps)
         self.tensor = tensor          # the weight's name in the model file, after the part's prefix
         self.optional = bool(optional)    # the model file may leave the weight out: the block then skips this norm
+        self.centred = bool(centred)
 
     def params(self):
-        return [ParamSpec("weight", (WeightSource(self.tensor, (self.width,), "norm"),), optional=self.optional)]
+        return [ParamSpec("weight", (WeightSource(self.tensor, (self.width,), "bias" if self.centred else "norm"),),
+                          optional=self.optional)]
+
+    def on_bound(self):
+        w = self.w.get("weight")
+        self.weight = (1.0 + w.float()).contiguous() if self.centred and w is not None else w
+
+    def leave_open(self, delta):
+        """This norm of a sublayer's result, to be carried out (and added to the stream) by the next norm."""
+        return NormedDelta(delta, self.weight, self.eps)
 
     def forward(self, ctx, residual, delta, rows=None, out_dtype=None):
         """``out_dtype``: the normed rows' dtype where it is not the compute dtype (float32 for a reader that goes on
         in 32-bit)."""
         n = residual.shape[0] if rows is None else rows.shape[0]
         out = ctx.alloc((n, self.width), out_dtype or ctx.dtype)
-        ops.add_rmsnorm(residual, delta, self.w["weight"], self.eps, out, rows)
+        if isinstance(delta, NormedDelta):
+            ops.add_normed_rmsnorm(residual, delta.delta, delta.weight, delta.eps, self.weight, self.eps, out, rows)
+        else:
+            ops.add_rmsnorm(residual, delta, self.weight, self.eps, out, rows)
         return out
 
     def forward_post(self, ctx, x, delta, alpha: float = 1.0):
         """Norm after the sum: ``x <- rmsnorm(alpha * x + delta) * weight`` in place on the float32 rows; returns
         the new rows in the compute dtype (``x`` itself in a float32 engine)."""
         copy = None if ctx.dtype == ops.torch.float32 else ctx.alloc(tuple(x.shape), ctx.dtype)
-        ops.scale_add_rmsnorm(x, alpha, delta, self.w["weight"], self.eps, copy)
+        ops.scale_add_rmsnorm(x, alpha, delta, self.weight, self.eps, copy)
         return x if copy is None else copy
 
 

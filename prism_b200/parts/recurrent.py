@@ -13,6 +13,7 @@ product, and a bonus for the current token in the read-out.
 low-rank product, and a low-rank sigmoid gate on the read-out.
 ``general_delta``: the generalized delta rule: a decay and a removal rate per
 key channel; what is removed is read along the unit key.
+``retention``: a sum of outer products under one constant decay per head, of rotated queries and keys.
 ``rglru``: a recurrence with one number of state per channel whose gates are
 block-diagonal products, behind a short convolution, beside a gelu branch.
 ``sum``: several mixers side by side on the same input, their results scaled
@@ -279,6 +280,64 @@ class GeneralDeltaMixer(Mixer):
         ops.recurrent_scan(ops.SCAN_GENERAL, r, k, v, state.state, ctx, H, 1, d, d, o, ww=ww, ex=ex)
         inner = ctx.alloc((T, A), ctx.dtype)
         ops.headnorm_gate(o, g, self.w["norm"], self.eps, self.out_scale, inner, gate_act="sigmoid")
+        return ops.linear_delta(inner, self.w["o_w"], None, f32=True)
+
+
+@register_part("mixer", "retention")
+class RetentionMixer(Mixer):
+    """Linear attention with a fixed decay per head, without softmax or denominator.  With h the input, per token and
+    head (``num_heads`` heads of ``head_dim`` key and ``v_head_dim`` value channels)::
+
+        q, k, v = W_q h, W_k h, W_v h
+        q <- rot(q);   k <- rot(k) / sqrt(head_dim)          rotated by the token's position (``position``; None: not at all)
+        S <- decay S + k v^T;   o = S^T q                    the head's entry of ``decay``
+        out = W_o [o / rms(o) * silu(W_g h)]
+
+    State per request: S ``[H, v_head_dim, head_dim]`` (stored column by column), float32, starting at zero.  All input
+    projections are one product with float32 results; rotation, state, head norm and gate are float32.  ``names``: keys
+    q, k, v, g, o."""
+
+    NAMES = dict(q="q", k="k", v="v", g="g", o="o")
+    graph_safe = True
+    float32_projection = True
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, decay: Sequence[float], eps: float,
+                 position: Optional[PartSpec] = None, names: Optional[dict] = None):
+        self.hidden_size, self.H, self.dk, self.dv = int(hidden_size), int(num_heads), int(head_dim), int(v_head_dim)
+        if min(self.H, self.dk, self.dv) < 1 or self.dk > 1024:
+            raise ConfigError("retention: heads and sizes must be positive, head_dim at most 1024")
+        self.decay = [float(d) for d in decay]
+        if len(self.decay) != self.H:
+            raise ConfigError(f"retention: {len(self.decay)} decays for {self.H} heads")
+        self.eps = float(eps)
+        self.position = self.add_child("position", build_part("position", position)) if position else None
+        self.names = dict(self.NAMES, **(names or {}))
+
+    def cache_needs(self):
+        return (CacheNeed("state", state_shape=(self.H, self.dv, self.dk)),)
+
+    def cache_need(self):
+        return self.cache_needs()[0]
+
+    def params(self):
+        W, n, A, B = self.hidden_size, self.names, self.H * self.dk, self.H * self.dv
+        return [ParamSpec("in_w", (WeightSource(n["q"], (A, W)), WeightSource(n["k"], (A, W)), WeightSource(n["v"], (B, W)),
+                                   WeightSource(n["g"], (B, W)))),
+                ParamSpec("o_w", (WeightSource(n["o"], (W, B)),))]
+
+    def on_bound(self):
+        self.decays = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(self.device)
+        self.ones = torch.ones(self.dv, dtype=torch.float32, device=self.device)
+        self.rot = self.position.rotary() if self.position is not None else None
+        if self.position is not None and (self.rot is None or self.rot.rotary_dim > self.dk):
+            raise ConfigError(f"retention takes a rotary position encoding of at most head_dim {self.dk} entries")
+
+    def forward(self, ctx, x, cache):
+        state = cache[0] if isinstance(cache, tuple) else cache
+        T, H, dk, dv, A, B = x.shape[0], self.H, self.dk, self.dv, self.H * self.dk, self.H * self.dv
+        proj = ops.linear(x, self.w["in_w"], None, out_dtype=torch.float32)          # q | k | v | g
+        inner = ctx.alloc((T, B), ctx.dtype)
+        ops.retention(ctx, proj, H, dk, dv, self.rot, self.decays, state.state, self.eps, self.ones, inner)
         return ops.linear_delta(inner, self.w["o_w"], None, f32=True)
 
 
