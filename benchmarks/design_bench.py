@@ -1,9 +1,10 @@
-"""Prefill and decode throughput of the Dolezen, the Pofazen, the Zuvulorn or the Tagelorn design at layer sizes that resemble real models
+"""Prefill and decode throughput of the Dolezen, the Pofazen, the Zuvulorn, the Tagelorn or the Limatar design at layer sizes that resemble real models
 (random weights, bf16), beside the Qwen2 architecture at equal width, depth and parameter count (Tagelorn also beside
-Zuvulorn, the closest of the other designs: attention with a sink, a delta rule with a decay per key channel, experts), and the
+Zuvulorn, the closest of the other designs: attention with a sink, a delta rule with a decay per key channel, experts; Limatar
+beside Dolezen: latent attention), and the
 design's own kernels beside the like kernels on the same problem with their fractions of the measured peaks.
 
-    python bench.py --design dolezen|pofazen|zuvulorn|tagelorn [--sizes 2k,4k] [--steps K] [--warmup W]
+    python bench.py --design dolezen|pofazen|zuvulorn|tagelorn|limatar [--sizes 2k,4k] [--steps K] [--warmup W]
     python benchmarks/design_bench.py [--design pofazen] [--sizes 2k] [--kernels-only] [--once KERNEL]
 
 One JSON line.  Timing: CUDA events after W >= 3 warm-up runs; every timed step reads all weights (more than
@@ -619,10 +620,146 @@ def tagelorn_kernel_numbers(s, pk, once=None):
     return out
 
 
+def limatar_ff(s):
+    """Inner width of a Limatar expert: eight routed experts and the shared one together weigh what Qwen2's gated
+    feed-forward does."""
+    return s["ff"] * 2 // 3 // 256 * 256 // (MOE_EXPERTS + 1) // 32 * 32
+
+
+def limatar_config(s):
+    """Layers: latent attention (sink, gate, rotation under frequency scaling), latent attention, retention, latent
+    attention, ...; dense clamped and routed feed-forwards in turn.  No loop: every layer's weights are read once a step,
+    as the other designs' are."""
+    lat = dict(heads=s["lat_heads"], dim=s["lat_dim"], rot_dim=s["rot"], vdim=s["lat_vdim"], q_rank=s["q_rank"], kv_rank=s["kv_rank"],
+               scale=(s["lat_dim"] + s["rot"]) ** -0.5,
+               rot=dict(base=10000.0, dims=s["rot"], scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0)))
+    ret = dict(heads=s["heads"], dim=s["dim"], vdim=s["vdim"], decay=[1.0 - 2.0 ** (-5 - i % 8) for i in range(s["heads"])],
+               rot=dict(base=10000.0, dims=s["dim"]))
+    F = limatar_ff(s)
+    dense = dict(kind="dense", ff=s["ff"] * 2 // 3 // 256 * 256, limit=7.0)
+    routed = dict(kind="moe", expert=dict(ff=F), shared=dict(ff=F), router=dict(experts=MOE_EXPERTS, top=MOE_TOP))
+    layers = []
+    for i in range(s["layers"]):
+        r = i % 4 == 2
+        layers.append(dict(type="retention" if r else "latent_attention", mixer=dict(ret if r else lat), mlp=dense if i % 2 == 0 else routed))
+    return dict(architecture="Limatar", vocab=s["vocab"], width=s["width"], norm=dict(eps=1e-6), layers=layers, max_positions=8192)
+
+
+def limatar_kernel_numbers(s, pk, once=None):
+    """The design's kernels alone, each beside the like kernel of the closest model on the same problem: latent attention
+    with a sink beside the same without (Dolezen's, causal here) and Qwen2's causal kernels; retention between its two projections beside
+    the delta rule's scan alone (a scalar decay per head); the clamped and the routed feed-forward beside Qwen2's dense
+    layer and gated experts without a shared one; norm, sum and norm in one launch beside the plain sum and norm."""
+    from prism_b200 import ops
+    from prism_b200.parts.base import RotaryParams
+    out = {}
+    T = 2048
+    W = s["width"]
+    shapes = (("prefill_2048", 1, 0, T), ("decode_b8", 8, T - 1, 1), ("decode_b64", 64, T - 1, 1))
+    causal = ops.KeyMask.causal()
+
+    def run(name, fn, flops, nbytes, fp32=False):
+        if once:
+            if once == name:
+                for _ in range(3):
+                    fn()
+                torch.cuda.synchronize()
+            return
+        ms = timeit(fn)
+        if fp32:
+            out[name] = dict(us=round(ms * 1e3, 1), fp32_tflops=round(flops / ms / 1e9, 2), gbs=round(nbytes / ms / 1e6, 1),
+                             frac_hbm_of_measured=round(nbytes / ms / 1e6 / pk["hbm_gbs"], 4))
+        else:
+            out[name] = _rates(ms, flops, nbytes, pk)
+
+    # latent attention: all heads over one key row per token whose first kv_rank entries are the value
+    nh, R, rd = s["lat_heads"], s["kv_rank"], s["rot"]
+    sink = torch.randn(nh, device=DEV)
+    for label, batch, cached, q_len in shapes:
+        c, kc, vc, bt, npages = paged(batch, cached, q_len, 1, R + rd, R, True)
+        q = torch.randn(batch * q_len, nh, R + rd, device=DEV, dtype=torch.bfloat16)
+        o = torch.empty(batch * q_len, nh * R, device=DEV, dtype=torch.bfloat16)
+        pairs = batch * visible_pairs(cached, q_len, causal)
+        flops = 2 * pairs * nh * (2 * R + rd)
+        nbytes = 2 * (batch * (cached + q_len) * (R + rd) + batch * q_len * nh * (2 * R + rd))
+        run(f"latent_sink_{label}", lambda: ops.masked_attention(c, q, o, kc, vc, bt, npages, causal, 0.07, sink), flops, nbytes)
+        run(f"like_latent_{label}", lambda: ops.masked_attention(c, q, o, kc, vc, bt, npages, causal, 0.07, None), flops, nbytes)
+    nq, nkv, hd = s["heads"], s["kv_heads"], s["dim"]
+    for label, batch, cached, q_len in shapes:
+        c, kc, vc, bt, npages = paged(batch, cached, q_len, nkv, hd, hd)
+        q = torch.randn(batch * q_len, nq, hd, device=DEV, dtype=torch.bfloat16)
+        o = torch.empty(batch * q_len, nq * hd, device=DEV, dtype=torch.bfloat16)
+        pairs = batch * visible_pairs(cached, q_len, causal)
+        flops, nbytes = 4 * pairs * nq * hd, 2 * (batch * (cached + q_len) * nkv * 2 * hd + 2 * batch * q_len * nq * hd)
+        if q_len == 1:
+            ns = ops.decode_splits(batch, nkv, cached + 1, None)
+            po, pml = torch.empty(batch, nq, ns, hd, device=DEV), torch.empty(batch, nq, ns, 2, device=DEV)
+            run(f"qwen2_causal_{label}", lambda: ops.attention_decode_bf16(q, o, kc, vc, bt, c.positions, c.tok_seg, npages, None,
+                                                                           hd ** -0.5, ns, po, pml, c.err), flops, nbytes)
+        else:
+            run(f"qwen2_causal_tcgen05_{label}", lambda: ops.attention_prefill_tc(q, o, kc, vc, bt, c.seg_start, c.cached_len, q_len,
+                                                                                  npages, None, hd ** -0.5, c.err), flops, nbytes)
+            run(f"qwen2_causal_mma_sync_{label}", lambda: ops.attention_prefill_bf16(q, o, kc, vc, bt, c.seg_start, c.cached_len,
+                                                                                     q_len, npages, None, hd ** -0.5, c.err), flops, nbytes)
+    # retention (rotation, recurrence, head norm, gate) beside the delta rule's scan (the recurrence alone)
+    H, dk, dv = s["heads"], s["dim"], s["vdim"]
+    freq = (10000.0 ** (-torch.arange(0, dk, 2).float() / dk)).to(DEV)
+    rot = RotaryParams(freq, dk, False)
+    decay = torch.tensor([1.0 - 2.0 ** (-5 - i % 8) for i in range(H)], device=DEV)
+    powers, ones = ops.decay_powers(decay), torch.ones(dv, device=DEV)
+    for label, batch, cached, q_len in shapes:
+        Tt = batch * q_len
+        c = types.SimpleNamespace(seg_start=(torch.arange(batch + 1, dtype=torch.int32) * q_len).to(DEV), S=batch, max_q_len=q_len,
+                                  state_slots=torch.arange(batch, dtype=torch.int32, device=DEV), decode_only=q_len == 1, scratch={},
+                                  positions=torch.arange(cached, cached + q_len, dtype=torch.int32).repeat(batch).to(DEV),
+                                  alloc=lambda shape, dtype: torch.empty(shape, dtype=dtype, device=DEV))
+        state = torch.zeros(batch + 1, H, dv, dk, device=DEV)
+        proj = torch.randn(Tt, 2 * H * (dk + dv), device=DEV) * 0.3
+        o = torch.empty(Tt, H * dv, device=DEV, dtype=torch.bfloat16)
+        run(f"retention_{label}", lambda: ops.retention(c, proj, H, dk, dv, rot, decay, powers, state, 1e-6, ones, o), 4 * Tt * H * dk * dv,
+            4 * (2 * batch * H * dk * dv + Tt * H * (2 * dk + 2 * dv)) + 2 * Tt * H * dv, fp32=True)
+        x = torch.nn.functional.normalize(torch.randn(Tt, 3 * H, dk, device=DEV), dim=-1).view(Tt, -1)
+        bg = torch.rand(Tt, 2 * H, device=DEV) * 0.5 + 0.5
+        of = torch.empty(Tt, H, dv, device=DEV)
+        run(f"like_delta_scan_{label}", lambda: ops.recurrent_scan(ops.SCAN_DELTA, x[:, :H * dk], x[:, H * dk:2 * H * dk], x[:, 2 * H * dk:],
+                                                                   state, c, H, 1, dk, dv, of, bg=bg), 6 * Tt * H * dk * dv,
+            4 * (2 * batch * H * dk * dv + Tt * H * (2 * dk + 2 * dv)), fp32=True)
+    # feed-forwards
+    E, top, F, Fz = MOE_EXPERTS, MOE_TOP, limatar_ff(s), moe_ff(s)
+    Fd = s["ff"] * 2 // 3 // 256 * 256
+    mk = lambda *sh: torch.randn(*sh, device=DEV, dtype=torch.bfloat16) / sh[-1] ** 0.5
+    gu, dn, guz, dnz, gud, dnd, gus, dns = (mk(E, 2 * F, W), mk(E, W, F), mk(E, 2 * Fz, W), mk(E, W, Fz), mk(2 * Fd, W), mk(W, Fd),
+                                            mk(2 * F, W), mk(W, F))
+    actx = types.SimpleNamespace(alloc=lambda shape, dtype: torch.empty(shape, dtype=dtype, device=DEV))
+
+    def shared_experts(xx, logits):
+        y = ops.moe_feed_forward(actx, xx, logits, gu, dn, top, True, True, False, extra_planes=1)
+        ops.linear(ops.glu_hidden(actx, xx, gus, "silu"), dns, None, out=y[top])
+    for label, Tt in (("prefill_2048", T), ("decode_b8", 8), ("decode_b64", 64)):
+        xx = torch.randn(Tt, W, device=DEV, dtype=torch.bfloat16)
+        logits = torch.randn(Tt, E, device=DEV)
+        used = min(E, Tt * top)
+        run(f"experts_with_shared_{label}", lambda: shared_experts(xx, logits), 6 * Tt * (top + 1) * F * W,
+            2 * (3 * (used + 1) * F * W + Tt * W * (2 + 2 * (top + 1))))
+        run(f"like_gated_experts_{label}", lambda: ops.moe_feed_forward(actx, xx, logits, guz, dnz, top), 6 * Tt * top * Fz * W,
+            2 * (3 * used * Fz * W + Tt * W * (1 + 2 * top)))
+        run(f"clamped_feed_forward_{label}", lambda: ops.feed_forward_glu(actx, xx, gud, dnd, "clamped", 7.0), 6 * Tt * Fd * W,
+            2 * (3 * Fd * W + 3 * Tt * W))
+        run(f"qwen2_feed_forward_{label}", lambda: ops.feed_forward_swiglu(actx, xx, gud, dnd), 6 * Tt * Fd * W,
+            2 * (3 * Fd * W + 3 * Tt * W))
+    wn = torch.ones(W, device=DEV)
+    for label, Tt in (("prefill_2048", T), ("decode_b64", 64)):
+        h, d, x1 = torch.empty(Tt, W, device=DEV, dtype=torch.bfloat16), torch.randn(Tt, W, device=DEV), torch.randn(Tt, W, device=DEV)
+        run(f"norm_sum_norm_{label}", lambda: ops.add_normed_rmsnorm(x1, d, wn, 1e-6, wn, 1e-6, h), 0, 4 * Tt * W * 3 + 2 * Tt * W, fp32=True)
+        run(f"qwen2_add_norm_{label}", lambda: ops.add_rmsnorm(x1, d, wn, 1e-6, h), 0, 4 * Tt * W * 3 + 2 * Tt * W, fp32=True)
+    return out
+
+
 DESIGNS = {"dolezen": (dolezen_config, kernel_numbers), "pofazen": (pofazen_config, pofazen_kernel_numbers),
-           "zuvulorn": (zuvulorn_config, zuvulorn_kernel_numbers), "tagelorn": (tagelorn_config, tagelorn_kernel_numbers)}
+           "zuvulorn": (zuvulorn_config, zuvulorn_kernel_numbers), "tagelorn": (tagelorn_config, tagelorn_kernel_numbers),
+           "limatar": (limatar_config, limatar_kernel_numbers)}
 # designs measured beside another design as well as beside Qwen2: the closest of the models that ran before
-BESIDE = {"tagelorn": ("zuvulorn", zuvulorn_config)}
+BESIDE = {"tagelorn": ("zuvulorn", zuvulorn_config), "limatar": ("dolezen", dolezen_config)}
 
 
 def run(sizes, steps, warmup, prompt_len=2048, batch=8, kernels_only=False, once=None, peaks=None, design="dolezen"):

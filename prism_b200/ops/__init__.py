@@ -105,6 +105,10 @@ class _Sig:
     prism_shift_mix = [_p, _i, _p, _p, _i, _i, _p, _p, _p, _i, _p, _i, _ll, _i, _p]
     prism_headnorm_gate = [_p, _p, _ll, _p, _i, _i, _f, _f, _i, _i, _i, _p, _i, _ll, _i, _p]
     prism_recurrent_scan = [_i, _p, _ll, _ll, _ll, _ll, _p, _p, _ll, _p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _i, _p, _ll, _p]
+    prism_retention_step_supported = [_i, _i]
+    prism_retention_chunks_supported = [_i, _i, _i, _i]
+    prism_retention_step = [_p, _ll, _i, _i, _i, _i, _i, _i, _i, _p, _i, _i, _f, _f, _p, _p, _p, _p, _f, _p, _i, _ll, _p]
+    prism_retention_chunks = [_p, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _p, _i, _i, _f, _f, _p, _p, _p, _p, _f, _p, _p, _ll, _p]
     prism_unit_removal = [_p, _p, _ll, _p, _i, _f, _i, _i, _i, _p, _p]
     prism_decay_from_exponent = [_p, _ll, _p, _i, _i, _i, _p]
     prism_lowrank_decay = [_p, _ll, _i, _p, _p, _i, _i, _i, _p, _ll, _i, _i, _p, _i, _i, _f, _p]
@@ -1793,16 +1797,67 @@ def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
         "recurrent_scan")
 
 
-def retention(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, rot, decay: torch.Tensor, state: torch.Tensor, eps: float,
-              ones: torch.Tensor, out: torch.Tensor):
+RETENTION_CHUNK = 64           # csrc/retention.cu: RET_CHUNK
+RETENTION_CHUNKED_FROM = int(os.environ.get("PRISM_RETENTION_CHUNKED_FROM", "16"))      # tokens of one request in a step
+
+
+def decay_powers(decay: torch.Tensor) -> torch.Tensor:
+    """``[H, RETENTION_CHUNK + 1]`` float32: powers 0, 1, .. of the float32 decays ``[H]``, formed in float64."""
+    n = torch.arange(RETENTION_CHUNK + 1, dtype=torch.float64, device=decay.device)
+    return (decay.double()[:, None] ** n[None, :]).to(torch.float32).contiguous()
+
+
+def retention(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, rot, decay: torch.Tensor, powers: torch.Tensor,
+              state: torch.Tensor, eps: float, ones: torch.Tensor, out: torch.Tensor, path: Optional[str] = None):
     """Retention between its input and its output projection, for the step's tokens: from the float32 product ``proj [T,
-    H (2 dk + 2 dv)]`` (columns q | k | v | gate; q and k are rotated in place by ``rot``, a ``RotaryParams`` or None, and k
-    multiplied by ``dk^-1/2``), ``S <- decay[h] S + k v^T; o = S^T q`` from and into ``state [slots, H, dv, dk]``, ``out = o /
-    rms(o) * silu(gate)`` in the compute dtype."""
+    H (2 dk + 2 dv)]`` (columns q | k | v | gate), q and k rotated by ``rot`` (a ``RotaryParams`` or None) and k multiplied
+    by ``dk^-1/2``, ``S <- decay[h] S + k v^T; o = S^T q`` from and into ``state [slots, H, dv, dk]``, ``out = o / rms(o) *
+    silu(gate)`` in the compute dtype.  ``powers``: ``decay_powers(decay)``; ``ones [dv]``.
+
+    ``path`` (None: chosen here): ``"step"`` one launch for a step of single tokens (it asks for the state before the kernel
+    before it has ended, so something that is not a kernel of this library - the copy of the step's descriptor - has to lie
+    between two calls on one state); ``"chunks"`` long stretches in bfloat16, on tensor cores; ``"scan"`` any
+    size, token after token (rotates q and k in place)."""
     T, A, B = proj.shape[0], H * dk, H * dv
+    _cuda(proj, decay, powers, state, out)
+    assert proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[1] == 2 * A + 2 * B
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dv, dk)
+    assert decay.dtype == powers.dtype == torch.float32 and decay.shape == (H,) and powers.shape == (H, RETENTION_CHUNK + 1)
+    assert out.shape == (T, B) and out.stride(1) == 1 and powers.is_contiguous() and decay.is_contiguous()
+    rd, freq = (rot.rotary_dim, rot.inv_freq) if rot is not None and rot.rotary_dim else (0, None)
+    il, amp = (rot.interleaved, rot.amplitude) if rd else (False, 1.0)
+    L = lib()
+    if path is None:
+        if ctx.decode_only and L.prism_retention_step_supported(dk, dv):
+            path = "step"
+        elif (ctx.max_q_len >= RETENTION_CHUNKED_FROM and out.dtype == torch.bfloat16
+              and L.prism_retention_chunks_supported(dk, dv, rd, 1 if il else 0)):
+            path = "chunks"
+        else:
+            path = "scan"
+    if path == "step":
+        assert T == ctx.S
+        _check(L.prism_retention_step(_ptr(proj), proj.stride(0), A, 2 * A, 2 * A + B, T, H, dk, dv, _ptr(freq), rd, 1 if il else 0,
+                                      float(amp), dk ** -0.5, _ptr(decay), _ptr(state), _ptr(ctx.positions), _ptr(ctx.state_slots),
+                                      float(eps), _ptr(out), _dt(out), out.stride(0), _stream()), "retention_step")
+        return
+    if path == "chunks":
+        global launch_count
+        table = None
+        if rd:
+            key = ("rotary_table", freq.data_ptr())          # one table per step for all layers
+            table = ctx.scratch.get(key)
+            if table is None:
+                table = ctx.scratch[key] = ctx.alloc((T, rd // 2, 2), torch.float32)
+                rope_table(ctx.positions, freq, table)
+        ws = ctx.alloc(((T // RETENTION_CHUNK + ctx.S) * H * dv * dk,), torch.float32)
+        _check(L.prism_retention_chunks(_ptr(proj), proj.stride(0), A, 2 * A, 2 * A + B, T, ctx.S, H, dk, dv, _ptr(table), rd,
+                                        1 if il else 0, float(amp), dk ** -0.5, _ptr(powers), _ptr(state), _ptr(ctx.seg_start),
+                                        _ptr(ctx.state_slots), float(eps), _ptr(ws), _ptr(out), out.stride(0), _stream()),
+               "retention_chunks")
+        launch_count += 2
+        return
     q, k = proj[:, :A].view(T, H, dk), proj[:, A:2 * A].view(T, H, dk)
-    rd, freq = (rot.rotary_dim, rot.inv_freq) if rot is not None else (0, None)
-    il, amp = (rot.interleaved, rot.amplitude) if rot is not None else (False, 1.0)
     if rd:
         rotate_slice(q, q, rd, freq, ctx.positions, il, amp)
     rotate_slice(k, k, rd, freq, ctx.positions, il, amp, dk ** -0.5)
