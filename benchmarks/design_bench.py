@@ -129,6 +129,21 @@ def timeit(fn, reps=10, flush=True, warmup=3):
     return total / reps       # ms
 
 
+def graphed(fn):
+    """``fn`` captured in a CUDA graph: what its launches cost on the device, without the host's time to make them."""
+    stream = torch.cuda.Stream()
+    stream.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(stream):
+        for _ in range(2):
+            fn()
+    torch.cuda.current_stream().wait_stream(stream)
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph, stream=stream):
+        fn()
+    return graph.replay
+
+
 def engine_numbers(raw, prompt_len, batch, steps, warmup):
     """Prefill tokens/s (one prompt of ``prompt_len`` tokens a step) and decode tokens/s (``batch`` requests
     behind ``prompt_len`` tokens each, CUDA graphs) through the engine's step function."""
@@ -665,7 +680,7 @@ def limatar_kernel_numbers(s, pk, once=None):
                     fn()
                 torch.cuda.synchronize()
             return
-        ms = timeit(fn)
+        ms = timeit(graphed(fn))          # as in a decode step; several launches make up some of these
         if fp32:
             out[name] = dict(us=round(ms * 1e3, 1), fp32_tflops=round(flops / ms / 1e9, 2), gbs=round(nbytes / ms / 1e6, 1),
                              frac_hbm_of_measured=round(nbytes / ms / 1e6 / pk["hbm_gbs"], 4))
@@ -731,15 +746,11 @@ def limatar_kernel_numbers(s, pk, once=None):
     gu, dn, guz, dnz, gud, dnd, gus, dns = (mk(E, 2 * F, W), mk(E, W, F), mk(E, 2 * Fz, W), mk(E, W, Fz), mk(2 * Fd, W), mk(W, Fd),
                                             mk(2 * F, W), mk(W, F))
     actx = types.SimpleNamespace(alloc=lambda shape, dtype: torch.empty(shape, dtype=dtype, device=DEV))
-
-    def shared_experts(xx, logits):
-        y = ops.moe_feed_forward(actx, xx, logits, gu, dn, top, True, True, False, extra_planes=1)
-        ops.linear(ops.glu_hidden(actx, xx, gus, "silu"), dns, None, out=y[top])
     for label, Tt in (("prefill_2048", T), ("decode_b8", 8), ("decode_b64", 64)):
         xx = torch.randn(Tt, W, device=DEV, dtype=torch.bfloat16)
         logits = torch.randn(Tt, E, device=DEV)
         used = min(E, Tt * top)
-        run(f"experts_with_shared_{label}", lambda: shared_experts(xx, logits), 6 * Tt * (top + 1) * F * W,
+        run(f"experts_with_shared_{label}", lambda: ops.moe_feed_forward(actx, xx, logits, gu, dn, top, True, True, False, shared=(gus, dns)), 6 * Tt * (top + 1) * F * W,
             2 * (3 * (used + 1) * F * W + Tt * W * (2 + 2 * (top + 1))))
         run(f"like_gated_experts_{label}", lambda: ops.moe_feed_forward(actx, xx, logits, guz, dnz, top), 6 * Tt * top * Fz * W,
             2 * (3 * used * Fz * W + Tt * W * (1 + 2 * top)))

@@ -38,6 +38,7 @@ namespace prism {
 constexpr int MA_TILE_DECODE = 64;
 constexpr int MA_TILE_PORTION = PRISM_MA_PORTION_TILE;
 constexpr int MA_THREADS = 128;
+constexpr int MA_MERGE_MAX = 1024;        // key splits the merge kernel takes
 constexpr int MA_ROWS = 64;
 
 struct MaskedAttn {
@@ -100,6 +101,32 @@ __device__ __forceinline__ void ma_load_tile(__nv_bfloat16* ks, int kstride, int
                                              int page_size, int page_shift, int num_pages, int* err, int tid) {
     const int rr = tid >> 4, cc = tid & 15;
     constexpr int PASSES = ROWS / 8;
+    // a tile that lies in one page and wholly among the visible keys: one look-up, rows at a constant distance
+    if (page_shift >= 0 && (1 << page_shift) >= ROWS && first_key >= lo && first_key + ROWS - 1 <= hi) {
+        const int page = bt[first_key >> page_shift];
+        if (page >= 0 && page < num_pages) {
+            const size_t slot0 = ((size_t)page << page_shift) + (first_key & (page_size - 1)) + rr;
+            const __nv_bfloat16* ksrc = kplane + slot0 * (size_t)k_row_stride + k_head_off + cc * 8;
+            __nv_bfloat16* kdst = ks + rr * kstride + cc * 8;
+            const size_t kstep = 8 * (size_t)k_row_stride;
+            for (int c = cc; c < kchunks; c += 16, ksrc += 128, kdst += 128) {
+                const bool v = c < kreal;
+#pragma unroll
+                for (int j = 0; j < PASSES; ++j) cp_async16(kdst + j * 8 * kstride, v ? ksrc + j * kstep : kplane, v);
+            }
+            if (WITH_V) {
+                const __nv_bfloat16* vsrc = vplane + slot0 * (size_t)v_row_stride + v_head_off + cc * 8;
+                __nv_bfloat16* vdst = vs + rr * vstride + cc * 8;
+                const size_t vstep = 8 * (size_t)v_row_stride;
+                for (int c = cc; c < vchunks; c += 16, vsrc += 128, vdst += 128) {
+                    const bool v = c < vreal;
+#pragma unroll
+                    for (int j = 0; j < PASSES; ++j) cp_async16(vdst + j * 8 * vstride, v ? vsrc + j * vstep : vplane, v);
+                }
+            }
+            return;
+        }
+    }
     long long slot[PASSES];
 #pragma unroll
     for (int j = 0; j < PASSES; ++j) {
@@ -135,7 +162,6 @@ template <int DVP, bool V_IN_K, bool SPLITK>
 __global__ void __launch_bounds__(MA_THREADS, (!SPLITK && DVP <= 128 && PRISM_MA_PORTION_TILE == 32) ? 3 : 1)
 attn_masked_kernel(const MaskedAttn a) {
     pdl_trigger();
-    pdl_wait();
     constexpr int MA_TILE = SPLITK ? MA_TILE_DECODE : MA_TILE_PORTION;
     constexpr int NT = SPLITK ? 2 : MA_TILE / 8;       // 8-key score tiles per warp and key tile
     constexpr int STAGES = SPLITK ? 3 : PRISM_MA_PORTION_STAGES;   // a decode CTA has little to compute: more tiles in flight
@@ -174,17 +200,18 @@ attn_masked_kernel(const MaskedAttn a) {
     }
     auto tile_of = [&](int v) { return v < kt ? v : tw0 + (v - kt); };
 
-    {   // the CTA's query rows
+    auto load_queries = [&]() {   // the CTA's query rows
         const int chunks = a.dkp / 8, real = a.dk / 8;
+        const __nv_bfloat16* q = pdl_fresh(a.q);
         for (int i = tid; i < QROWS * chunks; i += MA_THREADS) {
             const int r = i / chunks, c = i - r * chunks;
             const int tk = r / a.rpt, hh = r - tk * a.rpt;
             const bool valid = tk < ntok && hh < nheads && c < real;
-            const __nv_bfloat16* src = a.q;
+            const __nv_bfloat16* src = q;
             if (valid) src += (size_t)(s0 + q0 + tk) * a.q_stride + (size_t)(head0 + hh) * a.q_head_stride + c * 8;
             cp_async16(Qs + r * kstride + c * 8, src, valid);
         }
-    }
+    };
     auto load_tile = [&](int tile, int stage) {
         __nv_bfloat16* ks = KV + (size_t)stage * (k_elems + v_elems);
         ma_load_tile<!V_IN_K, MA_TILE>(ks, kstride, a.dkp / 8, a.dk / 8, ks + k_elems, vstride, DVP / 8, (a.dv + 7) / 8, a.kc,
@@ -192,9 +219,19 @@ attn_masked_kernel(const MaskedAttn a) {
                               (size_t)kvh * a.v_head_stride, bt, tile * MA_TILE, lo, hi, a.mask_keep, a.page_size, a.page_shift,
                               a.num_pages, a.err, tid);
     };
+    // The step's descriptor is there before its first kernel starts, and keys of earlier steps are in the cache: a decode
+    // CTA asks for its first tiles, as far as they hold no key of this step, before the kernels before it have ended.
+    int early = 0;
+    if (SPLITK)
+        while (early < STAGES - 1 && v0 + early < v1 && (tile_of(v0 + early) + 1) * MA_TILE <= a.cached_len[seg]) {
+            load_tile(tile_of(v0 + early), early);
+            ++early;
+        }
+    pdl_wait();
+    load_queries();
 #pragma unroll
-    for (int st = 0; st < STAGES - 1; ++st) {           // the first group also holds the query rows
-        if (v0 + st < v1) load_tile(tile_of(v0 + st), st);
+    for (int st = 0; st < STAGES - 1; ++st) {           // the first group also holds the query rows (and the early tiles)
+        if (st >= early && v0 + st < v1) load_tile(tile_of(v0 + st), st);
         cp_async_commit();
     }
 
@@ -238,6 +275,7 @@ attn_masked_kernel(const MaskedAttn a) {
             float s[NT][4];
 #pragma unroll
             for (int i = 0; i < NT; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+#pragma unroll 4
             for (int ks = 0; ks < a.dkp / 16; ++ks) {
                 uint32_t qa[4];
                 ldmatrix_x4(qa, Qs + (rowbase + lr + (mat & 1) * 8) * kstride + ks * 16 + (mat >> 1) * 8);
@@ -420,17 +458,27 @@ __global__ void attn_masked_merge_kernel(const float* __restrict__ part_o_, cons
     const int t = blockIdx.x / nh, h = blockIdx.x % nh;
     const float* po = pdl_fresh(part_o_) + (size_t)blockIdx.x * nsplit * dv;
     const float* pml = pdl_fresh(part_ml_) + (size_t)blockIdx.x * nsplit * 2;
-    float M = -INFINITY;
-    for (int s = 0; s < nsplit; ++s) M = fmaxf(M, pml[2 * s]);
+    // every warp forms the splits' factors itself, a lane a split (and every 32nd after it)
+    __shared__ float fac[MA_MERGE_MAX];
+    const int lane = threadIdx.x & 31;
     const float sk = sink != nullptr ? load_param(sink, sink_bf16, h) * 1.4426950408889634f : -INFINITY;
-    M = fmaxf(M, sk);
+    float M = sk;
+    for (int s = lane; s < nsplit; s += 32) M = fmaxf(M, pml[2 * s]);
+    M = warp_max(M);
     const float Mu = M == -INFINITY ? 0.f : M;
-    float L = ma_exp2(sk - Mu);
-    for (int s = 0; s < nsplit; ++s) L += pml[2 * s + 1] * ma_exp2(pml[2 * s] - Mu);
+    float L = 0.f;
+    for (int s = lane; s < nsplit; s += 32) {
+        const float f = ma_exp2(pml[2 * s] - Mu);
+        L += pml[2 * s + 1] * f;
+        if (threadIdx.x < 32) fac[s] = f;
+    }
+    L = warp_sum(L) + ma_exp2(sk - Mu);
+    __syncthreads();
     const float inv = L > 0.f ? 1.f / L : 0.f;
     for (int d = threadIdx.x; d < dv; d += blockDim.x) {
         float acc = 0.f;
-        for (int s = 0; s < nsplit; ++s) acc += po[(size_t)s * dv + d] * ma_exp2(pml[2 * s] - Mu);
+#pragma unroll 8
+        for (int s = 0; s < nsplit; ++s) acc += po[(size_t)s * dv + d] * fac[s];
         out[(size_t)t * out_stride + (size_t)h * dv + d] = __float2bfloat16_rn(acc * inv);
     }
 }
@@ -451,7 +499,7 @@ static int launch_masked(const MaskedAttn& a, int S, int max_q_len, cudaStream_t
     dim3 grid(SPLITK ? a.nsplit : (max_q_len + a.tok_per_cta - 1) / a.tok_per_cta, a.nkv * a.hgroups, S);
     const cudaError_t rc = launch_kernel(kern, grid, dim3(MA_THREADS), smem, stream, a);
     if (rc != cudaSuccess || !SPLITK || a.nsplit <= 1) return (int)rc;
-    return (int)launch_kernel(attn_masked_merge_kernel, dim3(S * a.nh), dim3(a.dv >= 128 ? 128 : 64), 0, stream,
+    return (int)launch_kernel(attn_masked_merge_kernel, dim3(S * a.nh), dim3(a.dv >= 256 ? 256 : (a.dv + 31) / 32 * 32), 0, stream,
                               (const float*)a.part_o, (const float*)a.part_ml, a.nsplit, a.dv, a.nh, a.sink, a.sink_bf16,
                               a.out, a.out_stride);
 }
@@ -487,7 +535,7 @@ PRISM_EXPORT int prism_attention_masked_bf16(const void* q, long long q_stride, 
         (mask_kind != PRISM_MASK_CAUSAL && mask_size < 1) || mask_keep < 0 || (mask_keep > 0 && mask_kind != PRISM_MASK_WINDOW))
         return (int)cudaErrorInvalidValue;
     const int rep = nh / nkv;
-    if (few_rows && (max_q_len != 1 || nsplit < 1 || nsplit > 65535 ||
+    if (few_rows && (max_q_len != 1 || nsplit < 1 || nsplit > MA_MERGE_MAX ||
                      (nsplit > 1 && (part_o == nullptr || part_ml == nullptr))))
         return (int)cudaErrorInvalidValue;
     MaskedAttn a;
@@ -521,6 +569,7 @@ PRISM_EXPORT int prism_attention_masked_bf16(const void* q, long long q_stride, 
     if (dv <= 32) PRISM_MA_LAUNCH(32);
     if (dv <= 64) PRISM_MA_LAUNCH(64);
     if (dv <= 128) PRISM_MA_LAUNCH(128);
+    if (dv <= 192) PRISM_MA_LAUNCH(192);
     PRISM_MA_LAUNCH(256);
 #undef PRISM_MA_LAUNCH
 }

@@ -177,14 +177,17 @@ gemm_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                     for (int n = 0; n < NTOK; ++n) acc[w][n] = 0.f;
             }
             bool finish = true;
-            if ((EPI == EPI_BF16 || EPI == EPI_F32) && gridDim.y > 1) {
+            if (EPI != EPI_PARTIAL && (EPI != EPI_SWIGLU || NTOK == 16) && gridDim.y > 1) {
                 // K was split over gridDim.y CTAs: every CTA leaves its partial sums in the workspace and
                 // the one that arrives last at the tile's counter adds them up, in split order, and
-                // finishes the tile.  Nobody waits for anybody.
+                // finishes the tile.  Nobody waits for anybody.  (Paired, for 16 tokens: the up
+                // rows' sums follow the gate rows'.)
                 if (m < N)
 #pragma unroll
-                    for (int n = 0; n < NTOK; ++n)
-                        if (n < M) ws[((size_t)blockIdx.y * M + n) * N + m] = acc[0][n];
+                    for (int w = 0; w < W_TILES; ++w)
+#pragma unroll
+                        for (int n = 0; n < NTOK; ++n)
+                            if (n < M) ws[(((size_t)blockIdx.y * W_TILES + w) * M + n) * N + m] = acc[w][n];
                 __threadfence();
                 asm volatile("bar.sync 1, 128;" ::: "memory");            // the four epilogue warps
                 if (threadIdx.x == 64) {
@@ -196,12 +199,21 @@ gemm_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                 finish = is_last != 0;
                 if (finish && m < N) {
                     __threadfence();
+                    // one split after another, but a split's values for all tokens in one round of loads
 #pragma unroll
-                    for (int n = 0; n < NTOK; ++n) {
-                        if (n >= M) continue;
-                        float v = 0.f;
-                        for (int sp = 0; sp < (int)gridDim.y; ++sp) v += __ldcg(&ws[((size_t)sp * M + n) * N + m]);
-                        acc[0][n] = v;
+                    for (int w = 0; w < W_TILES; ++w)
+#pragma unroll
+                        for (int n = 0; n < NTOK; ++n) acc[w][n] = 0.f;
+                    for (int sp = 0; sp < (int)gridDim.y; ++sp) {
+                        const float* part = ws + (size_t)sp * W_TILES * M * N + m;
+#pragma unroll
+                        for (int w = 0; w < W_TILES; ++w) {
+                            float v[NTOK];
+#pragma unroll
+                            for (int n = 0; n < NTOK; ++n) v[n] = n < M ? __ldcg(part + ((size_t)w * M + n) * N) : 0.f;
+#pragma unroll
+                            for (int n = 0; n < NTOK; ++n) acc[w][n] += v[n];
+                        }
                     }
                 }
             }
@@ -277,7 +289,8 @@ PRISM_EXPORT int prism_gemm_tcgen05_supported(int M, int N, int K) {
 // 5: as 2 in the clamped form with `glu_limit` (common.cuh: clamped_glu).
 // ksplit > 1 with epi 0 or 1 needs a workspace `ws` of ksplit * M * N floats and `counters`, one int per
 // 128-row tile of N, zero before the first launch (the kernel leaves them zero); the last CTA of each
-// tile adds the partial sums in split order, so the result does not depend on timing.  Not with epi 2.
+// tile adds the partial sums in split order, so the result does not depend on timing.  The paired epilogues take it up to
+// 16 tokens and need twice the workspace.
 // group_rows > 0 (a multiple of 128): x holds one [M, K] block of rows per group of group_rows weight rows,
 // group_tokens rows apart, and every group of output features reads its own block.
 PRISM_EXPORT int prism_gemm_tcgen05(const void* W, int ldw, const void* x, int ldx, const void* bias, int bias_dtype,
@@ -290,12 +303,13 @@ PRISM_EXPORT int prism_gemm_tcgen05(const void* W, int ldw, const void* x, int l
     if (epi == 4 || epi == 5) epi = EPI_SWIGLU;
     if (group_rows < 0 || group_rows % 128 || (group_rows > 0 && (group_tokens < M || epi == EPI_SWIGLU)))
         return (int)cudaErrorInvalidValue;
-    if (!prism_gemm_tcgen05_supported(M, N, K) || ldw % 8 || ldx % 8 || ksplit < 1 || (ksplit > 1 && epi == EPI_SWIGLU) ||
+    if (!prism_gemm_tcgen05_supported(M, N, K) || ldw % 8 || ldx % 8 || ksplit < 1 ||
         (ksplit > 1 && epi != EPI_PARTIAL && (ws == nullptr || counters == nullptr)) ||
         ((uintptr_t)W & 15) || ((uintptr_t)x & 15))
         return (int)cudaErrorInvalidValue;
     const int bb = bias_dtype == PRISM_DTYPE_BF16;
     const int ntok = M <= 16 ? 16 : (M <= 32 ? 32 : 64);
+    if (epi == EPI_SWIGLU && ksplit > 1 && ntok != 16) return (int)cudaErrorInvalidValue;
     const long long w_rows = epi == EPI_SWIGLU ? 2LL * N : N;
     const int pair = epi == EPI_SWIGLU ? N : 0;
 #define ARGS W, ldw, w_rows, x, ldx, bias, bb, y, ldy, M, N, K, ksplit, pair, ws, counters, err, group_rows, group_tokens, glu_act, glu_limit, stream

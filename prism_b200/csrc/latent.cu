@@ -17,6 +17,40 @@
 
 namespace prism {
 
+// x[c] for c = threadIdx.x, + blockDim.x, ... < n in registers (KV_REGS of them; the rest are read again), and the sum of their squares
+constexpr int KV_REGS = 8;
+__device__ __forceinline__ float load_row(const float* __restrict__ x, int n, float (&v)[KV_REGS]) {
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < KV_REGS; ++j) {
+        const int c = threadIdx.x + j * blockDim.x;
+        v[j] = c < n ? x[c] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < KV_REGS; ++j) ss += v[j] * v[j];
+    for (int c = threadIdx.x + KV_REGS * blockDim.x; c < n; c += blockDim.x) ss += x[c] * x[c];
+    return ss;
+}
+__device__ __forceinline__ void load_weights(const void* __restrict__ w, int bf16, int n, float (&v)[KV_REGS]) {
+#pragma unroll
+    for (int j = 0; j < KV_REGS; ++j) {
+        const int c = threadIdx.x + j * blockDim.x;
+        v[j] = c < n ? load_param(w, bf16, c) : 0.f;
+    }
+}
+template <typename T>
+__device__ __forceinline__ void store_row(const float* __restrict__ x, int n, const float (&v)[KV_REGS], const float (&wv)[KV_REGS],
+                                          float inv, const void* __restrict__ w, int bf16, T* dst) {
+#pragma unroll
+    for (int j = 0; j < KV_REGS; ++j) {
+        const int c = threadIdx.x + j * blockDim.x;
+        if (c < n) dst[c] = from_float<T>(v[j] * inv * wv[j]);
+    }
+    for (int c = threadIdx.x + KV_REGS * blockDim.x; c < n; c += blockDim.x) dst[c] = from_float<T>(x[c] * inv * load_param(w, bf16, c));
+}
+
+// grid (tokens, 1 or 2): y = 0 the cache row, y = 1 the query latent of the same token.  The norms' weights and the token's
+// slot are read before the wait (the weights are constants, the descriptor precedes the step's first kernel).
 template <typename T>
 __global__ void latent_kv_store_kernel(const float* __restrict__ x_in, long long x_stride,
                                        const void* __restrict__ weight, int weight_bf16, float eps, int R, int r,
@@ -27,45 +61,44 @@ __global__ void latent_kv_store_kernel(const float* __restrict__ x_in, long long
                                        const float* __restrict__ xq_in, int q_rank, const void* __restrict__ q_weight,
                                        int q_weight_bf16, T* __restrict__ q_out, long long q_out_stride, int pairs, float amp) {
     pdl_trigger();
-    pdl_wait();
     __shared__ float scratch[33];
-    if (q_out != nullptr) {         // the query latent of the same token (same row stride), normed, in the same launch
+    float v[KV_REGS], wv[KV_REGS];
+    if (blockIdx.y == 1) {          // the query latent of the same token (same row stride), normed, in the same launch
+        load_weights(q_weight, q_weight_bf16, q_rank, wv);
+        pdl_wait();
         const float* xq = pdl_fresh(xq_in) + (size_t)blockIdx.x * x_stride;
-        float sq = 0.f;
-        for (int c = threadIdx.x; c < q_rank; c += blockDim.x) sq += xq[c] * xq[c];
-        sq = block_sum(sq, scratch);
-        const float invq = 1.f / sqrtf(sq / (float)q_rank + eps);
-        T* o = q_out + (size_t)blockIdx.x * q_out_stride;
-        for (int c = threadIdx.x; c < q_rank; c += blockDim.x)
-            o[c] = from_float<T>(xq[c] * invq * load_param(q_weight, q_weight_bf16, c));
+        const float sq = block_sum(load_row(xq, q_rank, v), scratch);
+        store_row(xq, q_rank, v, wv, 1.f / sqrtf(sq / (float)q_rank + eps), q_weight, q_weight_bf16,
+                  q_out + (size_t)blockIdx.x * q_out_stride);
+        return;
     }
-    const float* x = pdl_fresh(x_in) + (size_t)blockIdx.x * x_stride;
     const int pos = positions[blockIdx.x];
-    float ss = 0.f;
-    for (int c = threadIdx.x; c < R; c += blockDim.x) ss += x[c] * x[c];
-    ss = block_sum(ss, scratch);
+    int page = -1;
+    if (pos >= 0 && pos < max_pos) page = block_table[(size_t)tok_seg[blockIdx.x] * bt_width + pos / page_size];
+    load_weights(weight, weight_bf16, R, wv);
+    const int half = rot_dims / 2;
+    float sn = 0.f, cs = 0.f;
+    if ((int)threadIdx.x < half) sincosf((float)pos * inv_freq[threadIdx.x], &sn, &cs);
+    pdl_wait();
+    const float* x = pdl_fresh(x_in) + (size_t)blockIdx.x * x_stride;
+    const float ss = block_sum(load_row(x, R, v), scratch);
     if (pos < 0 || pos >= max_pos) {
         if (threadIdx.x == 0) report_error(err, PRISM_ERR_POSITION_RANGE);
         return;
     }
-    const int page = block_table[(size_t)tok_seg[blockIdx.x] * bt_width + pos / page_size];
     if (page < 0 || page >= num_pages) {
         if (threadIdx.x == 0) report_error(err, PRISM_ERR_PAGE_RANGE);
         return;
     }
     T* dst = cache + ((size_t)page * page_size + pos % page_size) * (size_t)(R + r);
-    const float inv = 1.f / sqrtf(ss / (float)R + eps);
-    for (int c = threadIdx.x; c < R; c += blockDim.x) dst[c] = from_float<T>(x[c] * inv * load_param(weight, weight_bf16, c));
-    const int half = rot_dims / 2;
+    store_row(x, R, v, wv, 1.f / sqrtf(ss / (float)R + eps), weight, weight_bf16, dst);
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
-        float sn, cs;
-        sincosf((float)pos * inv_freq[i], &sn, &cs);
-        sn *= amp;
-        cs *= amp;
+        if (i != (int)threadIdx.x) sincosf((float)pos * inv_freq[i], &sn, &cs);
+        const float s = sn * amp, c = cs * amp;
         const int a = pairs ? 2 * i : i, b = pairs ? 2 * i + 1 : i + half;
-        const float u = x[R + a], v = x[R + b];
-        dst[R + a] = from_float<T>(u * cs - v * sn);
-        dst[R + b] = from_float<T>(v * cs + u * sn);
+        const float u = x[R + a], w = x[R + b];
+        dst[R + a] = from_float<T>(u * c - w * s);
+        dst[R + b] = from_float<T>(w * c + u * s);
     }
     for (int c = rot_dims + threadIdx.x; c < r; c += blockDim.x) dst[R + c] = from_float<T>(x[R + c]);
 }
@@ -144,13 +177,14 @@ PRISM_EXPORT int prism_latent_kv_store(const float* x, long long x_stride, const
     if (R <= 0 || r < 0 || rot_dims < 0 || rot_dims > r || rot_dims % 2) return (int)cudaErrorInvalidValue;
     if (q_out != nullptr && (xq == nullptr || q_weight == nullptr || q_rank <= 0)) return (int)cudaErrorInvalidValue;
     const int wb = weight_dtype == PRISM_DTYPE_BF16, qwb = q_weight_dtype == PRISM_DTYPE_BF16;
-    const int threads = R >= 1024 ? 256 : 128;
+    const int threads = R >= 1024 || q_rank >= 1024 ? 256 : 128;
+    const dim3 grid(T, q_out != nullptr ? 2 : 1);
     if (dtype == PRISM_DTYPE_BF16)
-        return (int)prism::launch_kernel(prism::latent_kv_store_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, x,
+        return (int)prism::launch_kernel(prism::latent_kv_store_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, x,
                                          x_stride, weight, wb, eps, R, r, rot_dims, inv_freq, (__nv_bfloat16*)cache,
                                          block_table, bt_width, positions, tok_seg, page_size, num_pages, max_pos, err, xq,
                                          q_rank, q_weight, qwb, (__nv_bfloat16*)q_out, q_out_stride, pairs, amp);
-    return (int)prism::launch_kernel(prism::latent_kv_store_kernel<float>, dim3(T), dim3(threads), 0, stream, x, x_stride,
+    return (int)prism::launch_kernel(prism::latent_kv_store_kernel<float>, grid, dim3(threads), 0, stream, x, x_stride,
                                      weight, wb, eps, R, r, rot_dims, inv_freq, (float*)cache, block_table, bt_width,
                                      positions, tok_seg, page_size, num_pages, max_pos, err, xq, q_rank, q_weight, qwb,
                                      (float*)q_out, q_out_stride, pairs, amp);

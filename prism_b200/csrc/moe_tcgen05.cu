@@ -15,6 +15,12 @@
 //   single: y[dst[p], n] = (down_e h_p)[n] (* weight[p])         float32; W is [E, N, K]
 //           without dst: hidden[p, n] = act(up_e a_p)[n]         bf16: the hidden layer of experts without a gate
 //
+// An expert that every token goes through (a shared one, with an inner width of its own) can ride in the same launches:
+// the first token tiles of the grid are then its own, with matrices, rows and result of theirs (MoeShared).  K may be
+// split over grid.z: every CTA leaves its partial sums in a workspace and the one that arrives last at the tile's
+// counter adds them up, in split order, and finishes the tile (as in gemm_tcgen05.cu; for steps of few tokens, whose
+// experts have few tiles).
+//
 // A decode step (a few rows per expert) reads every chosen expert's weights once; a prompt's tiles of one expert
 // re-read them from L2.  Every mbarrier wait is bounded, as in gemm_tcgen05.cu.
 #include "tcgen05.cuh"
@@ -44,12 +50,21 @@ template <int NTOK, bool DUAL> struct MoeCfg {
     static constexpr size_t SMEM = (size_t)STAGES * STAGE_BYTES + 1024 + 256;
 };
 
+// The shared expert's part of a launch: tiles token tiles in front of the others' (0: none) over rows 0 .. rows - 1 of its
+// input; dual: hidden [rows, N] bf16 at y; single: y [rows, N] float32.
+struct MoeShared {
+    int tiles, rows, N, K;
+    void* y;
+    long long ldy;
+};
+
 template <int NTOK, bool DUAL>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                 const int* __restrict__ offs_in, const int* __restrict__ counts_in, const int* __restrict__ row_dst_in,
                 const float* __restrict__ row_w_in, int E, int N, int K, int act, void* __restrict__ y, long long ldy,
-                int* err) {
+                int* err, const __grid_constant__ CUtensorMap map_sw, const __grid_constant__ CUtensorMap map_sx,
+                const MoeShared sh, float* __restrict__ ws, int* __restrict__ counters) {
     using C = MoeCfg<NTOK, DUAL>;
     constexpr int W_TILES = C::W_TILES;
     constexpr int STAGES = C::STAGES;
@@ -61,9 +76,14 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_bar + 1);
     __shared__ int abort_flag;
     __shared__ int tile_e, tile_valid;
+    __shared__ int is_last;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int row0 = blockIdx.y * NTOK;                    // first padded row of this token tile
+    const bool shared_tile = (int)blockIdx.y < sh.tiles;
+    const int row0 = ((int)blockIdx.y - (shared_tile ? 0 : sh.tiles)) * NTOK;      // first (padded) row of this token tile
+    if (shared_tile) { N = sh.N; K = sh.K; y = sh.y; ldy = sh.ldy; }
+    const int m_in = blockIdx.x * MOE_TILE_M;              // first output feature of this tile, inside the expert
+    if (m_in >= N) return;
     pdl_trigger();
     if (threadIdx.x == 0) {
         abort_flag = 0;
@@ -74,7 +94,10 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
         const int* offs = pdl_fresh(offs_in);
         const int* counts = pdl_fresh(counts_in);
         int found = -1, valid = 0;
-        for (int e = 0; e < E; ++e) {
+        if (shared_tile) {
+            found = 0;
+            valid = min(NTOK, sh.rows - row0);
+        } else for (int e = 0; e < E; ++e) {
             const int a = offs[e], b = offs[e + 1];
             if (row0 >= a && row0 < b) {
                 found = e;
@@ -88,9 +111,11 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
     __syncthreads();
     const int e = tile_e, valid = tile_valid;
     if (e < 0 || valid <= 0) return;                       // the whole CTA: nothing allocated yet
-    const int m_in = blockIdx.x * MOE_TILE_M;              // first output feature of this tile, inside the expert
     const int w_row0 = e * (DUAL ? 2 : 1) * N + m_in;
-    const int nkb = (K + TILE_K - 1) / TILE_K;
+    const CUtensorMap* mw = shared_tile ? &map_sw : &map_w;
+    const CUtensorMap* mx = shared_tile ? &map_sx : &map_x;
+    const int total_kb = (K + TILE_K - 1) / TILE_K, per_split = (total_kb + (int)gridDim.z - 1) / (int)gridDim.z;
+    const int kb0 = min(total_kb, (int)blockIdx.z * per_split), nkb = min(total_kb, kb0 + per_split) - kb0;
 
     if (warp == 1) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_addr(tmem_slot)), "r"(C::TMEM_COLS));
@@ -111,11 +136,11 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                 if (i >= STAGES && !mbar_wait(&empty_bar[s], ((i / STAGES) - 1) & 1, abortp)) break;
                 unsigned char* st = tiles + (size_t)s * C::STAGE_BYTES;
                 mbar_expect_tx(&full_bar[s], C::STAGE_BYTES);
-                const int kc = i * TILE_K;
+                const int kc = (kb0 + i) * TILE_K;
 #pragma unroll
                 for (int w = 0; w < W_TILES; ++w)
-                    tma_load_2d(st + w * MOE_TILE_M * TILE_K * 2, &map_w, &full_bar[s], kc, w_row0 + w * N);
-                tma_load_2d(st + W_TILES * MOE_TILE_M * TILE_K * 2, &map_x, &full_bar[s], kc, row0);
+                    tma_load_2d(st + w * MOE_TILE_M * TILE_K * 2, mw, &full_bar[s], kc, w_row0 + w * N);
+                tma_load_2d(st + W_TILES * MOE_TILE_M * TILE_K * 2, mx, &full_bar[s], kc, row0);
                 issued = i + 1;
             }
             if (*abortp) {
@@ -144,7 +169,7 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                 }
                 umma_commit(&empty_bar[s]);
             }
-            umma_commit(acc_bar);
+            if (nkb > 0) umma_commit(acc_bar);
         }
     } else {
         const int q = warp & 3;
@@ -152,20 +177,63 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
         pdl_wait();
         const int* row_dst = pdl_fresh(row_dst_in);
         const float* row_w = pdl_fresh(row_w_in);
-        mbar_wait(acc_bar, 0, abortp);
+        if (nkb > 0) mbar_wait(acc_bar, 0, abortp);
         asm volatile("bar.sync 1, 128;" ::: "memory");
         const bool go = *abortp == 0;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         if (go) {
             float acc[W_TILES][NTOK];
 #pragma unroll
-            for (int w = 0; w < W_TILES; ++w) tmem_load<NTOK>(tmem_base + ((uint32_t)(q * 32) << 16) + w * NTOK, acc[w]);
-            if (m < N) {
+            for (int w = 0; w < W_TILES; ++w) {
+                if (nkb > 0) tmem_load<NTOK>(tmem_base + ((uint32_t)(q * 32) << 16) + w * NTOK, acc[w]);
+                else
+#pragma unroll
+                    for (int n = 0; n < NTOK; ++n) acc[w][n] = 0.f;
+            }
+            bool finish = true;
+            if (gridDim.z > 1) {
+                const size_t plane = (size_t)NTOK * MOE_TILE_M;                  // one tile's sums of one matrix
+                float* mine = ws + ((size_t)blockIdx.y * gridDim.x + blockIdx.x) * gridDim.z * W_TILES * plane + q * 32 + lane;
+#pragma unroll
+                for (int w = 0; w < W_TILES; ++w)
+#pragma unroll
+                    for (int n = 0; n < NTOK; ++n)
+                        if (n < valid) mine[((size_t)blockIdx.z * W_TILES + w) * plane + n * MOE_TILE_M] = acc[w][n];
+                __threadfence();
+                asm volatile("bar.sync 1, 128;" ::: "memory");
+                if (threadIdx.x == 64) {
+                    int* c = counters + blockIdx.y * gridDim.x + blockIdx.x;
+                    is_last = atomicAdd(c, 1) == (int)gridDim.z - 1;
+                    if (is_last) *c = 0;                                         // ready for the next launch
+                }
+                asm volatile("bar.sync 1, 128;" ::: "memory");
+                finish = is_last != 0;
+                if (finish) {
+                    __threadfence();
+#pragma unroll
+                    for (int w = 0; w < W_TILES; ++w)
+#pragma unroll
+                        for (int n = 0; n < NTOK; ++n) acc[w][n] = 0.f;
+                    for (int sp = 0; sp < (int)gridDim.z; ++sp)
+#pragma unroll
+                        for (int w = 0; w < W_TILES; ++w) {
+                            const float* part = mine + ((size_t)sp * W_TILES + w) * plane;
+                            float v[NTOK];
+#pragma unroll
+                            for (int n = 0; n < NTOK; ++n) v[n] = n < valid ? __ldcg(part + n * MOE_TILE_M) : 0.f;
+#pragma unroll
+                            for (int n = 0; n < NTOK; ++n) acc[w][n] += v[n];
+                        }
+                }
+            }
+            if (finish && m < N) {
 #pragma unroll
                 for (int n = 0; n < NTOK; ++n) {
                     if (n >= valid) continue;
                     const int p = row0 + n;
-                    if (DUAL) {
+                    if (shared_tile && !DUAL) {
+                        reinterpret_cast<float*>(y)[(size_t)p * ldy + m] = acc[0][n];
+                    } else if (DUAL) {
                         reinterpret_cast<__nv_bfloat16*>(y)[(size_t)p * ldy + m] =
                             __float2bfloat16_rn(moe_tc_act(acc[0][n], act) * acc[W_TILES - 1][n]);
                     } else if (row_dst == nullptr) {          // an expert without a gate: its hidden layer, act(up a_p)
@@ -190,18 +258,27 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
 template <int NTOK, bool DUAL>
 int moe_launch(const void* x, long long ldx, long long x_rows, const void* W, const int* offs, const int* counts,
                const int* row_dst, const float* row_w, int token_tiles, int E, int N, int K, int act, void* y,
-               long long ldy, int* err, cudaStream_t stream) {
+               long long ldy, int* err, const void* sw, const void* sx, long long ldsx, const MoeShared& sh, int ksplit, float* ws,
+               int* counters, cudaStream_t stream) {
     using C = MoeCfg<NTOK, DUAL>;
     CUtensorMap mw, mx;
     int rc = make_map(&mw, W, (long long)E * (DUAL ? 2 : 1) * N, K, K, MOE_TILE_M);
     if (rc) return rc;
     rc = make_map(&mx, x, x_rows, K, ldx, NTOK);
     if (rc) return rc;
+    CUtensorMap msw = mw, msx = mx;
+    if (sh.tiles > 0) {
+        rc = make_map(&msw, sw, (long long)(DUAL ? 2 : 1) * sh.N, sh.K, sh.K, MOE_TILE_M);
+        if (rc) return rc;
+        rc = make_map(&msx, sx, sh.rows, sh.K, ldsx, NTOK);
+        if (rc) return rc;
+    }
     auto kern = moe_swap_kernel<NTOK, DUAL>;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM);
-    dim3 grid((N + MOE_TILE_M - 1) / MOE_TILE_M, token_tiles);
+    const int widest = sh.tiles > 0 && sh.N > N ? sh.N : N;
+    dim3 grid((widest + MOE_TILE_M - 1) / MOE_TILE_M, token_tiles + sh.tiles, ksplit);
     return (int)launch_kernel(kern, grid, dim3(MOE_THREADS), C::SMEM, stream, mw, mx, offs, counts, row_dst, row_w, E, N, K, act,
-                              y, ldy, err);
+                              y, ldy, err, msw, msx, sh, ws, counters);
 }
 
 // One block per (token, choice): its row of x, times its weight (scale_in), rounded to bf16, at its padded place;
@@ -250,16 +327,30 @@ PRISM_EXPORT int prism_moe_gather(const void* x, long long ldx, const int* offs,
 // dual 1: out [x_rows, N] bf16 (row stride ldo), out[p] = act(gate a_p) * (up a_p).
 // dual 0: out float32, out[row_dst[p]] = w a_p (times row_w[p] if row_w is given); row_dst null: out [x_rows, N] bf16,
 // out[p] = act(w a_p).
+// shared_rows > 0: an expert that all of them go through rides along: sw [(2) sN, sK] bf16 contiguous, sx [shared_rows, sK]
+// (row stride ldsx), its result at sy (dual: bf16, else float32; row stride ldsy).
+// ksplit > 1: ws of grid tiles * ksplit * (dual 2) * ntok * 128 floats and counters, one int per tile, zero before the
+// first launch; tiles: ceil(max(N, sN) / 128) * (token_tiles + ceil(shared_rows / ntok)).
 PRISM_EXPORT int prism_moe_gemm_tcgen05(const void* a, long long lda, const void* w, const int* offs, const int* counts,
                                         const int* row_dst, const float* row_w, int ntok, int token_tiles, int E, int N,
-                                        int K, int dual, int act, void* out, long long ldo, int* err, cudaStream_t stream) {
+                                        int K, int dual, int act, void* out, long long ldo, int* err, const void* sw,
+                                        const void* sx, long long ldsx, int shared_rows, int sN, int sK, void* sy, long long ldsy,
+                                        int ksplit, float* ws, int* counters, cudaStream_t stream) {
     using namespace prism::tc;
     if (token_tiles <= 0 || N <= 0) return 0;
     if (E < 1 || K < 8 || K % 8 || lda % 8 || ((uintptr_t)a & 15) || ((uintptr_t)w & 15) || token_tiles > 65535 ||
         (ntok != 16 && ntok != 32 && ntok != 64))
         return (int)cudaErrorInvalidValue;
+    if (ksplit < 1 || ksplit > 64 || (ksplit > 1 && (ws == nullptr || counters == nullptr))) return (int)cudaErrorInvalidValue;
+    if (shared_rows > 0 && (sw == nullptr || sx == nullptr || sy == nullptr || sN < 1 || sK < 8 || sK % 8 || ldsx % 8 ||
+                            ((uintptr_t)sw & 15) || ((uintptr_t)sx & 15) || (!dual && row_dst == nullptr)))
+        return (int)cudaErrorInvalidValue;
+    MoeShared sh;
+    sh.tiles = shared_rows > 0 ? (shared_rows + ntok - 1) / ntok : 0;
+    sh.rows = shared_rows; sh.N = sN; sh.K = sK; sh.y = sy; sh.ldy = ldsy;
+    if (token_tiles + sh.tiles > 65535) return (int)cudaErrorInvalidValue;
     const long long x_rows = (long long)token_tiles * ntok;
-#define ARGS a, lda, x_rows, w, offs, counts, row_dst, row_w, token_tiles, E, N, K, act, out, ldo, err, stream
+#define ARGS a, lda, x_rows, w, offs, counts, row_dst, row_w, token_tiles, E, N, K, act, out, ldo, err, sw, sx, ldsx, sh, ksplit, ws, counters, stream
     if (dual) return ntok == 16 ? moe_launch<16, true>(ARGS) : ntok == 32 ? moe_launch<32, true>(ARGS) : moe_launch<64, true>(ARGS);
     return ntok == 16 ? moe_launch<16, false>(ARGS) : ntok == 32 ? moe_launch<32, false>(ARGS) : moe_launch<64, false>(ARGS);
 #undef ARGS

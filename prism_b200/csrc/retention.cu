@@ -159,23 +159,54 @@ __device__ __forceinline__ void ret_split4(float4 v, __nv_bfloat16* hi, __nv_bfl
     *reinterpret_cast<uint2*>(lo) = make_uint2(pack_bf16(v.x - f0.x, v.y - f0.y), pack_bf16(v.z - f1.x, v.w - f1.y));
 }
 
-// quad at column d (a multiple of 4) of token t's q or k, rotated
-__device__ __forceinline__ float4 ret_rotated(const RetChunks& a, const float* __restrict__ x, int t, int d) {
-    float4 u = *reinterpret_cast<const float4*>(x + d);
-    if (d >= a.rot) return u;
-    const float2* tb = a.table + (size_t)t * (a.rot >> 1);
-    if (a.pairs) {
-        const float4 c = *reinterpret_cast<const float4*>(tb + (d >> 1));        // cos, sin of two pairs
-        return make_float4((u.x * c.x - u.y * c.y) * a.amp, (u.y * c.x + u.x * c.y) * a.amp, (u.z * c.z - u.w * c.w) * a.amp,
-                           (u.w * c.z + u.z * c.w) * a.amp);
-    }
+// What a rotated quad is made of: the quad at column d (a multiple of 4) of token t's q or k, its partner, and the cosines
+// and sines.  Loads only, all of them in any case (from a legal place where they are not needed), so that a batch of
+// quads has all its loads on their way together; the arithmetic follows in ret_turn.
+struct RetQuad {
+    float4 u, w, c0, c1;
+};
+__device__ __forceinline__ RetQuad ret_quad(const RetChunks& a, const float* __restrict__ x, int t, int d) {
     const int half = a.rot >> 1;
-    const bool second = d >= half;
-    const float4 w = *reinterpret_cast<const float4*>(x + (second ? d - half : d + half));
-    const float4 c0 = *reinterpret_cast<const float4*>(tb + (second ? d - half : d)), c1 = *reinterpret_cast<const float4*>(tb + (second ? d - half : d) + 2);
-    const float sg = second ? a.amp : -a.amp;
-    return make_float4(u.x * (c0.x * a.amp) + w.x * (c0.y * sg), u.y * (c0.z * a.amp) + w.y * (c0.w * sg),
-                       u.z * (c1.x * a.amp) + w.z * (c1.y * sg), u.w * (c1.z * a.amp) + w.w * (c1.w * sg));
+    const bool turns = d < a.rot, second = d >= half;
+    const int e = !turns || a.pairs ? d : (second ? d - half : d + half);
+    const int ti = !turns ? 0 : (a.pairs ? d >> 1 : (second ? d - half : d));
+    const float* tb = a.rot > 0 ? reinterpret_cast<const float*>(a.table + (size_t)t * half + ti) : x;
+    RetQuad q;
+    q.u = *reinterpret_cast<const float4*>(x + d);
+    q.w = *reinterpret_cast<const float4*>(x + e);
+    q.c0 = *reinterpret_cast<const float4*>(tb);
+    q.c1 = *reinterpret_cast<const float4*>(tb + (a.pairs || a.rot == 0 ? 0 : 4));
+    return q;
+}
+// the quad, rotated and times f
+__device__ __forceinline__ float4 ret_turn(const RetChunks& a, const RetQuad& q, int d, float f) {
+    const float4 u = q.u, w = q.w, c0 = q.c0, c1 = q.c1;
+    const float g = d < a.rot ? a.amp * f : f;
+    float4 r = u;
+    if (d < a.rot) {
+        if (a.pairs) r = make_float4(u.x * c0.x - u.y * c0.y, u.y * c0.x + u.x * c0.y, u.z * c0.z - u.w * c0.w, u.w * c0.z + u.z * c0.w);
+        else {
+            const float s = d >= (a.rot >> 1) ? 1.f : -1.f;
+            r = make_float4(u.x * c0.x + w.x * (c0.y * s), u.y * c0.z + w.y * (c0.w * s), u.z * c1.x + w.z * (c1.y * s),
+                            u.w * c1.z + w.w * (c1.w * s));
+        }
+    }
+    return make_float4(r.x * g, r.y * g, r.z * g, r.w * g);
+}
+__device__ __forceinline__ float4 ret_zero4() { return make_float4(0.f, 0.f, 0.f, 0.f); }
+
+// items tid, tid + THREADS, .. of `total` in batches of U: all of a batch's loads are on their way before its first store
+// (the last batch loads its last item again instead of branching)
+template <int U, int THREADS, typename V, typename Load, typename Store>
+__device__ __forceinline__ void ret_batches(int total, Load load, Store store) {
+    for (int i0 = threadIdx.x; i0 < total; i0 += U * THREADS) {
+        V v[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) v[u] = load(min(i0 + u * THREADS, total - 1));
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+            if (i0 + u * THREADS < total) store(i0 + u * THREADS, v[u]);
+    }
 }
 
 constexpr int RET_STATE_THREADS = 256;
@@ -195,22 +226,20 @@ __global__ void __launch_bounds__(RET_STATE_THREADS) retention_chunk_state_kerne
     const float* proj = pdl_fresh(a.proj);
     const float* pw = a.pw + (size_t)h * (RET_CHUNK + 1);
     const int kq = (ks - 8) / 4, vq = (vs - 8) / 4;
-    for (int i = tid; i < RET_CHUNK * kq; i += RET_STATE_THREADS) {
+    ret_batches<4, RET_STATE_THREADS, RetQuad>(RET_CHUNK * kq, [&](int i) {
+        const int r = i / kq, d = (i - r * kq) * 4, t = t0 + min(r, n - 1);
+        return ret_quad(a, proj + (size_t)t * a.ps + a.ko + (size_t)h * dk, t, d < dk ? d : 0);
+    }, [&](int i, const RetQuad& q) {
         const int r = i / kq, d = (i - r * kq) * 4;
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r < n && d < dk) {
-            v = ret_rotated(a, proj + (size_t)(t0 + r) * a.ps + a.ko + (size_t)h * dk, t0 + r, d);
-            const float f = a.kmul * pw[n - 1 - r];
-            v.x *= f; v.y *= f; v.z *= f; v.w *= f;
-        }
-        ret_split4(v, kh + r * ks + d, kl + r * ks + d);
-    }
-    for (int i = tid; i < RET_CHUNK * vq; i += RET_STATE_THREADS) {
+        ret_split4(r < n && d < dk ? ret_turn(a, q, d, a.kmul * pw[n - 1 - r]) : ret_zero4(), kh + r * ks + d, kl + r * ks + d);
+    });
+    ret_batches<8, RET_STATE_THREADS, float4>(RET_CHUNK * vq, [&](int i) {
         const int r = i / vq, d = (i - r * vq) * 4;
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r < n && d < dv) v = *reinterpret_cast<const float4*>(proj + (size_t)(t0 + r) * a.ps + a.vo + (size_t)h * dv + d);
-        ret_split4(v, vh + r * vs + d, vl + r * vs + d);
-    }
+        return *reinterpret_cast<const float4*>(proj + (size_t)(t0 + min(r, n - 1)) * a.ps + a.vo + (size_t)h * dv + (d < dv ? d : 0));
+    }, [&](int i, float4 v) {
+        const int r = i / vq, d = (i - r * vq) * 4;
+        ret_split4(r < n && d < dv ? v : ret_zero4(), vh + r * vs + d, vl + r * vs + d);
+    });
     __syncthreads();
     float* U = a.ws + ((size_t)blockIdx.x * a.H + h) * (size_t)dv * dk;
     const int mat = lane >> 3, lr = lane & 7;
@@ -289,8 +318,7 @@ __global__ void __launch_bounds__(256) retention_carry_kernel(const RetChunks a)
     for (int c0 = 0; c0 < nc; c0 += AHEAD) {
         float4 v[AHEAD];
 #pragma unroll
-        for (int j = 0; j < AHEAD; ++j)
-            if (c0 + j < nc) v[j] = u[(size_t)(c0 + j) * stride];
+        for (int j = 0; j < AHEAD; ++j) v[j] = u[(size_t)min(c0 + j, nc - 1) * stride];
 #pragma unroll
         for (int j = 0; j < AHEAD; ++j) {
             if (c0 + j >= nc) continue;
@@ -310,7 +338,7 @@ constexpr int RET_OUT_THREADS = 128;
 // The outputs of one chunk and head.  Warp w owns tokens 16 w .. 16 w + 15 of the chunk; the operand on the other side
 // (64 value channels of the incoming state, the chunk's keys, its values) passes through one shared buffer.
 template <int DVP>
-__global__ void __launch_bounds__(RET_OUT_THREADS) retention_chunk_out_kernel(const RetChunks a) {
+__global__ void __launch_bounds__(RET_OUT_THREADS, DVP <= 128 ? 3 : 1) retention_chunk_out_kernel(const RetChunks a) {
     pdl_trigger();
     int t0, n;
     ret_chunk(a, blockIdx.x, t0, n);
@@ -329,15 +357,13 @@ __global__ void __launch_bounds__(RET_OUT_THREADS) retention_chunk_out_kernel(co
     const bool mine = row0 < n;                            // this warp has tokens
     // q (is_k 0) or k rows of the chunk, rotated, as two terms
     auto load_rows = [&](int off, float mul, __nv_bfloat16* hi, __nv_bfloat16* lo) {
-        for (int i = tid; i < RET_CHUNK * kq; i += RET_OUT_THREADS) {
+        ret_batches<4, RET_OUT_THREADS, RetQuad>(RET_CHUNK * kq, [&](int i) {
+            const int r = i / kq, d = (i - r * kq) * 4, t = t0 + min(r, n - 1);
+            return ret_quad(a, proj + (size_t)t * a.ps + off + (size_t)h * dk, t, d < dk ? d : 0);
+        }, [&](int i, const RetQuad& q) {
             const int r = i / kq, d = (i - r * kq) * 4;
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (r < n && d < dk) {
-                v = ret_rotated(a, proj + (size_t)(t0 + r) * a.ps + off + (size_t)h * dk, t0 + r, d);
-                v.x *= mul; v.y *= mul; v.z *= mul; v.w *= mul;
-            }
-            ret_split4(v, hi + r * qs + d, lo + r * qs + d);
-        }
+            ret_split4(r < n && d < dk ? ret_turn(a, q, d, mul) : ret_zero4(), hi + r * qs + d, lo + r * qs + d);
+        });
     };
     load_rows(0, 1.f, qh, ql);
     float o[DVP / 8][4];
@@ -350,13 +376,15 @@ __global__ void __launch_bounds__(RET_OUT_THREADS) retention_chunk_out_kernel(co
 #pragma unroll
     for (int n0 = 0; n0 < DVP; n0 += SB) {
         if (n0 < dv) {
-            for (int i = tid; i < SB * kq; i += RET_OUT_THREADS) {
+            ret_batches<8, RET_OUT_THREADS, uint4>(SB * kq, [&](int i) {
                 const int r = i / kq, d = (i - r * kq) * 4;
-                uint4 v = make_uint4(0u, 0u, 0u, 0u);
-                if (n0 + r < dv && d < dk) v = *reinterpret_cast<const uint4*>(sin + (size_t)(n0 + r) * dk + d);
+                return *reinterpret_cast<const uint4*>(sin + (size_t)min(n0 + r, dv - 1) * dk + (d < dk ? d : 0));
+            }, [&](int i, uint4 v) {
+                const int r = i / kq, d = (i - r * kq) * 4;
+                if (n0 + r >= dv || d >= dk) v = make_uint4(0u, 0u, 0u, 0u);
                 *reinterpret_cast<uint2*>(bh + r * qs + d) = make_uint2(__byte_perm(v.x, v.y, 0x5410), __byte_perm(v.z, v.w, 0x5410));
                 *reinterpret_cast<uint2*>(bl + r * qs + d) = make_uint2(__byte_perm(v.x, v.y, 0x7632), __byte_perm(v.z, v.w, 0x7632));
-            }
+            });
             __syncthreads();
             if (mine)
                 for (int ks = 0; ks < dkp / 16; ++ks) {
@@ -423,12 +451,13 @@ __global__ void __launch_bounds__(RET_OUT_THREADS) retention_chunk_out_kernel(co
             s[nt][e] = back >= 0 ? s[nt][e] * pw[back] : 0.f;
         }
     __syncthreads();
-    for (int i = tid; i < RET_CHUNK * (DVP / 4); i += RET_OUT_THREADS) {
+    ret_batches<8, RET_OUT_THREADS, float4>(RET_CHUNK * (DVP / 4), [&](int i) {
         const int r = i / (DVP / 4), d = (i - r * (DVP / 4)) * 4;
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r < n && d < dv) v = *reinterpret_cast<const float4*>(proj + (size_t)(t0 + r) * a.ps + a.vo + (size_t)h * dv + d);
-        ret_split4(v, bh + r * VS + d, bl + r * VS + d);
-    }
+        return *reinterpret_cast<const float4*>(proj + (size_t)(t0 + min(r, n - 1)) * a.ps + a.vo + (size_t)h * dv + (d < dv ? d : 0));
+    }, [&](int i, float4 v) {
+        const int r = i / (DVP / 4), d = (i - r * (DVP / 4)) * 4;
+        ret_split4(r < n && d < dv ? v : ret_zero4(), bh + r * VS + d, bl + r * VS + d);
+    });
     __syncthreads();
     if (!mine) return;
 #pragma unroll

@@ -118,13 +118,16 @@ class _Sig:
     prism_moe_route_place = [_p, _ll, _i, _i, _i, _i, _i, _i, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f, _f, _p]
     prism_moe_tcgen05_supported = [_i, _i]
     prism_moe_gather = [_p, _ll, _p, _p, _p, _p, _i, _i, _i, _i, _p, _p, _p, _p]
-    prism_moe_gemm_tcgen05 = [_p, _ll, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _ll, _p, _p]
+    prism_moe_gemm_tcgen05 = [_p, _ll, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _ll, _p, _p, _p, _ll, _i, _i, _i, _p,
+                              _ll, _i, _p, _p, _p]
     prism_moe_gemm = [_p, _ll, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _ll, _i, _p]
     prism_hyper_norm = [_p, _ll, _p, _ll, _p, _i, _i, _ll, _p, _i, _p, _i, _p, _i, _i, _p, _i, _f, _i, _p, _i, _p, _i, _i, _p]
     prism_causal_conv = [_p, _ll, _p, _i, _p, _i, _i, _i, _p, _p, _p, _p, _i, _p, _i, _ll, _i, _i, _p, _p]
     prism_block_gates = [_p, _ll, _p, _p, _i, _p, _p, _i, _p, _i, _f, _i, _i, _i, _p, _p, _ll, _p]
     prism_rglru_scan = [_p, _p, _ll, _p, _ll, _p, _p, _p, _i, _i, _i, _p, _i, _ll, _p]
     prism_cache_store = [_p, _ll, _p, _i, _i, _p, _ll, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i, _p, _p]
+    prism_head_product_supported = [_i, _i, _i]
+    prism_head_product = [_p, _ll, _i, _p, _p, _ll, _i, _p, _ll, _i, _i, _i, _i, _p, _p, _i, _i, _i, _f, _p]
     prism_latent_kv_store = [_p, _ll, _p, _i, _f, _i, _i, _i, _p, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i, _p, _p, _i, _p, _i,
                              _p, _ll, _i, _f, _p]
     prism_rotate_slice = [_p, _ll, _i, _p, _ll, _i, _i, _i, _i, _p, _p, _i, _i, _i, _f, _f, _p]
@@ -336,12 +339,12 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out:
     if epi == EPI_PARTIAL:
         assert out.dtype == torch.float32 and out.shape == (ksplit, M, N) and bias is None
     else:
-        assert out.shape == (M, N) and (ksplit == 1 or epi not in _PAIRED)
+        assert out.shape == (M, N)
         assert out.dtype == (torch.float32 if epi == EPI_F32 else torch.bfloat16)
     err = err if err is not None else _tc_err_word(x.device)
     ws = cnt = None
     if ksplit > 1 and epi != EPI_PARTIAL:
-        ws, cnt = _tc_workspace(x.device, ksplit * M * N, (N + 127) // 128)
+        ws, cnt = _tc_workspace(x.device, ksplit * M * w.shape[0], (N + 127) // 128)
     _check(lib().prism_gemm_tcgen05(_ptr(w), w.stride(0), _ptr(x), x.stride(0) if M > 1 else K, _ptr(bias),
                                     F32 if bias is None else _dt(bias), _ptr(out), N, M, N, K, epi, ksplit,
                                     _ptr(ws), _ptr(cnt), _ptr(err), int(group_rows), int(group_tokens), float(limit), _stream()),
@@ -393,6 +396,19 @@ def tc_ksplit(N: int, K: int, sms: Optional[int] = None, M: Optional[int] = None
     if few and kblocks // ks >= 48:
         ks = max(ks, min((3 * n_sms // 2) // tiles, kblocks // 32))
     return ks
+
+
+TC_PAIRED_SPLIT_MAX_M = 16      # csrc/gemm_tcgen05.cu; with more tokens the partial sums cost what the shares gain
+
+
+def tc_ksplit_paired(N: int, K: int, sms: Optional[int] = None, M: Optional[int] = None) -> int:
+    """The same for a paired product (gate and up rows, ``N`` hidden columns): one CTA fills an SM, so as many as leave
+    none waiting, and at least 8 blocks of 64 k each.  A layer with few hidden columns has few tiles, and a CTA streams
+    its weights at some 70 GB/s whatever the rest of the GPU does."""
+    tiles, kblocks = (N + 127) // 128, (K + 63) // 64
+    if M is not None and M > TC_PAIRED_SPLIT_MAX_M:
+        return 1
+    return max(1, min((sms or num_sms()) // tiles, kblocks // 8))
 
 
 def check_tc_errors():
@@ -448,10 +464,13 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
         return out
     # bf16 x bf16, library product with float32 accumulation
     if want == torch.float32:
-        res = torch.mm(x, w.t(), out_dtype=torch.float32)
+        if out is not None and out.is_contiguous():
+            res = torch.mm(x, w.t(), out_dtype=torch.float32, out=out)
+        else:
+            res = torch.mm(x, w.t(), out_dtype=torch.float32)
         if bias is not None:
-            res += bias.float()
-        if out is not None:
+            res += bias
+        if out is not None and res is not out:
             out.copy_(res)
             return out
         return res
@@ -1198,7 +1217,7 @@ def feed_forward_swiglu(ctx, x: torch.Tensor, gate_up_w: torch.Tensor, down_w: t
     M, I = x.shape[0], gate_up_w.shape[0] // 2
     if tc_gemm_ok(x, gate_up_w, TC_GEMM_MAX_M_SWIGLU):
         act = ctx.alloc((M, I), x.dtype)
-        gemm_tc(x, gate_up_w, None, act, EPI_SWIGLU)       # gate/up product with the SwiGLU in its epilogue
+        gemm_tc(x, gate_up_w, None, act, EPI_SWIGLU, ksplit=tc_ksplit_paired(I, x.shape[1], M=M))    # the SwiGLU in its epilogue
         return linear_delta(act, down_w)
     if x.dtype == torch.bfloat16 and gate_up_w.dtype == torch.bfloat16 and M <= GEMV_MAX_M \
             and gemv_supported(M, I, x.shape[1]) and (M == 1 or x.stride(0) % 8 == 0):
@@ -1444,7 +1463,8 @@ def glu_hidden(ctx, x: torch.Tensor, gate_up_w: torch.Tensor, kind: str, limit: 
     the gated activation is the product's epilogue."""
     act = ctx.alloc((x.shape[0], gate_up_w.shape[0] // 2), x.dtype)
     if tc_gemm_ok(x, gate_up_w, TC_GEMM_MAX_M_SWIGLU):
-        gemm_tc(x, gate_up_w, None, act, {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU, "clamped": EPI_CLAMPED}[kind], limit=limit)
+        gemm_tc(x, gate_up_w, None, act, {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU, "clamped": EPI_CLAMPED}[kind],
+                ksplit=tc_ksplit_paired(act.shape[1], x.shape[1], M=x.shape[0]), limit=limit)
     else:
         glu(linear(x, gate_up_w), act, kind, limit)
     return act
@@ -1599,6 +1619,37 @@ def matmul_heads(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor):
             sgemm(x[:, h], w[h], None, out[:, h])
         return
     torch.bmm(x.transpose(0, 1), w.transpose(1, 2), out=out.transpose(0, 1))
+
+
+HEAD_PRODUCT_TOKENS = int(os.environ.get("PRISM_HEAD_PRODUCT_TOKENS", "64"))      # the library's batched product above
+
+
+def head_product_ok(x: torch.Tensor, w: torch.Tensor) -> bool:
+    """Whether the per-head product of a few tokens (csrc/head_product.cu) takes this call."""
+    T, H, K = x.shape
+    return (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and T <= HEAD_PRODUCT_TOKENS
+            and bool(lib().prism_head_product_supported(T, w.shape[1], w.shape[2])) and (T == 1 or x.stride(0) % 8 == 0)
+            and (H == 1 or x.stride(1) % 8 == 0) and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0 and w.is_contiguous())
+
+
+def head_product(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None, rot=None,
+                 positions: Optional[torch.Tensor] = None):
+    """Per head h, for a few tokens: ``out[:, h, :N] = x[:, h, :K] @ w[h].T`` for ``w [H, N, K]``, times ``sigmoid(gate [T,
+    H N])`` where there is a gate; with ``rot`` (a ``RotaryParams``) the entries of ``x`` behind its first K are rotated by
+    the tokens' positions (or copied, beyond the rotated ones) to those of ``out`` behind its first N, in the same launch."""
+    _cuda(x, w, out, gate, positions)
+    T, H, _ = x.shape
+    N, K = w.shape[1], w.shape[2]
+    r = x.shape[2] - K if rot is not None else 0
+    assert w.shape[0] == H and out.shape == (T, H, N + r) and x.stride(2) == 1 and out.stride(2) == 1 and x.shape[2] >= K
+    assert out.dtype == x.dtype == w.dtype == torch.bfloat16
+    if gate is not None:
+        assert gate.shape == (T, H * N) and gate.dtype == torch.float32 and gate.stride(1) == 1
+    rd = rot.rotary_dim if rot is not None else 0
+    _check(lib().prism_head_product(
+        _ptr(x), x.stride(0) if T > 1 else H * x.stride(1), x.stride(1), _ptr(w), _ptr(out), out.stride(0), out.stride(1), _ptr(gate),
+        0 if gate is None else gate.stride(0), T, H, N, K, _ptr(rot.inv_freq) if rd else None, _ptr(positions) if r else None, r, rd,
+        1 if rd and rot.interleaved else 0, float(rot.amplitude) if rd else 1.0, _stream()), "head_product")
 
 
 # --------------------------------------------------------------------------
@@ -2023,6 +2074,15 @@ moe_tensor_cores = True                                 # bf16 experts on tcgen0
 MOE_ONE_CTA_TOKENS = 16       # steps of up to this many tokens are routed and placed by one CTA in one launch (a warp a token at a time: 64 tokens take longer than the three launches)
 
 
+MOE_SHARED_TOKENS = int(os.environ.get("PRISM_MOE_SHARED_TOKENS", "64"))        # steps of up to this many tokens run a shared expert in the experts' own launches
+
+
+def _moe_ksplit(N: int, K: int, live: int) -> int:
+    """CTAs that share one tile's K range in the experts' products of a step of few tokens: as many as the ``live`` experts'
+    tiles leave SMs for, at least 8 blocks of 64 k each."""
+    return max(1, min(num_sms() // (live * -(-N // 128)), (K + 63) // 64 // 8))
+
+
 class MoeChoice:
     """How a router's scores become a choice beyond "the largest": ``correction [E]`` is added to every score for
     the choice only (the weights use the scores without it); the experts form ``groups`` equal groups of
@@ -2062,7 +2122,7 @@ def _moe_route_place(L, logits, T, E, top, softmax, renorm, pad, counts, offs, s
 
 def moe_feed_forward(ctx, x: torch.Tensor, logits: torch.Tensor, gate_up_w: torch.Tensor, down_w: torch.Tensor, top: int,
                      softmax: bool = False, renorm: bool = False, scale_input: bool = True, act: str = "silu",
-                     gated: bool = True, choice: Optional[MoeChoice] = None, extra_planes: int = 0) -> torch.Tensor:
+                     gated: bool = True, choice: Optional[MoeChoice] = None, extra_planes: int = 0, shared=None) -> torch.Tensor:
     """Mixture of experts on the step's rows: ``x [T, W]`` (compute dtype), router ``logits [T, E]`` float32,
     ``gate_up_w [E, 2 F, W]`` (an expert's gate rows, then its up rows), ``down_w [E, W, F]``.  Each token takes the
     ``top`` experts with the largest scores (sigmoid of the logits, or their softmax); a choice's weight is its score
@@ -2070,6 +2130,9 @@ def moe_feed_forward(ctx, x: torch.Tensor, logits: torch.Tensor, gate_up_w: torc
     ``gated`` False: experts without a gate, ``down(act(up(a)))``, and ``gate_up_w`` is ``[E, F, W]``.  ``choice``: a
     ``MoeChoice`` (correction, groups, weight scale).  ``extra_planes``: the stack gets that many more planes after the
     choices' for the caller to fill (a shared expert's result), so that nothing is copied together afterwards.
+    ``shared``: ``(gate_up [2 Fs, W], down [W, Fs])`` of a gated expert with the same activation that every token goes
+    through: its result is the stack's last plane (one more than ``extra_planes``); a step of up to ``MOE_SHARED_TOKENS`` tokens
+    runs it in the experts' own launches.
     Returns float32 ``[top, T, W]``: one plane per choice, which the next norm adds up.  The rows are sorted by
     expert on the device and run as grouped products; the host never learns the counts.  bf16 with rows of 16-byte
     multiples: tcgen05 tiles of one expert each (``csrc/moe_tcgen05.cu``); otherwise CUDA cores (``csrc/moe.cu``)."""
@@ -2085,6 +2148,18 @@ def moe_feed_forward(ctx, x: torch.Tensor, logits: torch.Tensor, gate_up_w: torc
     dev = x.device
     L = lib()
     si = 1 if scale_input else 0
+    if shared is not None:
+        sgu, sdn = shared
+        Fs = sdn.shape[1]
+        assert gated and sgu.shape == (2 * Fs, W) and sdn.shape[0] == W and sgu.is_contiguous() and sdn.is_contiguous()
+        ride = (T <= MOE_SHARED_TOKENS and x.dtype == torch.bfloat16 and moe_tensor_cores and sgu.dtype == sdn.dtype == x.dtype
+                and Fs % 8 == 0 and L.prism_moe_tcgen05_supported(W, F) and x.stride(0) % 8 == 0 and sgu.data_ptr() % 16 == 0
+                and sdn.data_ptr() % 16 == 0 and x.data_ptr() % 16 == 0)
+        if not ride:
+            y = moe_feed_forward(ctx, x, logits, gate_up_w, down_w, top, softmax, renorm, scale_input, act, gated, choice,
+                                 extra_planes + 1)
+            linear(glu_hidden(ctx, x, sgu, act), sdn, None, out=y[-1])
+            return y
     if x.dtype == torch.bfloat16 and moe_tensor_cores and L.prism_moe_tcgen05_supported(W, F) and x.stride(0) % 8 == 0:
         # tensor cores: every expert's rows start at a multiple of the token tile, one tile has one expert
         ntok = 16 if T <= 16 else (32 if T <= 32 else 64)
@@ -2098,16 +2173,30 @@ def moe_feed_forward(ctx, x: torch.Tensor, logits: torch.Tensor, gate_up_w: torc
         sel_w, row_w = flt[:rows], flt[rows:]
         err = _tc_err_word(dev)
         _moe_route_place(L, logits, T, E, top, softmax, renorm, ntok, counts, offs, sel_e, sel_w, sel_rank, None, None, None, choice)
+        sT, s1, s2, k1, k2 = 0, (None, None, 0, 0, 0, 0, None, 0), (None, None, 0, 0, 0, 0, None, 0), 1, 1
+        y = ctx.alloc((top + extra_planes + (1 if shared is not None else 0), T, W), torch.float32)
+        if shared is not None:
+            sT, sh = T, ctx.alloc((T, Fs), x.dtype)
+            s1 = (_ptr(sgu), _ptr(x), x.stride(0) if T > 1 else W, T, Fs, W, _ptr(sh), Fs)
+            s2 = (_ptr(sdn), _ptr(sh), Fs, T, W, Fs, _ptr(y[-1]), W)
+        if T <= MOE_ONE_CTA_TOKENS:
+            # few tokens: an expert's tiles are few, and each is a long walk over K for its CTA
+            live = min(E, rows) + (1 if sT else 0)
+            k1, k2 = _moe_ksplit(max(F, Fs if sT else 0), W, live), _moe_ksplit(W, F, live)
+        tx1, tx2, ty = -(-max(F, Fs if sT else 0) // 128), -(-W // 128), tiles + -(-sT // ntok)
+        ws = cnt = None
+        if max(k1, k2) > 1:
+            ws, cnt = _tc_workspace(dev, max(tx1 * k1 * (2 if gated else 1), tx2 * k2) * ty * ntok * 128, max(tx1, tx2) * ty)
         xs = ctx.alloc((padded, W), x.dtype)
         _check(L.prism_moe_gather(_ptr(x), x.stride(0), _ptr(offs), _ptr(sel_e), _ptr(sel_w), _ptr(sel_rank), T, int(top), W, si,
                                   _ptr(xs), _ptr(row_dst), _ptr(row_w), _stream()), "moe_gather")
         hidden = ctx.alloc((padded, F), x.dtype)
         _check(L.prism_moe_gemm_tcgen05(_ptr(xs), W, _ptr(gate_up_w), _ptr(offs), _ptr(counts), None, None, ntok, tiles, E, F, W,
-                                        gt, MOE_ACTS[act], _ptr(hidden), F, _ptr(err), _stream()), "moe_gemm_tcgen05")
-        y = ctx.alloc((top + extra_planes, T, W), torch.float32)
+                                        gt, MOE_ACTS[act], _ptr(hidden), F, _ptr(err), *s1, k1, _ptr(ws), _ptr(cnt), _stream()),
+               "moe_gemm_tcgen05")
         _check(L.prism_moe_gemm_tcgen05(_ptr(hidden), F, _ptr(down_w), _ptr(offs), _ptr(counts), _ptr(row_dst),
                                         None if scale_input else _ptr(row_w), ntok, tiles, E, W, F, 0, 0, _ptr(y), W, _ptr(err),
-                                        _stream()), "moe_gemm_tcgen05")
+                                        *s2, k2, _ptr(ws), _ptr(cnt), _stream()), "moe_gemm_tcgen05")
         return y
     ints = torch.empty(E + (E + 1) + 4 * rows, dtype=torch.int32, device=dev)
     counts, offs = ints[:E], ints[E:2 * E + 1]

@@ -442,14 +442,22 @@ class LatentAttention(Mixer):
                             interleaved=rot.interleaved, amplitude=rot.amplitude)
         q = ops.linear(cq, self.w["uq_w"]).view(T, nh, hd + rd)
         qf = ctx.alloc((T, nh, R + rd), x.dtype)                   # per head [plain part in latent space | rotated part]
-        ops.matmul_heads(q[:, :, :hd], self.uk_t, qf[:, :, :R])
-        if rd:
+        few = ops.head_product_ok(q, self.uk_t)
+        if few:                                                    # both parts of a query in one launch
+            ops.head_product(q, self.uk_t, qf, rot=rot, positions=ctx.positions)
+        else:
+            ops.matmul_heads(q[:, :, :hd], self.uk_t, qf[:, :, :R])
+        if rd and not few:
             ops.rotate_slice(q[:, :, hd:], qf[:, :, R:], rot.rotary_dim, rot.inv_freq, ctx.positions, rot.interleaved,
                              rot.amplitude)
         lat = ctx.alloc((T, nh * R), x.dtype)
         ops.masked_attention(ctx, qf, lat, cache.k, cache.k[..., :R], cache.block_table, cache.num_pages, self.mask,
                              self.scale, self.w["sink"] if self.sink else None)
+        gate = down[:, g0:] if self.gate else None
+        if ops.head_product_ok(lat.view(T, nh, R), self.uv):
+            ops.head_product(lat.view(T, nh, R), self.uv, out.view(T, nh, self.vhd), gate)
+            return
         heads = ctx.alloc((T, nh * self.vhd), x.dtype) if self.gate else out
         ops.matmul_heads(lat.view(T, nh, R), self.uv, heads.view(T, nh, self.vhd))
         if self.gate:
-            ops.gated_product(heads, down[:, g0:], out, "sigmoid")
+            ops.gated_product(heads, gate, out, "sigmoid")

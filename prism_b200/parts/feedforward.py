@@ -154,10 +154,13 @@ class MixtureOfExperts(FeedForward):
 
     def forward(self, ctx, x):
         H, I, E = self.hidden_size, self.intermediate_size, self.experts
+        # a gated shared expert with the experts' own activation runs with them
+        alike = isinstance(self.shared, SwiGLU) and self.gated and self.shared.activation == self.activation
         logits = ops.linear(x, self.w["router_w"], self.w.get("router_b"), out_dtype=ops.torch.float32)
         y = ops.moe_feed_forward(ctx, x, logits, self.w["gate_up_w"].view(E, (2 if self.gated else 1) * I, H),
                                  self.w["down_w"].view(E, H, I), self.top, self.softmax, self.renorm, self.scale_input,
-                                 self.activation, self.gated, self.choice, extra_planes=0 if self.shared is None else 1)
-        if self.shared is not None:
+                                 self.activation, self.gated, self.choice, extra_planes=0 if self.shared is None or alike else 1,
+                                 shared=(self.shared.w["gate_up_w"], self.shared.w["down_w"]) if alike else None)
+        if self.shared is not None and not alike:
             self.shared.forward_to(ctx, x, y[self.top])          # the shared expert's result is the stack's last plane
         return y
