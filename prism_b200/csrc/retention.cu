@@ -195,17 +195,28 @@ __device__ __forceinline__ float4 ret_turn(const RetChunks& a, const RetQuad& q,
 }
 __device__ __forceinline__ float4 ret_zero4() { return make_float4(0.f, 0.f, 0.f, 0.f); }
 
-// items tid, tid + THREADS, .. of `total` in batches of U: all of a batch's loads are on their way before its first store
-// (the last batch loads its last item again instead of branching)
+// The quads of a [rows, 4 cols] tile, dealt out to the threads in turn, in batches of U: all of a batch's loads are on their
+// way before its first store (past the end the tile's last row is loaded again instead of branching).  A thread walks its
+// (row, quad) pairs by adding, it divides once.
 template <int U, int THREADS, typename V, typename Load, typename Store>
-__device__ __forceinline__ void ret_batches(int total, Load load, Store store) {
-    for (int i0 = threadIdx.x; i0 < total; i0 += U * THREADS) {
+__device__ __forceinline__ void ret_batches(int rows, int cols, Load load, Store store) {
+    const int dr = THREADS / cols, dc = THREADS - dr * cols;
+    int r = threadIdx.x / cols, c = threadIdx.x - r * cols;
+    while (r < rows) {
         V v[U];
+        int rr[U], cc[U];
 #pragma unroll
-        for (int u = 0; u < U; ++u) v[u] = load(min(i0 + u * THREADS, total - 1));
+        for (int u = 0; u < U; ++u) {
+            rr[u] = r;
+            cc[u] = c;
+            r += dr;
+            c += dc;
+            if (c >= cols) { c -= cols; ++r; }
+            v[u] = load(min(rr[u], rows - 1), cc[u] * 4);
+        }
 #pragma unroll
         for (int u = 0; u < U; ++u)
-            if (i0 + u * THREADS < total) store(i0 + u * THREADS, v[u]);
+            if (rr[u] < rows) store(rr[u], cc[u] * 4, v[u]);
     }
 }
 
@@ -226,18 +237,15 @@ __global__ void __launch_bounds__(RET_STATE_THREADS) retention_chunk_state_kerne
     const float* proj = pdl_fresh(a.proj);
     const float* pw = a.pw + (size_t)h * (RET_CHUNK + 1);
     const int kq = (ks - 8) / 4, vq = (vs - 8) / 4;
-    ret_batches<4, RET_STATE_THREADS, RetQuad>(RET_CHUNK * kq, [&](int i) {
-        const int r = i / kq, d = (i - r * kq) * 4, t = t0 + min(r, n - 1);
+    ret_batches<4, RET_STATE_THREADS, RetQuad>(RET_CHUNK, kq, [&](int r, int d) {
+        const int t = t0 + min(r, n - 1);
         return ret_quad(a, proj + (size_t)t * a.ps + a.ko + (size_t)h * dk, t, d < dk ? d : 0);
-    }, [&](int i, const RetQuad& q) {
-        const int r = i / kq, d = (i - r * kq) * 4;
+    }, [&](int r, int d, const RetQuad& q) {
         ret_split4(r < n && d < dk ? ret_turn(a, q, d, a.kmul * pw[n - 1 - r]) : ret_zero4(), kh + r * ks + d, kl + r * ks + d);
     });
-    ret_batches<8, RET_STATE_THREADS, float4>(RET_CHUNK * vq, [&](int i) {
-        const int r = i / vq, d = (i - r * vq) * 4;
+    ret_batches<8, RET_STATE_THREADS, float4>(RET_CHUNK, vq, [&](int r, int d) {
         return *reinterpret_cast<const float4*>(proj + (size_t)(t0 + min(r, n - 1)) * a.ps + a.vo + (size_t)h * dv + (d < dv ? d : 0));
-    }, [&](int i, float4 v) {
-        const int r = i / vq, d = (i - r * vq) * 4;
+    }, [&](int r, int d, float4 v) {
         ret_split4(r < n && d < dv ? v : ret_zero4(), vh + r * vs + d, vl + r * vs + d);
     });
     __syncthreads();
@@ -357,11 +365,10 @@ __global__ void __launch_bounds__(RET_OUT_THREADS, DVP <= 128 ? 3 : 1) retention
     const bool mine = row0 < n;                            // this warp has tokens
     // q (is_k 0) or k rows of the chunk, rotated, as two terms
     auto load_rows = [&](int off, float mul, __nv_bfloat16* hi, __nv_bfloat16* lo) {
-        ret_batches<4, RET_OUT_THREADS, RetQuad>(RET_CHUNK * kq, [&](int i) {
-            const int r = i / kq, d = (i - r * kq) * 4, t = t0 + min(r, n - 1);
+        ret_batches<4, RET_OUT_THREADS, RetQuad>(RET_CHUNK, kq, [&](int r, int d) {
+            const int t = t0 + min(r, n - 1);
             return ret_quad(a, proj + (size_t)t * a.ps + off + (size_t)h * dk, t, d < dk ? d : 0);
-        }, [&](int i, const RetQuad& q) {
-            const int r = i / kq, d = (i - r * kq) * 4;
+        }, [&](int r, int d, const RetQuad& q) {
             ret_split4(r < n && d < dk ? ret_turn(a, q, d, mul) : ret_zero4(), hi + r * qs + d, lo + r * qs + d);
         });
     };
@@ -376,11 +383,9 @@ __global__ void __launch_bounds__(RET_OUT_THREADS, DVP <= 128 ? 3 : 1) retention
 #pragma unroll
     for (int n0 = 0; n0 < DVP; n0 += SB) {
         if (n0 < dv) {
-            ret_batches<8, RET_OUT_THREADS, uint4>(SB * kq, [&](int i) {
-                const int r = i / kq, d = (i - r * kq) * 4;
+            ret_batches<8, RET_OUT_THREADS, uint4>(SB, kq, [&](int r, int d) {
                 return *reinterpret_cast<const uint4*>(sin + (size_t)min(n0 + r, dv - 1) * dk + (d < dk ? d : 0));
-            }, [&](int i, uint4 v) {
-                const int r = i / kq, d = (i - r * kq) * 4;
+            }, [&](int r, int d, uint4 v) {
                 if (n0 + r >= dv || d >= dk) v = make_uint4(0u, 0u, 0u, 0u);
                 *reinterpret_cast<uint2*>(bh + r * qs + d) = make_uint2(__byte_perm(v.x, v.y, 0x5410), __byte_perm(v.z, v.w, 0x5410));
                 *reinterpret_cast<uint2*>(bl + r * qs + d) = make_uint2(__byte_perm(v.x, v.y, 0x7632), __byte_perm(v.z, v.w, 0x7632));
@@ -451,11 +456,9 @@ __global__ void __launch_bounds__(RET_OUT_THREADS, DVP <= 128 ? 3 : 1) retention
             s[nt][e] = back >= 0 ? s[nt][e] * pw[back] : 0.f;
         }
     __syncthreads();
-    ret_batches<8, RET_OUT_THREADS, float4>(RET_CHUNK * (DVP / 4), [&](int i) {
-        const int r = i / (DVP / 4), d = (i - r * (DVP / 4)) * 4;
+    ret_batches<8, RET_OUT_THREADS, float4>(RET_CHUNK, DVP / 4, [&](int r, int d) {
         return *reinterpret_cast<const float4*>(proj + (size_t)(t0 + min(r, n - 1)) * a.ps + a.vo + (size_t)h * dv + (d < dv ? d : 0));
-    }, [&](int i, float4 v) {
-        const int r = i / (DVP / 4), d = (i - r * (DVP / 4)) * 4;
+    }, [&](int r, int d, float4 v) {
         ret_split4(r < n && d < dv ? v : ret_zero4(), bh + r * VS + d, bl + r * VS + d);
     });
     __syncthreads();
