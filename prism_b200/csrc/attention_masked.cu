@@ -506,6 +506,18 @@ static int launch_masked(const MaskedAttn& a, int S, int max_q_len, cudaStream_t
 
 }  // namespace prism
 
+// out [T, nh * dv] bf16 from partial results part_o [T, nh, nsplit, dv] and part_ml [T, nh, nsplit, 2] (reference exponent in
+// the log2 domain, sum), sink included.
+PRISM_EXPORT int prism_attention_masked_merge(const float* part_o, const float* part_ml, int nsplit, int T, int nh, int dv,
+                                              const void* sink, int sink_dtype, void* out, long long out_stride,
+                                              cudaStream_t stream) {
+    using namespace prism;
+    if (T <= 0 || nh <= 0) return 0;
+    if (nsplit < 1 || nsplit > MA_MERGE_MAX || dv < 1) return (int)cudaErrorInvalidValue;
+    return (int)launch_kernel(attn_masked_merge_kernel, dim3(T * nh), dim3(dv >= 256 ? 256 : (dv + 31) / 32 * 32), 0, stream, part_o,
+                              part_ml, nsplit, dv, nh, sink, sink_dtype == PRISM_DTYPE_BF16, (__nv_bfloat16*)out, out_stride);
+}
+
 // Whether the tensor-core kernel takes these sizes: keys and values in whole 16-byte pieces, values up to
 // 256 entries (the output tile lives in registers), keys up to 576.
 PRISM_EXPORT int prism_attention_masked_supported(int dk, int dv, int nh, int nkv) {

@@ -96,6 +96,9 @@ class _Sig:
     prism_attention_masked_bf16 = [_p, _ll, _i, _p, _ll, _p, _ll, _i, _p, _ll, _i, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i,
                                    _i, _i, _i, _i, _i, _f, _p, _i, _i, _i, _p, _p, _p, _p, _i, _p]
     prism_add_normed_rmsnorm = [_p, _p, _i, _i, _ll, _p, _i, _f, _p, _i, _f, _p, _i, _p, _i, _i, _p]
+    prism_attention_latent_tc_supported = [_i, _i, _i]
+    prism_attention_latent_tc = [_p, _i, _p, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _i, _i, _p, _p, _p, _p]
+    prism_attention_masked_merge = [_p, _p, _i, _i, _i, _i, _p, _i, _p, _ll, _p]
     prism_scale_add_rmsnorm = [_p, _f, _p, _i, _i, _ll, _p, _i, _f, _p, _i, _i, _i, _p]
     prism_gated_product = [_p, _ll, _p, _ll, _p, _ll, _i, _i, _i, _i, _f, _i, _p]
     prism_qk_norm_rope_store = [_p, _p, _p, _ll, _p, _i, _p, _i, _f, _p, _i, _p, _p, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i,
@@ -1488,12 +1491,60 @@ def masked_attention(ctx, q: torch.Tensor, out: torch.Tensor, k_plane: torch.Ten
     if (q.dtype == torch.bfloat16 and MASKED_TC and not FORCE_GENERIC_ATTENTION
             and attention_masked_tc_ok(q, k_plane, v_plane, nh, nkv, dk, dv)):
         few = ctx.decode_only
+        if (not few and dist_bias is None and scale > 0 and ctx.max_q_len * nh >= LATENT_TC_MIN_ROWS
+                and attention_latent_tc_ok(q, out, k_plane, v_plane, mask)):
+            attention_latent_tc(q, out, k_plane, dv, block_table, ctx.seg_start, ctx.cached_len, ctx.S, ctx.max_q_len, num_pages, mask,
+                                scale, sink, ctx.err, nsplit=latent_splits(ctx.S, ctx.max_q_len * nh, mask.most_keys(ctx.max_kv_len)))
+            return
         ns = masked_decode_splits(ctx.S, nkv * (-(-(nh // nkv) // 16)), mask.most_keys(ctx.max_kv_len)) if few else 1
         attention_masked_bf16(q, out, k_plane, v_plane, block_table, ctx.seg_start, ctx.cached_len, ctx.S,
                               ctx.max_q_len, num_pages, mask, scale, sink, few, ctx.err, nsplit=ns, dist_bias=dist_bias)
         return
     attention_masked_generic(q, out, k_plane, v_plane, block_table, ctx.positions, ctx.tok_seg, num_pages, mask,
                              scale, sink, ctx.err, dist_bias)
+
+
+LATENT_TC_MIN_ROWS = int(os.environ.get("PRISM_LATENT_TC_MIN_ROWS", "64"))      # (token, head) rows of a portion; fewer: 64-row mma.sync tiles
+
+
+def attention_latent_tc_ok(q, out, k_plane, v_plane, mask: KeyMask) -> bool:
+    """Whether the tcgen05 kernel for one kv head with its values inside its keys takes this call."""
+    T, nh, dk = q.shape
+    return (k_plane.shape[2] == 1 and _values_in_keys(k_plane, v_plane) and k_plane.is_contiguous() and q.is_contiguous()
+            and out.is_contiguous() and mask.kind in (MASK_CAUSAL, MASK_WINDOW) and mask.keep == 0 and q.data_ptr() % 16 == 0
+            and out.data_ptr() % 16 == 0 and k_plane.data_ptr() % 16 == 0
+            and bool(lib().prism_attention_latent_tc_supported(dk, v_plane.shape[3], k_plane.shape[1])))
+
+
+def latent_splits(S: int, rows: int, most_keys: int, sms: Optional[int] = None) -> int:
+    """CTAs that share the key tiles of 128 rows: 1 unless the row tiles leave half of the GPU idle and the keys are many;
+    then as many as fill it (one a SM), each with at least 8 tiles of 64 keys."""
+    ctas, tiles = S * -(-rows // 128), -(-most_keys // 64)
+    return max(1, min((sms or num_sms()) // ctas, tiles // 8, 16))
+
+
+def attention_latent_tc(q, out, k_plane, dv: int, block_table, seg_start, cached_len, S: int, max_q_len: int, num_pages: int,
+                        mask: KeyMask, scale: float, sink: Optional[torch.Tensor], err: torch.Tensor, nsplit: int = 1):
+    """Attention of all heads of ``q [T, nh, dk]`` over one cached row per token (``k_plane [pages, P, 1, dk]``) whose first
+    ``dv`` entries are the value, for segments of any length, on the 5th-generation tensor cores; ``nsplit`` > 1: that many CTAs
+    share a row tile's keys and a second kernel merges their partial results."""
+    _cuda(q, out, k_plane, block_table, seg_start, cached_len, sink)
+    T, nh, dk = q.shape
+    assert q.dtype == k_plane.dtype == out.dtype == torch.bfloat16 and q.is_contiguous() and out.is_contiguous() and k_plane.is_contiguous()
+    assert out.shape == (T, nh * dv) and k_plane.shape[2:] == (1, dk) and seg_start.shape[0] == S + 1 and cached_len.shape[0] == S
+    assert sink is None or (sink.shape == (nh,) and sink.is_contiguous())
+    po = pml = None
+    if nsplit > 1:
+        po = torch.empty((T, nh, nsplit, dv), dtype=torch.float32, device=q.device)
+        pml = torch.empty((T, nh, nsplit, 2), dtype=torch.float32, device=q.device)
+    sdt = F32 if sink is None else _dt(sink)
+    _check(lib().prism_attention_latent_tc(_ptr(q), T, _ptr(out), _ptr(k_plane), k_plane.shape[0], _ptr(block_table), block_table.shape[1],
+                                           _ptr(seg_start), _ptr(cached_len), S, int(max_q_len), nh, dk, dv, k_plane.shape[1], num_pages,
+                                           mask.size if mask.kind == MASK_WINDOW else 0, float(scale), _ptr(sink), sdt, int(nsplit),
+                                           _ptr(po), _ptr(pml), _ptr(err), _stream()), "attention_latent_tc")
+    if nsplit > 1:
+        _check(lib().prism_attention_masked_merge(_ptr(po), _ptr(pml), int(nsplit), T, nh, dv, _ptr(sink), sdt, _ptr(out), out.stride(0),
+                                                  _stream()), "attention_masked_merge")
 
 
 MASKED_TC = os.environ.get("PRISM_MASKED_TC", "1") != "0"

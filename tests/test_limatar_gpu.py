@@ -284,7 +284,7 @@ def test_experts_with_a_shared_one_in_their_launches(T, W, F, E, top, Fs, dtype)
     ops.check_tc_errors()
 
 
-def latent_case(segs, nh, R, rd, page_size, dtype, seed, boost=None):
+def latent_case(segs, nh, R, rd, page_size, dtype, seed, boost=None, mask=None):
     """One key row per position (all heads share it), its first R entries the value; pages in a scrambled order."""
     g = torch.Generator().manual_seed(seed)
     per = [-(-(c + n) // page_size) for c, n in segs]
@@ -312,22 +312,30 @@ def latent_case(segs, nh, R, rd, page_size, dtype, seed, boost=None):
     for s, (c, n) in enumerate(segs):
         k = rows[ids[s]].reshape(-1, R + rd)[:c + n].double()
         for i in range(n):
-            sc = (q[t].double() @ k[:c + i + 1].T) * 0.2
-            outs.append(LP.sink_softmax(sc, sink.double()[:, None]) @ k[:c + i + 1, :R])
+            first = mask.first_key(c + i) if mask is not None else 0
+            sc = (q[t].double() @ k[first:c + i + 1].T) * 0.2
+            outs.append(LP.sink_softmax(sc, sink.double()[:, None]) @ k[first:c + i + 1, :R])
             t += 1
     return ctx, q.to(DEV), rows.to(DEV), bt.to(DEV), sink, torch.stack(outs).reshape(T, nh * R)
 
 
-KERNELS = ["generic_f32", "generic_bf16", "tc_portions", "tc_decode", "tc_decode:3", "tc_decode:7"]
+KERNELS = ["generic_f32", "generic_bf16", "tc_portions", "tc_decode", "tc_decode:3", "tc_decode:7", "tcgen05", "tcgen05:3"]
 
 
-def latent_attention(kernel, segs, nh, R, rd, page_size, seed, boost=None):
+def latent_attention(kernel, segs, nh, R, rd, page_size, seed, boost=None, mask=None):
     from prism_b200 import ops
     dtype = torch.float32 if kernel == "generic_f32" else torch.bfloat16
-    ctx, q, rows, bt, sink, ref = latent_case(segs, nh, R, rd, page_size, dtype, seed, boost)
+    ctx, q, rows, bt, sink, ref = latent_case(segs, nh, R, rd, page_size, dtype, seed, boost, mask)
     out = torch.empty(q.shape[0], nh * R, dtype=dtype, device=DEV)
-    mask, n = ops.KeyMask.causal(), rows.shape[0]
-    if kernel.startswith("generic"):
+    mask, n = mask or ops.KeyMask.causal(), rows.shape[0]
+    if kernel.startswith("tcgen05"):
+        if not ops.attention_latent_tc_ok(q, out, rows, rows[..., :R], mask):
+            assert page_size % 64
+            pytest.skip("key tiles do not lie in one page")
+        ops.attention_latent_tc(q, out, rows, R, bt, ctx.seg_start, ctx.cached_len, ctx.S, ctx.max_q_len, n, mask, 0.2, sink.to(DEV), ctx.err,
+                                nsplit=int(kernel.split(":")[1]) if ":" in kernel else 1)
+        ops.check_tc_errors()
+    elif kernel.startswith("generic"):
         ops.attention_masked_generic(q, out, rows, rows[..., :R], bt, ctx.positions, ctx.tok_seg, n, mask, 0.2, sink.to(DEV), ctx.err)
     else:
         few = kernel.startswith("tc_decode")
@@ -346,6 +354,31 @@ def test_latent_attention_with_a_sink(shape, page_size, kernel):
     segs = [(0, 1), (63, 1), (64, 1), (300, 1), (129, 1), (447, 1)] if kernel.startswith("tc_decode") else [(0, 3), (200, 40), (63, 2), (0, 130)]
     got, ref = latent_attention(kernel, segs, *shape, page_size, 5)
     assert float((got - ref).abs().max()) <= (2e-5 if kernel == "generic_f32" else 2e-2) * max(1.0, float(ref.abs().max()))
+
+
+@pytest.mark.parametrize("window", [1, 30, 64, 65, 100, 500])
+@pytest.mark.parametrize("kernel", ["generic_f32", "tc_portions", "tcgen05", "tcgen05:2"])
+def test_latent_attention_under_a_window(window, kernel):
+    from prism_b200 import ops
+    got, ref = latent_attention(kernel, [(0, 3), (200, 40), (63, 2), (0, 130), (330, 70)], 6, 80, 16, 64, 7, mask=ops.KeyMask.window(window))
+    assert float((got - ref).abs().max()) <= (2e-5 if kernel == "generic_f32" else 2e-2) * max(1.0, float(ref.abs().max()))
+
+
+def test_unwritten_rows_of_a_page_do_not_reach_the_result():
+    """The slots behind the last key of a page hold NaN (a pool that nothing was stored in yet): no kernel may let them in."""
+    from prism_b200 import ops
+    for segs in ([(0, 70), (64, 30)], [(69, 1), (3, 1)]):
+        few = segs[0][1] == 1
+
+        def boost(q, rows, ids):
+            for (c, n), pages in zip(segs, ids):
+                last = c + n
+                if last % 64:
+                    rows[pages[(last - 1) // 64], last % 64:] = math.nan
+        for kernel in (("generic_f32", "tc_decode", "tc_decode:3") if few else ("generic_f32", "tc_portions", "tcgen05", "tcgen05:2")):
+            got, ref = latent_attention(kernel, segs, 4, 96, 32, 64, 3, boost)
+            assert bool(torch.isfinite(got).all()), kernel
+            assert float((got - ref).abs().max()) <= 2e-2 * max(1.0, float(ref.abs().max())), kernel
 
 
 @pytest.mark.parametrize("kernel", KERNELS)
@@ -379,7 +412,10 @@ def test_a_large_sink_takes_the_weight(kernel):
     out = torch.empty(1, 32, dtype=dtype, device=DEV)
     for value, share in ((math.log(n), 0.5), (-40.0, 1.0), (math.log(3.0 * n), 0.25)):
         sink = torch.full((2,), value, device=DEV)
-        if kernel.startswith("generic"):
+        if kernel.startswith("tcgen05"):
+            ops.attention_latent_tc(q, out, rows, 16, bt, ctx.seg_start, ctx.cached_len, 1, 1, rows.shape[0], ops.KeyMask.causal(), 0.2, sink,
+                                    ctx.err, nsplit=int(kernel.split(":")[1]) if ":" in kernel else 1)
+        elif kernel.startswith("generic"):
             ops.attention_masked_generic(q, out, rows, rows[..., :16], bt, ctx.positions, ctx.tok_seg, rows.shape[0], ops.KeyMask.causal(), 0.2,
                                          sink, ctx.err)
         else:
