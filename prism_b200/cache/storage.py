@@ -65,11 +65,15 @@ class CacheStorage:
         return sum(t.numel() * t.element_size() for d in (self.k, self.v, self.state) for t in d.values())
 
     def clear_slots(self, slots: List[int]) -> None:
-        """State of requests that have just been admitted starts at zero."""
+        """State of requests that have just been admitted starts at zero.  (The indices travel from pinned memory and the
+        fill value with the launch: a copy from pageable memory would make the host wait for the step before.)"""
         if slots and self.state:
-            idx = torch.tensor(slots, dtype=torch.long, device=next(iter(self.state.values())).device)
+            dev = next(iter(self.state.values())).device
+            idx = torch.tensor(slots, dtype=torch.long)
+            if dev.type == "cuda":
+                idx = idx.pin_memory().to(dev, non_blocking=True)
             for t in self.state.values():
-                t[:, idx] = 0
+                t.index_fill_(1, idx, 0)
 
     def views(self, block_tables, slots_dev, host_slots) -> list:
         """Per schedule entry the view its mixer gets (None if it needs no cache)."""

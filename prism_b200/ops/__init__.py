@@ -163,7 +163,8 @@ class _Sig:
 
 
 def _stream() -> int:
-    return torch.cuda.current_stream().cuda_stream
+    # the raw handle: torch.cuda.current_stream() makes a Stream object first, microseconds a launch
+    return torch._C._cuda_getCurrentRawStream(torch._C._cuda_getDevice())
 
 
 def _ptr(t: Optional[torch.Tensor]):
