@@ -1,6 +1,6 @@
 // Causal (or windowed) attention of all heads over one cached row per token whose first entries are the value - latent
-// attention, and any layer with one kv head and its values inside its keys - for portions of prompts, on the
-// 5th-generation tensor cores.
+// attention, and any layer with one kv head and its values inside its keys - for portions of prompts and decode steps, on
+// the 5th-generation tensor cores.
 //
 // The (token, head) pairs of a segment are one run of rows: a CTA owns 128 of them (UMMA M), whatever the number of heads,
 // and walks the keys in tiles of 64.  Roles as in attention_tcgen05.cu (warp 0 TMA producer, warp 1 MMA issue, warps 2-5
@@ -47,7 +47,6 @@ template <int HALVES>                // 64-entry (128-byte) boxes per key row
 __global__ void __launch_bounds__(L_THREADS, 1)
 attn_latent_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const LatentAttn a) {
     constexpr int Q_BYTES = LQ * HALVES * 128, K_BYTES = LK * HALVES * 128;
-    pdl_wait();
     const int seg = blockIdx.y;
     const int s0 = a.seg_start[seg], nrows = (a.seg_start[seg + 1] - s0) * a.nh;
     const int split = blockIdx.x % a.nsplit;
@@ -82,6 +81,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         t0 += split * per;
         n = min(per, n - split * per);
         if (n <= 0) {                 // no key tile for this split: an empty partial
+            pdl_wait();
             for (int i = threadIdx.x; i < rows * a.dv; i += L_THREADS)
                 a.part_o[((size_t)(row0 + i / a.dv) * a.nsplit + split) * a.dv + i % a.dv] = 0.f;
             for (int r = threadIdx.x; r < rows; r += L_THREADS) {
@@ -93,6 +93,20 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         }
     }
 
+    // key tile j of this CTA into its stage (one thread)
+    auto load_keys = [&](int j) {
+        const int s = j % L_STAGES, key0 = (t0 + j) * LK;
+        int page = bt[key0 / a.page_size];
+        if (page < 0 || page >= a.num_pages) {
+            report_error(a.err, PRISM_ERR_PAGE_RANGE);
+            page = 0;                                    // the result is flagged; read something that exists
+        }
+        const int row = page * a.page_size + key0 % a.page_size;
+        mbar_expect_tx(&k_full[s], K_BYTES);
+#pragma unroll
+        for (int hh = 0; hh < HALVES; ++hh) tma_load_2d(Ks + s * K_BYTES + hh * LK * 128, &map_k, &k_full[s], hh * 64, row);
+    };
+    int early = 0;
     if (threadIdx.x == 0) {
         abort_flag = 0;
         mbar_init(q_full, 1);
@@ -100,7 +114,11 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         for (int s = 0; s < 2; ++s) { mbar_init(&s_full[s], 1); mbar_init(&p_full[s], 128); mbar_init(&pv_done[s], 1); }
         mbar_init(o_done, 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        // The step's descriptor is there before its first kernel starts, and keys of earlier steps are in the cache: the
+        // first tiles, as far as they hold no key of this step, are asked for before the kernels before this one have ended.
+        while (early < min(n, L_STAGES) && (t0 + early + 1) * LK <= cached) load_keys(early++);
     }
+    pdl_wait();
     if (warp == 1) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_addr(tmem_slot)), "r"(L_TMEM));
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::);
@@ -118,20 +136,10 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             mbar_expect_tx(q_full, Q_BYTES);
 #pragma unroll
             for (int hh = 0; hh < HALVES; ++hh) tma_load_2d(Qs + hh * LQ * 128, &map_q, q_full, hh * 64, (int)row0);
-            int issued = 0;
-            for (int j = 0; j < n; ++j) {
-                const int s = j % L_STAGES, key0 = (t0 + j) * LK;
-                int page = bt[key0 / a.page_size];
-                if (page < 0 || page >= a.num_pages) {
-                    report_error(a.err, PRISM_ERR_PAGE_RANGE);
-                    page = 0;                                    // the result is flagged; read something that exists
-                }
-                const int row = page * a.page_size + key0 % a.page_size;
-                if (j >= L_STAGES && !mbar_wait(&k_empty[s], ((j / L_STAGES) - 1) & 1, abortp)) break;
-                mbar_expect_tx(&k_full[s], K_BYTES);
-#pragma unroll
-                for (int hh = 0; hh < HALVES; ++hh)
-                    tma_load_2d(Ks + s * K_BYTES + hh * LK * 128, &map_k, &k_full[s], hh * 64, row);
+            int issued = early;
+            for (int j = early; j < n; ++j) {
+                if (j >= L_STAGES && !mbar_wait(&k_empty[j % L_STAGES], ((j / L_STAGES) - 1) & 1, abortp)) break;
+                load_keys(j);
                 issued = j + 1;
             }
             if (*abortp) {
@@ -210,9 +218,10 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                     if (kb > pos_r || kb < lo_r) sb[i] = 0xff800000u;
                 }
             }
-            float mx = -INFINITY;
+            float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};      // four chains side by side: a warp has its scheduler alone
 #pragma unroll
-            for (int i = 0; i < 32; ++i) mx = max3(mx, __uint_as_float(sa[i]), __uint_as_float(sb[i]));
+            for (int i = 0; i < 32; ++i) mx4[i & 3] = max3(mx4[i & 3], __uint_as_float(sa[i]), __uint_as_float(sb[i]));
+            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
             // the exponent's reference follows the row maximum lazily (attention_tcgen05.cu)
             const float m_tile = mx * a.scale_log2;                    // scale_log2 > 0
             const bool move = m_tile - m_run > L_RESCALE_STEP;         // also the first visible key (m_run = -inf)
@@ -220,7 +229,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             const float mu = m_new == -INFINITY ? 0.f : m_new;
             const float corr = move ? ex2(m_run - mu) : 1.f;           // 0 for a row that saw nothing yet
             const uint64_t scale2 = f2_pack(a.scale_log2, a.scale_log2), neg_mu2 = f2_pack(-mu, -mu);
-            uint64_t sum_a = f2_pack(0.f, 0.f), sum_b = sum_a;
+            uint64_t sum_a = f2_pack(0.f, 0.f), sum_b = sum_a, sum_c = sum_a, sum_d = sum_a;
             // a weight's two terms, hi = bf16(p) and lo = bf16(p - hi): hi over the scores' first half, lo over the second
             uint32_t hv[32], lv[32];
 #pragma unroll
@@ -229,8 +238,13 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 f2_unpack(f2_fma(f2_pack(__uint_as_float(sa[2 * i]), __uint_as_float(sa[2 * i + 1])), scale2, neg_mu2), p0, p1);
                 f2_unpack(f2_fma(f2_pack(__uint_as_float(sb[2 * i]), __uint_as_float(sb[2 * i + 1])), scale2, neg_mu2), p2, p3);
                 p0 = ex2(p0), p1 = ex2(p1), p2 = ex2(p2), p3 = ex2(p3);
-                sum_a = f2_add(sum_a, f2_pack(p0, p1));
-                sum_b = f2_add(sum_b, f2_pack(p2, p3));
+                if (i & 1) {
+                    sum_a = f2_add(sum_a, f2_pack(p0, p1));
+                    sum_b = f2_add(sum_b, f2_pack(p2, p3));
+                } else {
+                    sum_c = f2_add(sum_c, f2_pack(p0, p1));
+                    sum_d = f2_add(sum_d, f2_pack(p2, p3));
+                }
                 const uint32_t h0 = pack2(p0, p1), h1 = pack2(p2, p3);
                 hv[i] = h0;
                 hv[16 + i] = h1;
@@ -238,7 +252,7 @@ attn_latent_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 lv[16 + i] = pack2(p2 - __uint_as_float(h1 << 16), p3 - __uint_as_float(h1 & 0xffff0000u));
             }
             float l0, l1;
-            f2_unpack(f2_add(sum_a, sum_b), l0, l1);
+            f2_unpack(f2_add(f2_add(sum_a, sum_b), f2_add(sum_c, sum_d)), l0, l1);
             l_run = l_run * corr + (l0 + l1);
             m_run = m_new;
             // O holds the sum up to tile j-1 relative to the old reference: rescale this row when it moved

@@ -1492,10 +1492,10 @@ def masked_attention(ctx, q: torch.Tensor, out: torch.Tensor, k_plane: torch.Ten
     if (q.dtype == torch.bfloat16 and MASKED_TC and not FORCE_GENERIC_ATTENTION
             and attention_masked_tc_ok(q, k_plane, v_plane, nh, nkv, dk, dv)):
         few = ctx.decode_only
-        if (not few and dist_bias is None and scale > 0 and ctx.max_q_len * nh >= LATENT_TC_MIN_ROWS
-                and attention_latent_tc_ok(q, out, k_plane, v_plane, mask)):
+        if dist_bias is None and scale > 0 and attention_latent_tc_ok(q, out, k_plane, v_plane, mask):
             attention_latent_tc(q, out, k_plane, dv, block_table, ctx.seg_start, ctx.cached_len, ctx.S, ctx.max_q_len, num_pages, mask,
-                                scale, sink, ctx.err, nsplit=latent_splits(ctx.S, ctx.max_q_len * nh, mask.most_keys(ctx.max_kv_len)))
+                                scale, sink, ctx.err,
+                                nsplit=latent_splits(ctx.S, ctx.max_q_len * nh, mask.most_keys(ctx.max_kv_len), few))
             return
         ns = masked_decode_splits(ctx.S, nkv * (-(-(nh // nkv) // 16)), mask.most_keys(ctx.max_kv_len)) if few else 1
         attention_masked_bf16(q, out, k_plane, v_plane, block_table, ctx.seg_start, ctx.cached_len, ctx.S,
@@ -1505,7 +1505,8 @@ def masked_attention(ctx, q: torch.Tensor, out: torch.Tensor, k_plane: torch.Ten
                              scale, sink, ctx.err, dist_bias)
 
 
-LATENT_TC_MIN_ROWS = int(os.environ.get("PRISM_LATENT_TC_MIN_ROWS", "64"))      # (token, head) rows of a portion; fewer: 64-row mma.sync tiles
+LATENT_MIN_TILES = 8            # 64-key tiles a CTA keeps at least when a row tile's keys are shared among CTAs ...
+LATENT_MIN_TILES_DECODE = 2     # ... and in a decode step
 
 
 def attention_latent_tc_ok(q, out, k_plane, v_plane, mask: KeyMask) -> bool:
@@ -1517,11 +1518,11 @@ def attention_latent_tc_ok(q, out, k_plane, v_plane, mask: KeyMask) -> bool:
             and bool(lib().prism_attention_latent_tc_supported(dk, v_plane.shape[3], k_plane.shape[1])))
 
 
-def latent_splits(S: int, rows: int, most_keys: int, sms: Optional[int] = None) -> int:
+def latent_splits(S: int, rows: int, most_keys: int, decode: bool = False, sms: Optional[int] = None) -> int:
     """CTAs that share the key tiles of 128 rows: 1 unless the row tiles leave half of the GPU idle and the keys are many;
-    then as many as fill it (one a SM), each with at least 8 tiles of 64 keys."""
+    then as many as fill it (one a SM), each with at least ``LATENT_MIN_TILES`` (``LATENT_MIN_TILES_DECODE``) tiles."""
     ctas, tiles = S * -(-rows // 128), -(-most_keys // 64)
-    return max(1, min((sms or num_sms()) // ctas, tiles // 8, 16))
+    return max(1, min((sms or num_sms()) // ctas, tiles // (LATENT_MIN_TILES_DECODE if decode else LATENT_MIN_TILES), 64))
 
 
 def attention_latent_tc(q, out, k_plane, dv: int, block_table, seg_start, cached_len, S: int, max_q_len: int, num_pages: int,
@@ -2126,7 +2127,7 @@ moe_tensor_cores = True                                 # bf16 experts on tcgen0
 MOE_ONE_CTA_TOKENS = 16       # steps of up to this many tokens are routed and placed by one CTA in one launch (a warp a token at a time: 64 tokens take longer than the three launches)
 
 
-MOE_SHARED_TOKENS = int(os.environ.get("PRISM_MOE_SHARED_TOKENS", "64"))        # steps of up to this many tokens run a shared expert in the experts' own launches
+MOE_SHARED_TOKENS = 64        # steps of up to this many tokens run a shared expert in the experts' own launches
 
 
 def _moe_ksplit(N: int, K: int, live: int) -> int:
