@@ -218,12 +218,13 @@ gemm_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                 }
             }
             if (finish && m < N) {
-                const float b = (EPI == EPI_BF16 || EPI == EPI_F32) && bias != nullptr ? load_param(bias, bias_bf16, m) : 0.f;
+                const float b = EPI != EPI_PARTIAL && bias != nullptr ? load_param(bias, bias_bf16, m) : 0.f;
+                const float bu = EPI == EPI_SWIGLU && bias != nullptr ? load_param(bias, bias_bf16, N + m) : 0.f;
 #pragma unroll
                 for (int n = 0; n < NTOK; ++n) {
                     if (n >= M) continue;
                     if (EPI == EPI_SWIGLU) {
-                        const float g = acc[0][n], u = acc[W_TILES - 1][n];
+                        const float g = acc[0][n] + b, u = acc[W_TILES - 1][n] + bu;
                         const float a = glu_act == 1 ? 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)))
                                                      : g / (1.f + expf(-g));
                         reinterpret_cast<__nv_bfloat16*>(y)[(size_t)n * ldy + m] =
@@ -284,7 +285,7 @@ PRISM_EXPORT int prism_gemm_tcgen05_supported(int M, int N, int K) {
     return M >= 1 && M <= 64 && N >= 1 && K >= 8 && K % 8 == 0;
 }
 
-// epi: 0 bf16 (+bias), 1 float32 (+bias), 2 paired SwiGLU (W is [2N, K]; bf16 out [M, N]),
+// epi: 0 bf16 (+bias), 1 float32 (+bias), 2 paired SwiGLU (W is [2N, K], bias [2N] or null; bf16 out [M, N]),
 // 3 partial sums: y is float32 [ksplit, M, N] (ldy = N), no bias; 4: as 2 with the gate through gelu_tanh instead of silu,
 // 5: as 2 in the clamped form with `glu_limit` (common.cuh: clamped_glu).
 // ksplit > 1 with epi 0 or 1 needs a workspace `ws` of ksplit * M * N floats and `counters`, one int per

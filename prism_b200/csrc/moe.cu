@@ -26,6 +26,11 @@ __device__ __forceinline__ float moe_act(float z, int act) {
     return act == 3 ? r * r : r;                                                                      // relu squared, relu
 }
 
+// an expert's hidden value from its gate and up values; act 4: the clamped form (common.cuh: clamped_glu)
+__device__ __forceinline__ float moe_glu(float g, float u, int act, float limit) {
+    return act == 4 ? clamped_glu(g, u, limit) : moe_act(g, act) * u;
+}
+
 // One warp takes a token: scores into s [E] (shared), choice scores into c [E] (the score plus a correction per expert,
 // where one is given), the `top` largest choice scores chosen (the lower index wins a tie), counts [E] (shared or global)
 // raised by one per choice, whose old value is the choice's rank among its expert's rows.  With `groups` > 1 the experts
@@ -215,7 +220,7 @@ template <typename AT, bool DUAL, int BM, int BN, int BK, int TM, int TN>
 __global__ void __launch_bounds__((BM / TM) * (BN / TN))
 moe_gemm_kernel(const AT* __restrict__ A_in, long long lda, const AT* __restrict__ W, const int* __restrict__ offs_in,
                 const int* __restrict__ row_tok_in, const float* __restrict__ row_w_in, const int* __restrict__ row_dst_in, int E,
-                int N, int K, int scale_in, int act, void* __restrict__ out, long long ldo, int gated) {
+                int N, int K, int scale_in, int act, void* __restrict__ out, long long ldo, int gated, float limit) {
     pdl_trigger();
     pdl_wait();
     const AT* A = pdl_fresh(A_in);
@@ -317,7 +322,7 @@ moe_gemm_kernel(const AT* __restrict__ A_in, long long lda, const AT* __restrict
             if (n >= N) continue;
             if (DUAL) {
                 reinterpret_cast<AT*>(out)[(size_t)p * ldo + n] =
-                    from_float<AT>(gated ? moe_act(acc[i][j], act) * acu[i][j] : moe_act(acc[i][j], act));
+                    from_float<AT>(gated ? moe_glu(acc[i][j], acu[i][j], act, limit) : moe_act(acc[i][j], act));
             } else {
                 reinterpret_cast<float*>(out)[(size_t)row_dst[p] * ldo + n] = scale_in ? acc[i][j] : acc[i][j] * rows_w[r];
             }
@@ -325,7 +330,30 @@ moe_gemm_kernel(const AT* __restrict__ A_in, long long lda, const AT* __restrict
     }
 }
 
+// y[j T + t] <- own[t] times its weight for every choice j of a token t that names an expert from `experts` on (an identity
+// expert: its output is its input).  One CTA per (token, choice).
+__global__ void moe_identity_kernel(const float* __restrict__ own_in, const int* __restrict__ sel_e_in, const float* __restrict__ sel_w_in,
+                                    int T, int top, int W, int experts, float* __restrict__ y) {
+    pdl_trigger();
+    pdl_wait();
+    const int i = blockIdx.x;
+    if (pdl_fresh(sel_e_in)[i] < experts) return;
+    const int t = i / top, j = i - t * top;
+    const float w = pdl_fresh(sel_w_in)[i];
+    const float* own = pdl_fresh(own_in) + (size_t)t * W;
+    float* dst = y + ((size_t)j * T + t) * W;
+    for (int c = threadIdx.x; c < W; c += blockDim.x) dst[c] = own[c] * w;
+}
+
 }  // namespace prism
+
+// own [T, W] float32 contiguous; sel_e, sel_w [T, top]; y [top, T, W] float32: the planes' rows of identity experts only.
+PRISM_EXPORT int prism_moe_identity(const float* own, const int* sel_e, const float* sel_w, int T, int top, int W, int experts,
+                                    float* y, cudaStream_t stream) {
+    if (T <= 0 || W <= 0) return 0;
+    return (int)prism::launch_kernel(prism::moe_identity_kernel, dim3(T * top), dim3(W >= 512 ? 256 : 64), 0, stream, own, sel_e, sel_w,
+                                     T, top, W, experts, y);
+}
 
 // logits [T, E] float32; counts [E] int32, zero before the call; sel_e, sel_rank int32 and sel_w float32 [T, top].
 PRISM_EXPORT int prism_moe_route(const float* logits, long long logits_stride, int T, int E, int top, int softmax, int renorm,
@@ -371,11 +399,13 @@ PRISM_EXPORT int prism_moe_place(const int* counts, const int* sel_e, const floa
 }
 
 // rows = T top sorted rows.  dual 1: a [T, K], w [E, 2 N, K], out [rows, N] of dtype; dual 0: a [rows, K], w [E, N, K],
-// out [rows, N] float32 (written at row_dst).  act: 0 silu, 1 gelu_tanh, 2 relu, 3 relu squared.  gated 0 (with dual 1):
-// w [E, N, K] and out[p] = act(w a_p), an expert without a gate.
+// out [rows, N] float32 (written at row_dst).  act: 0 silu, 1 gelu_tanh, 2 relu, 3 relu squared,
+// 4 (gated experts) the clamped form with `limit`.  gated 0 (with dual 1): w [E, N, K] and out[p] = act(w a_p), an expert
+// without a gate.  With identity experts behind the E (a choice of theirs has no product) their rows are the last ones, and
+// no tile covers them.
 PRISM_EXPORT int prism_moe_gemm(const void* a, long long lda, const void* w, int dtype, const int* offs, const int* row_tok,
                                 const float* row_w, const int* row_dst, int rows, int E, int N, int K, int dual, int scale_in,
-                                int act, void* out, long long ldo, int gated, cudaStream_t stream) {
+                                int act, void* out, long long ldo, int gated, float limit, cudaStream_t stream) {
     if (rows <= 0 || N <= 0) return 0;
     if (E < 1 || K < 1) return (int)cudaErrorInvalidValue;
 #define PRISM_MG(AT, D, BM, BN, BK, TM, TN)                                                                              \
@@ -386,7 +416,7 @@ PRISM_EXPORT int prism_moe_gemm(const void* a, long long lda, const void* w, int
         dim3 grid((N + BN - 1) / BN, (unsigned)tiles);                                                                   \
         return (int)prism::launch_kernel(prism::moe_gemm_kernel<AT, D, BM, BN, BK, TM, TN>, grid,                         \
                                          dim3((BM / TM) * (BN / TN)), 0, stream, (const AT*)a, lda, (const AT*)w, offs,   \
-                                         row_tok, row_w, row_dst, E, N, K, scale_in, act, out, ldo, gated);              \
+                                         row_tok, row_w, row_dst, E, N, K, scale_in, act, out, ldo, gated, limit);       \
     } while (0)
     const bool few = rows <= 16 * E / 2 || rows <= 64;       // most experts see under a tile's worth of rows
     if (dtype == PRISM_DTYPE_BF16) {

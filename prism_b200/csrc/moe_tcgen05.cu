@@ -38,6 +38,11 @@ __device__ __forceinline__ float moe_tc_act(float z, int act) {
     return act == 3 ? r * r : r;                                                                      // relu squared, relu
 }
 
+// an expert's hidden value from its gate and up values; act 4: the clamped form (common.cuh: clamped_glu)
+__device__ __forceinline__ float moe_tc_glu(float g, float u, int act, float limit) {
+    return act == 4 ? clamped_glu(g, u, limit) : moe_tc_act(g, act) * u;
+}
+
 template <int NTOK, bool DUAL> struct MoeCfg {
     static constexpr int W_TILES = DUAL ? 2 : 1;
     static constexpr int STAGE_BYTES = W_TILES * MOE_TILE_M * TILE_K * 2 + NTOK * TILE_K * 2;
@@ -64,7 +69,7 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                 const int* __restrict__ offs_in, const int* __restrict__ counts_in, const int* __restrict__ row_dst_in,
                 const float* __restrict__ row_w_in, int E, int N, int K, int act, void* __restrict__ y, long long ldy,
                 int* err, const __grid_constant__ CUtensorMap map_sw, const __grid_constant__ CUtensorMap map_sx,
-                const MoeShared sh, float* __restrict__ ws, int* __restrict__ counters) {
+                const MoeShared sh, float* __restrict__ ws, int* __restrict__ counters, float limit) {
     using C = MoeCfg<NTOK, DUAL>;
     constexpr int W_TILES = C::W_TILES;
     constexpr int STAGES = C::STAGES;
@@ -235,7 +240,7 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                         reinterpret_cast<float*>(y)[(size_t)p * ldy + m] = acc[0][n];
                     } else if (DUAL) {
                         reinterpret_cast<__nv_bfloat16*>(y)[(size_t)p * ldy + m] =
-                            __float2bfloat16_rn(moe_tc_act(acc[0][n], act) * acc[W_TILES - 1][n]);
+                            __float2bfloat16_rn(moe_tc_glu(acc[0][n], acc[W_TILES - 1][n], act, limit));
                     } else if (row_dst == nullptr) {          // an expert without a gate: its hidden layer, act(up a_p)
                         reinterpret_cast<__nv_bfloat16*>(y)[(size_t)p * ldy + m] = __float2bfloat16_rn(moe_tc_act(acc[0][n], act));
                     } else {
@@ -259,7 +264,7 @@ template <int NTOK, bool DUAL>
 int moe_launch(const void* x, long long ldx, long long x_rows, const void* W, const int* offs, const int* counts,
                const int* row_dst, const float* row_w, int token_tiles, int E, int N, int K, int act, void* y,
                long long ldy, int* err, const void* sw, const void* sx, long long ldsx, const MoeShared& sh, int ksplit, float* ws,
-               int* counters, cudaStream_t stream) {
+               int* counters, float limit, cudaStream_t stream) {
     using C = MoeCfg<NTOK, DUAL>;
     CUtensorMap mw, mx;
     int rc = make_map(&mw, W, (long long)E * (DUAL ? 2 : 1) * N, K, K, MOE_TILE_M);
@@ -278,22 +283,34 @@ int moe_launch(const void* x, long long ldx, long long x_rows, const void* W, co
     const int widest = sh.tiles > 0 && sh.N > N ? sh.N : N;
     dim3 grid((widest + MOE_TILE_M - 1) / MOE_TILE_M, token_tiles + sh.tiles, ksplit);
     return (int)launch_kernel(kern, grid, dim3(MOE_THREADS), C::SMEM, stream, mw, mx, offs, counts, row_dst, row_w, E, N, K, act,
-                              y, ldy, err, msw, msx, sh, ws, counters);
+                              y, ldy, err, msw, msx, sh, ws, counters, limit);
 }
 
 // One block per (token, choice): its row of x, times its weight (scale_in), rounded to bf16, at its padded place;
-// and where the row's result goes.
+// and where the row's result goes.  A choice of an expert from `experts` on (an identity expert: its output is its input)
+// has no row there: its result, own[t] times the weight, goes to its place of y at once.
 __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x_in, long long ldx, const int* __restrict__ offs_in,
                                   const int* __restrict__ sel_e_in, const float* __restrict__ sel_w_in,
-                                  const int* __restrict__ sel_rank_in, int T, int top, int W, int scale_in,
+                                  const int* __restrict__ sel_rank_in, int T, int top, int W, int scale_in, int experts,
+                                  const float* __restrict__ own_in, float* __restrict__ y,
                                   __nv_bfloat16* __restrict__ xs, int* __restrict__ row_dst, float* __restrict__ row_w) {
     pdl_trigger();
     pdl_wait();
     const __nv_bfloat16* x = pdl_fresh(x_in);
     const int i = blockIdx.x;
     const int t = i / top, j = i - t * top;
-    const int p = pdl_fresh(offs_in)[pdl_fresh(sel_e_in)[i]] + pdl_fresh(sel_rank_in)[i];
+    const int e = pdl_fresh(sel_e_in)[i];
     const float w = pdl_fresh(sel_w_in)[i];
+    if (e >= experts) {
+        const float* own = pdl_fresh(own_in) + (size_t)t * W;
+        float* dst = y + ((size_t)j * T + t) * W;
+        for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {          // W is a multiple of 8 here
+            const float4 v = *reinterpret_cast<const float4*>(own + c);
+            *reinterpret_cast<float4*>(dst + c) = make_float4(v.x * w, v.y * w, v.z * w, v.w * w);
+        }
+        return;
+    }
+    const int p = pdl_fresh(offs_in)[e] + pdl_fresh(sel_rank_in)[i];
     if (threadIdx.x == 0) {
         row_dst[p] = j * T + t;
         row_w[p] = w;
@@ -313,16 +330,19 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x_in, long l
 PRISM_EXPORT int prism_moe_tcgen05_supported(int W, int F) { return W >= 8 && F >= 8 && W % 8 == 0 && F % 8 == 0; }
 
 // x [T, W] bf16 -> xs [padded rows, W] bf16 (row of (t, j) at offs[expert] + rank), row_dst and row_w at the same place.
-// offs: the padded offsets that prism_moe_place made with pad = the token tile.
+// offs: the padded offsets that prism_moe_place made with pad = the token tile.  Experts from `experts` on are identity
+// experts: own [T, W] float32 (contiguous) times the weight goes to y [top, T, W] float32 at the choice's place.
 PRISM_EXPORT int prism_moe_gather(const void* x, long long ldx, const int* offs, const int* sel_e, const float* sel_w,
-                                  const int* sel_rank, int T, int top, int W, int scale_in, void* xs, int* row_dst,
-                                  float* row_w, cudaStream_t stream) {
+                                  const int* sel_rank, int T, int top, int W, int scale_in, int experts, const float* own, float* y,
+                                  void* xs, int* row_dst, float* row_w, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (W % 8 || ((uintptr_t)own & 15) || ((uintptr_t)y & 15)) return (int)cudaErrorInvalidValue;
     return (int)prism::launch_kernel(prism::tc::moe_gather_kernel, dim3(T * top), dim3(W >= 2048 ? 256 : 128), 0, stream,
-                                     (const __nv_bfloat16*)x, ldx, offs, sel_e, sel_w, sel_rank, T, top, W, scale_in,
+                                     (const __nv_bfloat16*)x, ldx, offs, sel_e, sel_w, sel_rank, T, top, W, scale_in, experts, own, y,
                                      (__nv_bfloat16*)xs, row_dst, row_w);
 }
 
+// limit: of the clamped form (act 4).
 // a [x_rows, K] bf16 in padded order (x_rows = token_tiles * ntok); w [E, (2) N, K] bf16 contiguous.
 // dual 1: out [x_rows, N] bf16 (row stride ldo), out[p] = act(gate a_p) * (up a_p).
 // dual 0: out float32, out[row_dst[p]] = w a_p (times row_w[p] if row_w is given); row_dst null: out [x_rows, N] bf16,
@@ -335,7 +355,7 @@ PRISM_EXPORT int prism_moe_gemm_tcgen05(const void* a, long long lda, const void
                                         const int* row_dst, const float* row_w, int ntok, int token_tiles, int E, int N,
                                         int K, int dual, int act, void* out, long long ldo, int* err, const void* sw,
                                         const void* sx, long long ldsx, int shared_rows, int sN, int sK, void* sy, long long ldsy,
-                                        int ksplit, float* ws, int* counters, cudaStream_t stream) {
+                                        int ksplit, float* ws, int* counters, float limit, cudaStream_t stream) {
     using namespace prism::tc;
     if (token_tiles <= 0 || N <= 0) return 0;
     if (E < 1 || K < 8 || K % 8 || lda % 8 || ((uintptr_t)a & 15) || ((uintptr_t)w & 15) || token_tiles > 65535 ||
@@ -350,7 +370,7 @@ PRISM_EXPORT int prism_moe_gemm_tcgen05(const void* a, long long lda, const void
     sh.rows = shared_rows; sh.N = sN; sh.K = sK; sh.y = sy; sh.ldy = ldsy;
     if (token_tiles + sh.tiles > 65535) return (int)cudaErrorInvalidValue;
     const long long x_rows = (long long)token_tiles * ntok;
-#define ARGS a, lda, x_rows, w, offs, counts, row_dst, row_w, token_tiles, E, N, K, act, out, ldo, err, sw, sx, ldsx, sh, ksplit, ws, counters, stream
+#define ARGS a, lda, x_rows, w, offs, counts, row_dst, row_w, token_tiles, E, N, K, act, out, ldo, err, sw, sx, ldsx, sh, ksplit, ws, counters, limit, stream
     if (dual) return ntok == 16 ? moe_launch<16, true>(ARGS) : ntok == 32 ? moe_launch<32, true>(ARGS) : moe_launch<64, true>(ARGS);
     return ntok == 16 ? moe_launch<16, false>(ARGS) : ntok == 32 ? moe_launch<32, false>(ARGS) : moe_launch<64, false>(ARGS);
 #undef ARGS

@@ -2,7 +2,7 @@
 // rotate it.  From the float32 result of the input projection, per token:
 //   q_h <- rotate(q_h / sqrt(mean(q_h^2) + eps) * wq)      into q_out [T, nh, dk] (compute dtype)
 //   k_g <- rotate(k_g / sqrt(mean(k_g^2) + eps) * wk)      into the key plane, at the token's slot
-//   v_g                                                    into the value plane, at the token's slot
+//   v_g times a constant                                   into the value plane, at the token's slot
 // wq, wk: one weight vector of dk entries each, shared by the heads (null: no norm).  With `whole` the norm runs
 // over the whole projection instead, all heads of q (of k) at once, q <- q / sqrt(mean over nh dk (q^2) + eps) * wq
 // with wq of nh dk entries (wk: nkv dk).  The rotation turns the
@@ -25,7 +25,7 @@ __global__ void qk_norm_rope_store_kernel(const float* __restrict__ q_in, const 
                                           const int* __restrict__ block_table, int bt_width,
                                           const int* __restrict__ positions, const int* __restrict__ tok_seg, int nh, int nkv,
                                           int dk, int dv, int page_size, int num_pages, int max_pos, int* err, int whole,
-                                          int halves) {
+                                          int halves, float v_scale) {
     __shared__ float red[33];
     pdl_trigger();
     pdl_wait();
@@ -57,7 +57,7 @@ __global__ void qk_norm_rope_store_kernel(const float* __restrict__ q_in, const 
     const int lane = threadIdx.x & 31;
     const int unit = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);      // q heads, k heads, then the values
     if (unit == nh + nkv && page_ok && v_plane != nullptr)
-        for (int c = lane; c < nkv * dv; c += 32) v_plane[slot * nkv * dv + c] = from_float<T>(v[c]);
+        for (int c = lane; c < nkv * dv; c += 32) v_plane[slot * nkv * dv + c] = from_float<T>(v[c] * v_scale);
     const int half = rot >> 1;
     for (int hh = unit; hh < nh + nkv; hh += nh + nkv) {
         const bool is_q = hh < nh;
@@ -99,7 +99,7 @@ PRISM_EXPORT int prism_qk_norm_rope_store(const float* q, const float* k, const 
                                           void* q_out, void* k_plane, void* v_plane, int dtype, const int* block_table,
                                           int bt_width, const int* positions, const int* tok_seg, int T, int nh, int nkv, int dk,
                                           int dv, int page_size, int num_pages, int max_pos, int* err, int whole, int halves,
-                                          cudaStream_t stream) {
+                                          float v_scale, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (rot < 0 || rot > dk || rot % 2 || (rot > 0 && freq == nullptr) || nh < 1 || nkv < 1 || dk < 1 || dv < 1)
         return (int)cudaErrorInvalidValue;
@@ -112,8 +112,9 @@ PRISM_EXPORT int prism_qk_norm_rope_store(const float* q, const float* k, const 
         return (int)prism::launch_kernel(prism::qk_norm_rope_store_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, q, k,
                                          v, ps, wq, qb, wk, kb, eps, freq, rot, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_plane,
                                          (__nv_bfloat16*)v_plane, block_table, bt_width, positions, tok_seg, nh, nkv, dk, dv,
-                                         page_size, num_pages, max_pos, err, whole, halves);
+                                         page_size, num_pages, max_pos, err, whole, halves, v_scale);
     return (int)prism::launch_kernel(prism::qk_norm_rope_store_kernel<float>, grid, dim3(threads), 0, stream, q, k, v, ps, wq,
                                      qb, wk, kb, eps, freq, rot, (float*)q_out, (float*)k_plane, (float*)v_plane, block_table,
-                                     bt_width, positions, tok_seg, nh, nkv, dk, dv, page_size, num_pages, max_pos, err, whole, halves);
+                                     bt_width, positions, tok_seg, nh, nkv, dk, dv, page_size, num_pages, max_pos, err, whole, halves,
+                                     v_scale);
 }

@@ -12,6 +12,10 @@
 //       S <- diag(w) S - c (e^T S) + k v^T;   o = S^T r         (decay and removal both read the state before the token)
 //   decayed sum with one constant decay per head (SCAN_RETAIN):
 //       S <- g S + k v^T;   o = S^T q                           (the read-out sees this token's write)
+//   decayed sum with a step size per head and token (SCAN_TOKEN), dt and g = exp(-rate dt) scalars, D a constant per head:
+//       S <- g S + dt k v^T;   o = S^T q + D v
+//   decayed sum with one decay per key channel and token (SCAN_GATED), w a vector over the key channels:
+//       S <- diag(w) S + k v^T;   o = S^T q
 //
 // Everything that enters the recurrence is float32: the kernels here read the float32 results of the input
 // projections, and the state never leaves float32.  A request's state lives in its slot between steps, so
@@ -26,7 +30,9 @@
 //     convolution's tail; with one row, the previous token's input of a token-shift mix);
 //   * prism_shift_mix        x + (x_prev - x) mu_s for several mu at once (x_prev of a step's first token comes
 //     from the state);
-//   * prism_headnorm_gate    o / rms(o) per head, times a weight, times silu(gate), times a constant.
+//   * prism_headnorm_gate    o / rms(o) per head, times a weight, times silu(gate), times a constant;
+//   * prism_part_norm_gate   the same over equal parts of the concatenated heads, the gate before or after the norm;
+//   * prism_step_sizes       softplus(z + bias) and the decay exp(-exp(a_log) times it) per head and token.
 #include "mma_helpers.cuh"
 
 #define PRISM_SCAN_DELTA 0
@@ -34,6 +40,8 @@
 #define PRISM_SCAN_CHANNEL 2
 #define PRISM_SCAN_GENERAL 3
 #define PRISM_SCAN_RETAIN 4
+#define PRISM_SCAN_TOKEN 5
+#define PRISM_SCAN_GATED 6
 
 namespace prism {
 
@@ -155,6 +163,8 @@ __global__ void decay_from_exponent_kernel(float* __restrict__ w, long long ws, 
 //   PRISM_LR_SOFTPLUS  exp(-exp(alog[n / per]) softplus(z))  a per-channel decay with one rate per group of `per` channels
 //   PRISM_LR_SIGMOID   sigmoid(z)                            a gate
 //   PRISM_LR_EXPSIG    exp(-rate sigmoid(z))                 a per-channel decay kept inside (exp(-rate), 1), rate a constant
+//   PRISM_LR_SIGPOW    sigmoid(z)^rate                       a per-channel decay near one for a small constant rate
+//   PRISM_LR_LOGSIGPOW rate log sigmoid(z)                   its logarithm
 // b may be null.  A CTA takes 128 channels and sixteen tokens, so that every weight it reads serves sixteen tokens
 // (whose inner values sit side by side in shared memory: four 128-bit loads per weight); w2t is the second matrix
 // transposed, [R, N], so that neighbouring threads read neighbouring floats.
@@ -162,6 +172,8 @@ __global__ void decay_from_exponent_kernel(float* __restrict__ w, long long ws, 
 #define PRISM_LR_SOFTPLUS 1
 #define PRISM_LR_SIGMOID 2
 #define PRISM_LR_EXPSIG 3
+#define PRISM_LR_SIGPOW 4
+#define PRISM_LR_LOGSIGPOW 5
 constexpr int LRD_TOK = 16;
 __global__ void lowrank_decay_kernel(const float* __restrict__ low_in, long long ls, int R, const float* __restrict__ w2t,
                                      const void* __restrict__ w0, int w0_bf16, int N, int T, float* __restrict__ out,
@@ -201,7 +213,9 @@ __global__ void lowrank_decay_kernel(const float* __restrict__ low_in, long long
             const float z = acc[j] + b;
             out[(size_t)(t0 + j) * os + n] = epi == PRISM_LR_EXPEXP ? expf(-expf(z))
                                              : epi == PRISM_LR_SOFTPLUS ? expf(-rate * softplus_f(z))
-                                             : epi == PRISM_LR_EXPSIG ? expf(-crate * sigmoid_f(z)) : sigmoid_f(z);
+                                             : epi == PRISM_LR_EXPSIG ? expf(-crate * sigmoid_f(z))
+                                             : epi == PRISM_LR_SIGPOW ? expf(-crate * softplus_f(-z))
+                                             : epi == PRISM_LR_LOGSIGPOW ? -crate * softplus_f(-z) : sigmoid_f(z);
         }
 }
 
@@ -259,6 +273,84 @@ __global__ void headnorm_gate_kernel(const float* __restrict__ o_in, const float
     }
 }
 
+// bg[t][h] = softplus(z[t][h] + bias[h]) (a step size) and bg[t][H + h] = exp(-exp(a_log[h]) times it) (the decay it makes).
+__global__ void step_sizes_kernel(const float* __restrict__ z_in, long long zs, const void* __restrict__ bias, int bias_bf16,
+                                  const void* __restrict__ a_log, int a_log_bf16, int T, int H, float* __restrict__ bg) {
+    pdl_trigger();
+    pdl_wait();
+    const float* z = pdl_fresh(z_in);
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < (long long)T * H; i += (long long)gridDim.x * blockDim.x) {
+        const int t = (int)(i / H), h = (int)(i - (long long)t * H);
+        const float dt = softplus_f(z[(size_t)t * zs + h] + load_param(bias, bias_bf16, h));
+        bg[(size_t)t * 2 * H + h] = dt;
+        bg[(size_t)t * 2 * H + H + h] = expf(-expf(load_param(a_log, a_log_bf16, h)) * dt);
+    }
+}
+
+// Rows of `parts` equal parts of w entries each, normed part by part:
+//   before:  y = x * act(gate);  out = y / sqrt(mean_part(y^2) + eps) * weight * scale
+//   after:   out = x / sqrt(mean_part(x^2) + eps) * weight * act(gate) * scale
+// x [T, parts w] float32 contiguous, gate float32 and out with row strides of their own, weight [parts w]; act silu, or
+// sigmoid.  One CTA per (token, part); VEC 4 reads and writes four neighbouring entries at a time.
+template <typename T, int VEC>
+__global__ void part_norm_gate_kernel(const float* __restrict__ x_in, const float* __restrict__ gate_in, long long gs,
+                                      const void* __restrict__ weight, int weight_bf16, float eps, float scale, int parts, int w,
+                                      int before, int sigmoid_act, T* __restrict__ out, long long os) {
+    extern __shared__ __align__(16) float row[];       // [w]
+    __shared__ float scratch[33];
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x, p = blockIdx.y;
+    const float* x = pdl_fresh(x_in) + ((size_t)t * parts + p) * w;
+    const float* gate = pdl_fresh(gate_in) + (size_t)t * gs + (size_t)p * w;
+    T* o = out + (size_t)t * os + (size_t)p * w;
+    float ss = 0.f;
+    for (int c = threadIdx.x * VEC; c < w; c += blockDim.x * VEC) {
+        float v[VEC], g[VEC];
+        if (VEC == 4) {
+            const float4 a = *reinterpret_cast<const float4*>(x + c);
+            v[0] = a.x; v[1 % VEC] = a.y; v[2 % VEC] = a.z; v[3 % VEC] = a.w;
+            if (before) {
+                const float4 b = *reinterpret_cast<const float4*>(gate + c);
+                g[0] = b.x; g[1 % VEC] = b.y; g[2 % VEC] = b.z; g[3 % VEC] = b.w;
+            }
+        } else {
+            v[0] = x[c];
+            if (before) g[0] = gate[c];
+        }
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+            if (before) v[k] *= sigmoid_act ? sigmoid_f(g[k]) : silu_f(g[k]);
+            ss += v[k] * v[k];
+            row[c + k] = v[k];
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = scale / sqrtf(ss / (float)w + eps);
+    for (int c = threadIdx.x * VEC; c < w; c += blockDim.x * VEC) {
+        float g[VEC], y[VEC];
+        if (!before) {
+            if (VEC == 4) {
+                const float4 b = *reinterpret_cast<const float4*>(gate + c);
+                g[0] = b.x; g[1 % VEC] = b.y; g[2 % VEC] = b.z; g[3 % VEC] = b.w;
+            } else {
+                g[0] = gate[c];
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+            y[k] = row[c + k] * inv * load_param(weight, weight_bf16, (size_t)p * w + c + k);
+            if (!before) y[k] *= sigmoid_act ? sigmoid_f(g[k]) : silu_f(g[k]);
+        }
+        if (VEC == 4 && sizeof(T) == 2) {
+            *reinterpret_cast<uint2*>(o + c) = make_uint2(pack_bf16(y[0], y[1 % VEC]), pack_bf16(y[2 % VEC], y[3 % VEC]));
+        } else {
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) o[c + k] = from_float<T>(y[k]);
+        }
+    }
+}
+
 // ---------------------------------------------------------------------------------------------------------
 // The scan.  grid (heads, segments, column blocks); the L threads of a column are neighbouring lanes of a warp,
 // each owns R rows of that column of S in registers - quads of four neighbouring rows, quad part + L m - and
@@ -273,6 +365,8 @@ __global__ void headnorm_gate_kernel(const float* __restrict__ o_in, const float
 //   SCAN_CHANNEL: q, k, v as for SCAN_DELTA; the decay itself in ww [T, H dk] (row stride ws); bg [T, H]: beta.
 //   SCAN_GENERAL: r, k, v as for SCAN_BONUS; the decay itself in ww; ex [T, 2 H dk]: the unit key e at h dk, c at (H + h) dk.
 //   SCAN_RETAIN: q, k, v as for SCAN_BONUS; the decay of head h in w0[h].
+//   SCAN_TOKEN: q, k, v as for SCAN_DELTA; bg [T, 2 H]: dt | g; D of head h in w0[h] (null: no such term).
+//   SCAN_GATED: q, k, v as for SCAN_BONUS; the decay itself in ww [T, H dk].
 // ---------------------------------------------------------------------------------------------------------
 struct ScanArgs {
     const float* x;          // q | k | v (or r | k | v) rows
@@ -314,7 +408,7 @@ template <int L> __device__ __forceinline__ float column_sum(float v) {
 
 // vectors over the key channels that a token brings: q (or r) and k, a decay per channel, a unit key and what it removes
 __host__ __device__ constexpr int scan_vectors(int mode) {
-    return (mode == PRISM_SCAN_DELTA || mode == PRISM_SCAN_RETAIN) ? 2 : (mode == PRISM_SCAN_GENERAL ? 5 : 3);
+    return (mode == PRISM_SCAN_DELTA || mode == PRISM_SCAN_RETAIN || mode == PRISM_SCAN_TOKEN) ? 2 : (mode == PRISM_SCAN_GENERAL ? 5 : 3);
 }
 
 template <int MODE, int R, int L>
@@ -370,7 +464,7 @@ __global__ void scan_kernel(const ScanArgs a) {
         float* dst0 = sm + (size_t)buf * TB * per_tok;
         const int unit = a.vec ? 4 : 1;
         const int nk = (dk + unit - 1) / unit, nc = (ncols + unit - 1) / unit;     // pieces per vector
-        const size_t head_q = (size_t)((MODE == PRISM_SCAN_DELTA || MODE == PRISM_SCAN_CHANNEL) ? kvh : h) * dk;
+        const size_t head_q = (size_t)((MODE == PRISM_SCAN_DELTA || MODE == PRISM_SCAN_CHANNEL || MODE == PRISM_SCAN_TOKEN) ? kvh : h) * dk;
         for (int tt = 0; tt < nb; ++tt) {
             const size_t t = (size_t)(s0 + b0 + tt);
             const float* xr = x + t * a.xs;
@@ -386,7 +480,7 @@ __global__ void scan_kernel(const ScanArgs a) {
             }
             for (int c = lane; c < nc; c += 32)
                 cp_async_f(dst + NV * dkp + c * unit, xr + a.vo + (size_t)h * dv + col0 + c * unit, unit);
-            if (MODE == PRISM_SCAN_DELTA && lane < 2)                                // beta, then g
+            if ((MODE == PRISM_SCAN_DELTA || MODE == PRISM_SCAN_TOKEN) && lane < 2)  // beta (or dt), then g
                 cp_async_f(dst + NV * dkp + a.colsp + lane, bg + t * 2 * a.H + (size_t)lane * a.H + h, 1);
             if (MODE == PRISM_SCAN_CHANNEL && lane == 0)                             // beta
                 cp_async_f(dst + NV * dkp + a.colsp, bg + t * a.H + h, 1);
@@ -431,6 +525,7 @@ __global__ void scan_kernel(const ScanArgs a) {
     }
     __syncthreads();
     const float keep = MODE == PRISM_SCAN_RETAIN ? load_param(a.w0, a.w0_bf16, h) : 0.f;      // the head's constant decay
+    const float skip = MODE == PRISM_SCAN_TOKEN && a.w0 != nullptr ? load_param(a.w0, a.w0_bf16, h) : 0.f;
 
     int buf = 0;
     for (int b0 = 0; b0 < qlen; b0 += TB, buf = buf + 1 == NBUF ? 0 : buf + 1) {
@@ -544,16 +639,35 @@ __global__ void scan_kernel(const ScanArgs a) {
                     o2 += S[4 * m + 2] * rr.z;
                     o3 += S[4 * m + 3] * rr.w;
                 }
-            } else if (MODE == PRISM_SCAN_RETAIN) {
-                const float v = f2[dkp + lc];
+            } else if (MODE == PRISM_SCAN_RETAIN || MODE == PRISM_SCAN_TOKEN) {
+                const float* vv = f2 + dkp;
+                const float g = MODE == PRISM_SCAN_TOKEN ? vv[a.colsp + 1] : keep;
+                const float v = MODE == PRISM_SCAN_TOKEN ? vv[a.colsp] * vv[lc] : vv[lc];
 #pragma unroll
                 for (int m = 0; m < Q; ++m) {
                     const int i = 4 * (part + L * m);
                     const float4 qq = *reinterpret_cast<const float4*>(f1 + i), kk = *reinterpret_cast<const float4*>(f2 + i);
-                    S[4 * m] = keep * S[4 * m] + kk.x * v;
-                    S[4 * m + 1] = keep * S[4 * m + 1] + kk.y * v;
-                    S[4 * m + 2] = keep * S[4 * m + 2] + kk.z * v;
-                    S[4 * m + 3] = keep * S[4 * m + 3] + kk.w * v;
+                    S[4 * m] = g * S[4 * m] + kk.x * v;
+                    S[4 * m + 1] = g * S[4 * m + 1] + kk.y * v;
+                    S[4 * m + 2] = g * S[4 * m + 2] + kk.z * v;
+                    S[4 * m + 3] = g * S[4 * m + 3] + kk.w * v;
+                    o0 += S[4 * m] * qq.x;
+                    o1 += S[4 * m + 1] * qq.y;
+                    o2 += S[4 * m + 2] * qq.z;
+                    o3 += S[4 * m + 3] * qq.w;
+                }
+            } else if (MODE == PRISM_SCAN_GATED) {
+                const float* wd = f2 + dkp;
+                const float v = wd[dkp + lc];
+#pragma unroll
+                for (int m = 0; m < Q; ++m) {
+                    const int i = 4 * (part + L * m);
+                    const float4 qq = *reinterpret_cast<const float4*>(f1 + i), kk = *reinterpret_cast<const float4*>(f2 + i);
+                    const float4 w4 = *reinterpret_cast<const float4*>(wd + i);
+                    S[4 * m] = w4.x * S[4 * m] + kk.x * v;
+                    S[4 * m + 1] = w4.y * S[4 * m + 1] + kk.y * v;
+                    S[4 * m + 2] = w4.z * S[4 * m + 2] + kk.z * v;
+                    S[4 * m + 3] = w4.w * S[4 * m + 3] + kk.w * v;
                     o0 += S[4 * m] * qq.x;
                     o1 += S[4 * m + 1] * qq.y;
                     o2 += S[4 * m + 2] * qq.z;
@@ -580,6 +694,7 @@ __global__ void scan_kernel(const ScanArgs a) {
             }
             float o = (o0 + o1) + (o2 + o3);
             o = column_sum<L>(o);
+            if (MODE == PRISM_SCAN_TOKEN) o += skip * f2[dkp + lc];
             if (live && part == 0) a.out[((size_t)(s0 + b0 + tt) * a.H + h) * dv + col] = o;
         }
         __syncthreads();                               // the next block has landed, and this buffer is free
@@ -685,6 +800,45 @@ PRISM_EXPORT int prism_unit_removal(const float* k, const float* a, long long ps
                                      stream, k, a, ps, ab, ab_dtype == PRISM_DTYPE_BF16, unit_eps, T, H, dk, ex);
 }
 
+// z [T, H] float32 (row stride zs); bias, a_log [H]; bg [T, 2 H] float32 out.
+PRISM_EXPORT int prism_step_sizes(const float* z, long long zs, const void* bias, int bias_dtype, const void* a_log, int a_log_dtype,
+                                  int T, int H, float* bg, cudaStream_t stream) {
+    if (T <= 0 || H <= 0) return 0;
+    const long long blocks = ((long long)T * H + 255) / 256;
+    return (int)prism::launch_kernel(prism::step_sizes_kernel, dim3((unsigned)(blocks < 1184 ? blocks : 1184)), dim3(256), 0, stream, z, zs,
+                                     bias, bias_dtype == PRISM_DTYPE_BF16, a_log, a_log_dtype == PRISM_DTYPE_BF16, T, H, bg);
+}
+
+// x [T, parts * w] float32 contiguous; gate [T, parts * w] float32 (row stride gs); weight [parts * w]; out [T, parts * w] of
+// out_dtype (row stride os); before 1: the gate multiplies before the norm, 0: after it; sigmoid_act 1: sigmoid, 0: silu.
+PRISM_EXPORT int prism_part_norm_gate(const float* x, const float* gate, long long gs, const void* weight, int weight_dtype, float eps,
+                                      float scale, int T, int parts, int w, int before, int sigmoid_act, void* out, int out_dtype,
+                                      long long os, cudaStream_t stream) {
+    using namespace prism;
+    if (T <= 0 || parts <= 0 || w <= 0) return 0;
+    const size_t smem = (size_t)w * sizeof(float);
+    if (parts > 65535 || smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+    const bool vec = w % 4 == 0 && gs % 4 == 0 && os % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)gate % 16 == 0 &&
+                     (uintptr_t)out % (out_dtype == PRISM_DTYPE_BF16 ? 8 : 16) == 0;
+    const int per = vec ? w / 4 : w;
+    const int threads = per >= 1024 ? 512 : (per >= 256 ? 256 : (per >= 128 ? 128 : (per >= 64 ? 64 : 32)));
+    const int wb = weight_dtype == PRISM_DTYPE_BF16;
+#define PRISM_PN(TT, V)                                                                                                   \
+    do {                                                                                                                  \
+        auto kern = part_norm_gate_kernel<TT, V>;                                                                         \
+        if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
+        return (int)launch_kernel(kern, dim3(T, parts), dim3(threads), smem, stream, x, gate, gs, weight, wb, eps, scale, \
+                                  parts, w, before, sigmoid_act, (TT*)out, os);                                           \
+    } while (0)
+    if (out_dtype == PRISM_DTYPE_BF16) {
+        if (vec) PRISM_PN(__nv_bfloat16, 4);
+        PRISM_PN(__nv_bfloat16, 1);
+    }
+    if (vec) PRISM_PN(float, 4);
+    PRISM_PN(float, 1);
+#undef PRISM_PN
+}
+
 PRISM_EXPORT int prism_headnorm_gate(const float* o, const float* gate, long long gate_stride, const void* weight,
                                      int weight_dtype, int per_head_weight, float eps, float scale, int T, int H, int dv,
                                      void* out, int out_dtype, long long out_stride, int gate_sigmoid, cudaStream_t stream) {
@@ -720,6 +874,7 @@ PRISM_EXPORT int prism_recurrent_scan(int mode, const float* x, long long x_stri
     a.ex = ex; a.es = ex_stride;
     if (mode == PRISM_SCAN_RETAIN && (w0 == nullptr || rep != 1)) return (int)cudaErrorInvalidValue;
     if (mode == PRISM_SCAN_GENERAL && (ex == nullptr || ww == nullptr || rep != 1)) return (int)cudaErrorInvalidValue;
+    if ((mode == PRISM_SCAN_TOKEN && bg == nullptr) || (mode == PRISM_SCAN_GATED && (ww == nullptr || rep != 1))) return (int)cudaErrorInvalidValue;
     // A token's work is one chain (dot product, shuffles, update, dot product, shuffles), so a CTA is latency
     // bound: eight threads a column, four warps of them side by side, and as many CTAs as there are column blocks.
     const int R = dk <= 32 ? 4 : (dk <= 64 ? 8 : (dk <= 128 ? 16 : 32));
@@ -759,6 +914,8 @@ PRISM_EXPORT int prism_recurrent_scan(int mode, const float* x, long long x_stri
     if (mode == PRISM_SCAN_CHANNEL) PRISM_SCAN(PRISM_SCAN_CHANNEL);
     if (mode == PRISM_SCAN_GENERAL) PRISM_SCAN(PRISM_SCAN_GENERAL);
     if (mode == PRISM_SCAN_RETAIN) PRISM_SCAN(PRISM_SCAN_RETAIN);
+    if (mode == PRISM_SCAN_TOKEN) PRISM_SCAN(PRISM_SCAN_TOKEN);
+    if (mode == PRISM_SCAN_GATED) PRISM_SCAN(PRISM_SCAN_GATED);
 #undef PRISM_SCAN
     return (int)cudaErrorInvalidValue;
 }

@@ -19,7 +19,8 @@ __device__ __forceinline__ float rg_gelu_tanh(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
-// out[t][c] = bias[c] + sum_j taps[c][K-1-j] x[t-j][c] (+ x[t][c] with add_input: a convolution beside a skip path);
+// out[t][c] = bias[c] + sum_j taps[c][K-1-j] x[t-j][c] (+ x[t][c] with add_input: a convolution beside a skip path), with
+// `silu` through silu;
 // x [T, *] float32 with row stride xs; tail [slots, K-1, C]; out float32 or the compute dtype (rounded once).
 // taps_t (or null): the same taps as float32 [K, C], which the vector path reads 128 bits at a time.
 // One CTA per token: it looks up the token's segment, place and slot once, and its threads walk the channels VEC at a
@@ -29,7 +30,7 @@ __global__ void causal_conv_kernel(const float* __restrict__ x_in, long long xs,
                                    const void* __restrict__ bias, int bias_bf16, int K, int C, float* tail,
                                    const int* __restrict__ tok_seg, const int* __restrict__ seg_start,
                                    const int* __restrict__ slots, TO* __restrict__ out, long long os, int move_tail,
-                                   int add_input, const float* __restrict__ taps_t) {
+                                   int add_input, const float* __restrict__ taps_t, int silu) {
     pdl_trigger();
     const int t = blockIdx.x, seg = tok_seg[t];        // the step's descriptor is complete before the step's first kernel
     const int i = t - seg_start[seg];
@@ -67,7 +68,10 @@ __global__ void causal_conv_kernel(const float* __restrict__ x_in, long long xs,
             }
         }
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) out[(size_t)t * os + c0 + v] = from_float<TO>(add_input ? acc[v] + cur[v] : acc[v]);
+        for (int v = 0; v < VEC; ++v) {
+            const float y = add_input ? acc[v] + cur[v] : acc[v];
+            out[(size_t)t * os + c0 + v] = from_float<TO>(silu ? y * rg_sigmoid(y) : y);
+        }
         if (move_tail && K > 1) {          // one token per request: this thread is the only reader of its channels' tail
 #pragma unroll
             for (int v = 0; v < VEC; ++v) {
@@ -90,7 +94,7 @@ template <typename TO>
 __global__ void causal_conv_tile_kernel(const float* __restrict__ x_in, long long xs, const float* __restrict__ taps_t,
                                         const void* __restrict__ bias, int bias_bf16, int K, int C, const float* tail,
                                         const int* __restrict__ tok_seg, const int* __restrict__ seg_start,
-                                        const int* __restrict__ slots, TO* __restrict__ out, long long os, int add_input, int T) {
+                                        const int* __restrict__ slots, TO* __restrict__ out, long long os, int add_input, int T, int silu) {
     pdl_trigger();
     __shared__ int s_place[CONVT_TOK], s_slot[CONVT_TOK];
     const int t0 = blockIdx.x * CONVT_TOK;
@@ -135,6 +139,7 @@ __global__ void causal_conv_tile_kernel(const float* __restrict__ x_in, long lon
                 acc.x += w[j].x * v.x; acc.y += w[j].y * v.y; acc.z += w[j].z * v.z; acc.w += w[j].w * v.w;
             }
             if (add_input) { acc.x += xr[tt].x; acc.y += xr[tt].y; acc.z += xr[tt].z; acc.w += xr[tt].w; }
+            if (silu) { acc.x *= rg_sigmoid(acc.x); acc.y *= rg_sigmoid(acc.y); acc.z *= rg_sigmoid(acc.z); acc.w *= rg_sigmoid(acc.w); }
             TO* o = out + (size_t)t * os + c0;
             o[0] = from_float<TO>(acc.x); o[1] = from_float<TO>(acc.y); o[2] = from_float<TO>(acc.z); o[3] = from_float<TO>(acc.w);
         }
@@ -355,7 +360,7 @@ __global__ void rglru_apply_kernel(const float* __restrict__ a_in, const float* 
 PRISM_EXPORT int prism_causal_conv(const float* x, long long x_stride, const void* taps, int taps_dtype, const void* bias,
                                    int bias_dtype, int K, int C, float* tail, const int* tok_seg, const int* seg_start,
                                    const int* slots, int T, void* out, int out_dtype, long long out_stride, int move_tail,
-                                   int add_input, const float* taps_t, cudaStream_t stream) {
+                                   int add_input, const float* taps_t, int silu, cudaStream_t stream) {
     using namespace prism;
     if (T <= 0 || C <= 0) return 0;
     if (taps_t != nullptr && (uintptr_t)taps_t % 16 != 0) taps_t = nullptr;
@@ -380,13 +385,13 @@ PRISM_EXPORT int prism_causal_conv(const float* x, long long x_stride, const voi
         if (out_dtype == PRISM_DTYPE_BF16)
             return (int)launch_kernel(causal_conv_tile_kernel<__nv_bfloat16>, tgrid, dim3(tthreads), 0, stream, x, x_stride, taps_t, bias,
                                       bb, K, C, (const float*)tail, tok_seg, seg_start, slots, (__nv_bfloat16*)out, out_stride,
-                                      add_input, T);
+                                      add_input, T, silu);
         return (int)launch_kernel(causal_conv_tile_kernel<float>, tgrid, dim3(tthreads), 0, stream, x, x_stride, taps_t, bias, bb, K, C,
-                                  (const float*)tail, tok_seg, seg_start, slots, (float*)out, out_stride, add_input, T);
+                                  (const float*)tail, tok_seg, seg_start, slots, (float*)out, out_stride, add_input, T, silu);
     }
 #define PRISM_CONV(TO, V)                                                                                               \
     return (int)launch_kernel(causal_conv_kernel<TO, V>, grid, dim3(threads), 0, stream, x, x_stride, taps, tb, bias, bb, K, C, \
-                              tail, tok_seg, seg_start, slots, (TO*)out, out_stride, move_tail, add_input, taps_t)
+                              tail, tok_seg, seg_start, slots, (TO*)out, out_stride, move_tail, add_input, taps_t, silu)
     if (out_dtype == PRISM_DTYPE_BF16) {
         if (vec) PRISM_CONV(__nv_bfloat16, 4);
         PRISM_CONV(__nv_bfloat16, 1);

@@ -249,9 +249,14 @@ __global__ void add_normed_rmsnorm_kernel(float* __restrict__ residual, const TD
         if (rows == nullptr) res[c] = v;
         ss += v * v;
     }
+    if (out == nullptr) return;
+    TO* o = out + (size_t)i * H;
+    if (weight == nullptr) {                       // the rows themselves
+        for (int c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_float<TO>(row[c]);
+        return;
+    }
     ss = block_sum(ss, scratch);
     const float inv = 1.f / sqrtf(ss / (float)H + eps);
-    TO* o = out + (size_t)i * H;
     for (int c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_float<TO>(row[c] * inv * load_param(weight, weight_bf16, c));
 }
 
@@ -269,7 +274,7 @@ __global__ void __launch_bounds__(1024) add_normed_rmsnorm_vec_kernel(float* __r
         const int c = (threadIdx.x + it * blockDim.x) * 8;
         if (c < H) {
             load_param8(wd, wd_bf16, c, a[it]);
-            load_param8(weight, weight_bf16, c, w[it]);
+            if (weight != nullptr) load_param8(weight, weight_bf16, c, w[it]);
         }
     }
     pdl_wait();
@@ -310,8 +315,10 @@ __global__ void __launch_bounds__(1024) add_normed_rmsnorm_vec_kernel(float* __r
                 ss += x[it][k] * x[it][k];
             }
             if (rows == nullptr) store8(res + c, x[it]);
+            if (weight == nullptr && out != nullptr) store8(out + (size_t)i * H + c, x[it]);      // the rows themselves
         }
     }
+    if (weight == nullptr) return;
     ss = block_sum(ss, scratch);
     const float inv = 1.f / sqrtf(ss / (float)H + eps);
     TO* o = out + (size_t)i * H;
@@ -330,13 +337,14 @@ __global__ void __launch_bounds__(1024) add_normed_rmsnorm_vec_kernel(float* __r
 
 // residual float32 [T, H] in place; delta [nsplit, T, H] of delta_dtype, normed with wd and eps_d before it is added; out
 // [nrows, H] of out_dtype: the norm (weight, eps) of the new rows, for all of them or for `rows` (the residual is then
-// not written).
+// not written).  weight null: out receives the new rows themselves (null: nothing does).
 PRISM_EXPORT int prism_add_normed_rmsnorm(float* residual, const void* delta, int delta_dtype, int nsplit, long long split_stride,
                                           const void* wd, int wd_dtype, float eps_d, const void* weight, int weight_dtype,
                                           float eps, void* out, int out_dtype, const int* rows, int nrows, int H,
                                           cudaStream_t stream) {
     if (nrows <= 0) return 0;
-    if (nsplit < 1 || delta == nullptr || wd == nullptr || H < 1 || H > 50000) return (int)cudaErrorInvalidValue;
+    if (nsplit < 1 || delta == nullptr || wd == nullptr || H < 1 || H > 50000 || (weight != nullptr && out == nullptr))
+        return (int)cudaErrorInvalidValue;
     const int db = wd_dtype == PRISM_DTYPE_BF16, wb = weight_dtype == PRISM_DTYPE_BF16;
     const int chunks = H / 8;
     const bool vec = H % 8 == 0 && chunks <= 2048 && split_stride % 8 == 0 && (uintptr_t)residual % 32 == 0 &&

@@ -102,7 +102,9 @@ class _Sig:
     prism_scale_add_rmsnorm = [_p, _f, _p, _i, _i, _ll, _p, _i, _f, _p, _i, _i, _i, _p]
     prism_gated_product = [_p, _ll, _p, _ll, _p, _ll, _i, _i, _i, _i, _f, _i, _p]
     prism_qk_norm_rope_store = [_p, _p, _p, _ll, _p, _i, _p, _i, _f, _p, _i, _p, _p, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i,
-                                _i, _i, _i, _i, _p, _i, _i, _p]
+                                _i, _i, _i, _i, _p, _i, _i, _f, _p]
+    prism_step_sizes = [_p, _ll, _p, _i, _p, _i, _i, _i, _p, _p]
+    prism_part_norm_gate = [_p, _p, _ll, _p, _i, _f, _f, _i, _i, _i, _i, _i, _p, _i, _ll, _p]
     prism_conv_unit_gates = [_p, _ll, _i, _i, _p, _i, _i, _p, _p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _f, _p, _p, _i, _p]
     prism_state_tail = [_p, _ll, _i, _p, _i, _p, _p, _i, _p]
     prism_shift_mix = [_p, _i, _p, _p, _i, _i, _p, _p, _p, _i, _p, _i, _ll, _i, _p]
@@ -120,12 +122,13 @@ class _Sig:
     prism_moe_place = [_p, _p, _p, _p, _i, _i, _i, _i, _p, _p, _p, _p, _p]
     prism_moe_route_place = [_p, _ll, _i, _i, _i, _i, _i, _i, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f, _f, _p]
     prism_moe_tcgen05_supported = [_i, _i]
-    prism_moe_gather = [_p, _ll, _p, _p, _p, _p, _i, _i, _i, _i, _p, _p, _p, _p]
+    prism_moe_gather = [_p, _ll, _p, _p, _p, _p, _i, _i, _i, _i, _i, _p, _p, _p, _p, _p, _p]
+    prism_moe_identity = [_p, _p, _p, _i, _i, _i, _i, _p, _p]
     prism_moe_gemm_tcgen05 = [_p, _ll, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _ll, _p, _p, _p, _ll, _i, _i, _i, _p,
-                              _ll, _i, _p, _p, _p]
-    prism_moe_gemm = [_p, _ll, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _ll, _i, _p]
+                              _ll, _i, _p, _p, _f, _p]
+    prism_moe_gemm = [_p, _ll, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _ll, _i, _f, _p]
     prism_hyper_norm = [_p, _ll, _p, _ll, _p, _i, _i, _ll, _p, _i, _p, _i, _p, _i, _i, _p, _i, _f, _i, _p, _i, _p, _i, _i, _p]
-    prism_causal_conv = [_p, _ll, _p, _i, _p, _i, _i, _i, _p, _p, _p, _p, _i, _p, _i, _ll, _i, _i, _p, _p]
+    prism_causal_conv = [_p, _ll, _p, _i, _p, _i, _i, _i, _p, _p, _p, _p, _i, _p, _i, _ll, _i, _i, _p, _i, _p]
     prism_block_gates = [_p, _ll, _p, _p, _i, _p, _p, _i, _p, _i, _f, _i, _i, _i, _p, _p, _ll, _p]
     prism_rglru_scan = [_p, _p, _ll, _p, _ll, _p, _p, _p, _i, _i, _i, _p, _i, _ll, _p]
     prism_cache_store = [_p, _ll, _p, _i, _i, _p, _ll, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i, _p, _p]
@@ -229,19 +232,21 @@ def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: t
 
 
 def add_normed_rmsnorm(residual: torch.Tensor, delta: torch.Tensor, delta_weight: torch.Tensor, delta_eps: float,
-                       weight: torch.Tensor, eps: float, out: torch.Tensor, rows: Optional[torch.Tensor] = None):
+                       weight: Optional[torch.Tensor], eps: float, out: Optional[torch.Tensor], rows: Optional[torch.Tensor] = None):
     """``x = residual + rmsnorm(delta) * delta_weight`` (float32, in place; ``delta [T, H]`` or a stack ``[k, T, H]`` of
     partial sums, normed as their sum), then ``out = rmsnorm(x) * weight``: the norm behind one sublayer, the residual sum
-    and the norm before the next in one launch.  ``rows`` (int32): only these rows, and the residual is not written."""
+    and the norm before the next in one launch.  ``rows`` (int32): only these rows, and the residual is not written.
+    ``weight`` None: no second norm, ``out`` receives the new rows themselves (None: nothing does)."""
     _cuda(residual, delta, delta_weight, weight, out, rows)
-    assert residual.dtype == torch.float32 and residual.is_contiguous() and out.is_contiguous() and delta.is_contiguous()
+    assert residual.dtype == torch.float32 and residual.is_contiguous() and delta.is_contiguous()
     T, H = residual.shape
-    assert delta.shape[-2:] == (T, H) and delta_weight.shape == weight.shape == (H,)
+    assert delta.shape[-2:] == (T, H) and delta_weight.shape == (H,) and (weight is None or weight.shape == (H,))
     n = T if rows is None else rows.shape[0]
-    assert out.shape == (n, H)
+    assert (out is None and weight is None) or (out.shape == (n, H) and out.is_contiguous())
     _check(lib().prism_add_normed_rmsnorm(_ptr(residual), _ptr(delta), _dt(delta), 1 if delta.dim() == 2 else delta.shape[0],
                                           T * H, _ptr(delta_weight), _dt(delta_weight), float(delta_eps), _ptr(weight),
-                                          _dt(weight), float(eps), _ptr(out), _dt(out), _ptr(rows), n, H, _stream()),
+                                          F32 if weight is None else _dt(weight), float(eps), _ptr(out),
+                                          F32 if out is None else _dt(out), _ptr(rows), n, H, _stream()),
            "add_normed_rmsnorm")
 
 
@@ -339,7 +344,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out:
     N = out.shape[-1]
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[1] == K
     assert x.stride(1) == 1 and w.stride(1) == 1 and out.is_contiguous()
-    assert w.shape[0] == (2 * N if epi in _PAIRED else N)
+    assert w.shape[0] == (2 * N if epi in _PAIRED else N) and (bias is None or bias.shape == (w.shape[0],))
     if epi == EPI_PARTIAL:
         assert out.dtype == torch.float32 and out.shape == (ksplit, M, N) and bias is None
     else:
@@ -1462,23 +1467,25 @@ def add_rows(residual: torch.Tensor, delta: Optional[torch.Tensor], copy: Option
                                 F32 if copy is None else _dt(copy), T, H, _stream()), "add_rows")
 
 
-def glu_hidden(ctx, x: torch.Tensor, gate_up_w: torch.Tensor, kind: str, limit: float = 0.0) -> torch.Tensor:
+def glu_hidden(ctx, x: torch.Tensor, gate_up_w: torch.Tensor, kind: str, limit: float = 0.0,
+               bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The hidden layer of a gated feed-forward (``glu`` of the product with the fused gate/up weight); for a few tokens
-    the gated activation is the product's epilogue."""
+    the gated activation is the product's epilogue.  ``bias``: on the product's rows (gate, then up)."""
     act = ctx.alloc((x.shape[0], gate_up_w.shape[0] // 2), x.dtype)
     if tc_gemm_ok(x, gate_up_w, TC_GEMM_MAX_M_SWIGLU):
-        gemm_tc(x, gate_up_w, None, act, {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU, "clamped": EPI_CLAMPED}[kind],
+        gemm_tc(x, gate_up_w, bias, act, {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU, "clamped": EPI_CLAMPED}[kind],
                 ksplit=tc_ksplit_paired(act.shape[1], x.shape[1], M=x.shape[0]), limit=limit)
     else:
-        glu(linear(x, gate_up_w), act, kind, limit)
+        glu(linear(x, gate_up_w, bias), act, kind, limit)
     return act
 
 
-def feed_forward_glu(ctx, x: torch.Tensor, gate_up_w: torch.Tensor, down_w: torch.Tensor, kind: str, limit: float = 0.0):
-    """``down(glu(x))`` with the fused gate/up weight; ``kind`` and ``limit`` as in ``glu``."""
-    if kind == "silu":
+def feed_forward_glu(ctx, x: torch.Tensor, gate_up_w: torch.Tensor, down_w: torch.Tensor, kind: str, limit: float = 0.0,
+                     gate_up_b: Optional[torch.Tensor] = None, down_b: Optional[torch.Tensor] = None):
+    """``down(glu(x))`` with the fused gate/up weight (and biases); ``kind`` and ``limit`` as in ``glu``."""
+    if kind == "silu" and gate_up_b is None and down_b is None:
         return feed_forward_swiglu(ctx, x, gate_up_w, down_w)
-    return linear_delta(glu_hidden(ctx, x, gate_up_w, kind, limit), down_w)
+    return linear_delta(glu_hidden(ctx, x, gate_up_w, kind, limit, gate_up_b), down_w, down_b)
 
 
 def masked_attention(ctx, q: torch.Tensor, out: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor,
@@ -1747,12 +1754,12 @@ def qk_norm_rope_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[t
                        freq: Optional[torch.Tensor], rot: int, q_out: torch.Tensor, k_plane: Optional[torch.Tensor],
                        v_plane: Optional[torch.Tensor], block_table: torch.Tensor, positions: torch.Tensor,
                        tok_seg: torch.Tensor, num_pages: int, max_pos: int, err: torch.Tensor, whole: bool = False,
-                       halves: bool = False, nkv: Optional[int] = None):
+                       halves: bool = False, nkv: Optional[int] = None, v_scale: float = 1.0):
     """From float32 column blocks ``q [T, nh * dk]``, ``k [T, nkv * dk]``, ``v [T, nkv * dv]`` of one product (one
     row stride): RMS norm of every q and k head with ``q_weight`` / ``k_weight`` (``[dk]``, None: no norm) - or,
     with ``whole``, of the whole projection at once (weights ``[nh * dk]`` and ``[nkv * dk]``); rotation of the
     first ``rot`` entries by ``position * freq[i]``, in interleaved pairs or (``halves``) entry i with entry
-    ``i + rot / 2``; q into ``q_out [T, nh, dk]``, k and v into their cache planes at the token's slot.  ``k``, ``v``
+    ``i + rot / 2``; q into ``q_out [T, nh, dk]``, k and ``v * v_scale`` into their cache planes at the token's slot.  ``k``, ``v``
     and the planes None: the layer has no keys and values of its own, only q is made."""
     _cuda(q, k, v, q_weight, k_weight, freq, q_out, k_plane, v_plane, block_table, positions, tok_seg)
     T, nh, dk = q_out.shape
@@ -1776,7 +1783,8 @@ def qk_norm_rope_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[t
         _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(q_weight), F32 if q_weight is None else _dt(q_weight), _ptr(k_weight),
         F32 if k_weight is None else _dt(k_weight), float(eps), _ptr(freq), int(rot), _ptr(q_out), _ptr(k_plane),
         _ptr(v_plane), _dt(q_out), _ptr(block_table), block_table.shape[1], _ptr(positions), _ptr(tok_seg), T, nh, nkv, dk,
-        dv, P, num_pages, int(max_pos), _ptr(err), 1 if whole else 0, 1 if halves else 0, _stream()), "qk_norm_rope_store")
+        dv, P, num_pages, int(max_pos), _ptr(err), 1 if whole else 0, 1 if halves else 0, float(v_scale),
+        _stream()), "qk_norm_rope_store")
 
 
 def conv_unit_gates(proj: torch.Tensor, b_off: int, a_off: int, taps: torch.Tensor, tail: torch.Tensor,
@@ -1852,7 +1860,34 @@ def headnorm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps
                                      {"silu": 0, "sigmoid": 1, "none": 2}[gate_act], _stream()), "headnorm_gate")
 
 
-SCAN_DELTA, SCAN_BONUS, SCAN_CHANNEL, SCAN_GENERAL, SCAN_RETAIN = 0, 1, 2, 3, 4      # csrc/recurrent.cu: PRISM_SCAN_*
+def part_norm_gate(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, parts: int, out: torch.Tensor,
+                   gate_act: str = "silu", gate_first: bool = False, scale: float = 1.0):
+    """RMS norm of rows in ``parts`` equal parts (each by its own root mean square) with a gate: ``out = norm(x) * weight *
+    act(gate) * scale``, or with ``gate_first`` ``out = norm(x * act(gate)) * weight * scale``.  ``x [T, D]`` float32 contiguous,
+    ``gate [T, D]`` float32 and ``out [T, D]`` (compute dtype) with row strides of their own; ``gate_act``: ``silu`` or
+    ``sigmoid``."""
+    _cuda(x, gate, weight, out)
+    T, D = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and gate.dtype == torch.float32 and gate.stride(1) == 1
+    assert gate.shape == out.shape == (T, D) and out.stride(1) == 1 and weight.shape == (D,) and weight.is_contiguous() and D % parts == 0
+    _check(lib().prism_part_norm_gate(_ptr(x), _ptr(gate), gate.stride(0), _ptr(weight), _dt(weight), float(eps), float(scale), T,
+                                      int(parts), D // parts, 1 if gate_first else 0, {"silu": 0, "sigmoid": 1}[gate_act], _ptr(out),
+                                      _dt(out), out.stride(0), _stream()), "part_norm_gate")
+
+
+def step_sizes(z: torch.Tensor, bias: torch.Tensor, a_log: torch.Tensor, bg: torch.Tensor):
+    """``bg[:, :H] = dt = softplus(z + bias)`` and ``bg[:, H:] = exp(-exp(a_log) dt)``; ``z [T, H]`` float32 (row stride free),
+    ``bg [T, 2 H]`` float32."""
+    _cuda(z, bias, a_log, bg)
+    T, H = z.shape
+    assert z.dtype == torch.float32 and z.stride(1) == 1 and bg.dtype == torch.float32 and bg.shape == (T, 2 * H) and bg.is_contiguous()
+    assert bias.shape == a_log.shape == (H,) and bias.is_contiguous() and a_log.is_contiguous()
+    _check(lib().prism_step_sizes(_ptr(z), z.stride(0), _ptr(bias), _dt(bias), _ptr(a_log), _dt(a_log), T, H, _ptr(bg), _stream()),
+           "step_sizes")
+
+
+# csrc/recurrent.cu: PRISM_SCAN_*
+SCAN_DELTA, SCAN_BONUS, SCAN_CHANNEL, SCAN_GENERAL, SCAN_RETAIN, SCAN_TOKEN, SCAN_GATED = 0, 1, 2, 3, 4, 5, 6
 
 
 def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, ctx, H: int,
@@ -1868,7 +1903,9 @@ def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
     key channels, ``ww [T, H * dk]`` (the decay itself), with ``bg [T, H]`` (beta).  ``SCAN_GENERAL``: the generalized
     delta rule ``S <- diag(w) S - c (e^T S) + k v^T; o = S^T r`` with the decay ``ww [T, H * dk]`` and ``ex [T, 2 H dk]``
     = unit key e | removal rate times e (``unit_removal``); every head has its own r and k.  ``SCAN_RETAIN``: ``S <- w0[h] S
-    + k v^T; o = S^T q`` with one constant decay per head, ``w0 [H]``.  ``out [T, H, dv]`` float32."""
+    + k v^T; o = S^T q`` with one constant decay per head, ``w0 [H]``.  ``SCAN_TOKEN``: ``S <- g S + dt k v^T; o = S^T q + w0[h]
+    v`` with ``bg [T, 2 H]`` (dt | g, ``step_sizes``) and ``w0 [H]`` or None; ``rep`` heads share a q/k head.  ``SCAN_GATED``: ``S <-
+    diag(w) S + k v^T; o = S^T q`` with the decay ``ww [T, H * dk]``.  ``out [T, H, dv]`` float32."""
     _cuda(q, k, v, state, out, bg, ww, w0, u, ex)
     T = q.shape[0]
     for t in (q, k, v):
@@ -1877,7 +1914,7 @@ def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
     assert q.shape[1] == k.shape[1] == (H // rep) * dk and v.shape[1] == H * dv
     assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dv, dk)
     assert out.shape == (T, H, dv) and out.is_contiguous() and out.dtype == torch.float32
-    if mode == SCAN_DELTA:
+    if mode in (SCAN_DELTA, SCAN_TOKEN):
         assert bg is not None and bg.shape == (T, 2 * H) and bg.is_contiguous() and bg.dtype == torch.float32
     elif mode == SCAN_CHANNEL:
         assert bg is not None and bg.shape == (T, H) and bg.is_contiguous() and bg.dtype == torch.float32
@@ -1885,6 +1922,8 @@ def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
     elif mode == SCAN_GENERAL:
         assert rep == 1 and ww.dtype == torch.float32 and ww.shape == (T, H * dk) and ww.stride(1) == 1
         assert ex is not None and ex.dtype == torch.float32 and ex.shape == (T, 2 * H * dk) and ex.is_contiguous()
+    elif mode == SCAN_GATED:
+        assert rep == 1 and ww.dtype == torch.float32 and ww.shape == (T, H * dk) and ww.stride(1) == 1
     elif mode == SCAN_RETAIN:
         assert rep == 1 and w0.numel() == H and w0.is_contiguous()
     else:
@@ -1970,6 +2009,53 @@ def retention(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, rot, decay: tor
     headnorm_gate(o, proj[:, 2 * A + B:], ones, eps, 1.0, out)
 
 
+def lightning(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, decay: torch.Tensor, powers: torch.Tensor, state: torch.Tensor,
+              weight: torch.Tensor, eps: float, out: torch.Tensor, path: Optional[str] = None):
+    """Lightning attention between its input and its output projection: from the float32 product ``proj [T, H (2 dk + 2 dv)]``
+    (columns q | k | v | gate), q, k and v through silu, ``S <- decay[h] S + k v^T; o = S^T q`` from and into ``state [slots,
+    H, dv, dk]``, ``out = rms(o over all heads) * weight * sigmoid(gate)`` in the compute dtype.  ``powers`` and ``path`` as in
+    ``retention`` (``"scan"`` puts q, k and v through silu in place)."""
+    T, A, B = proj.shape[0], H * dk, H * dv
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] == 2 * A + 2 * B
+    o = ctx.alloc((T, H, dv), torch.float32)
+    activation(proj[:, :2 * A + B], proj[:, :2 * A + B], "silu")
+    recurrent_scan(SCAN_RETAIN, proj[:, :A], proj[:, A:2 * A], proj[:, 2 * A:2 * A + B], state, ctx, H, 1, dk, dv, o, w0=decay)
+    part_norm_gate(o.view(T, B), proj[:, 2 * A + B:], weight, eps, 1, out, "sigmoid")
+
+
+def gated_linear(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, a2t: torch.Tensor, a2_bias: torch.Tensor, rate: float,
+                 state: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, path: Optional[str] = None):
+    """Gated linear attention between its input and its output projection: from the float32 product ``proj [T, H (2 dk + 2
+    dv) + R]`` (columns q | k | v | gate | the decay's low-rank part), ``w = sigmoid(low @ a2t + a2_bias)^rate``, ``S <- diag(w) S
+    + k v^T; o = S^T q dk^-1/2`` from and into ``state [slots, H, dv, dk]``, ``out = rms(o per head) * weight * silu(gate)`` in
+    the compute dtype.  ``a2t [R, H dk]`` float32, ``weight [dv]``; ``path`` as in ``retention``."""
+    T, A, B, R = proj.shape[0], H * dk, H * dv, a2t.shape[0]
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] == 2 * A + 2 * B + R
+    q, k, v, gate, low = proj[:, :A], proj[:, A:2 * A], proj[:, 2 * A:2 * A + B], proj[:, 2 * A + B:2 * A + 2 * B], proj[:, 2 * A + 2 * B:]
+    ww = ctx.alloc((T, A), torch.float32)
+    lowrank_decay(low, a2t, a2_bias, ww, inner_tanh=False, epilogue=LR_SIGPOW, rate=rate)
+    rotate_slice(q.view(T, H, dk), q.view(T, H, dk), 0, None, ctx.positions, False, 1.0, dk ** -0.5)
+    o = ctx.alloc((T, H, dv), torch.float32)
+    recurrent_scan(SCAN_GATED, q, k, v, state, ctx, H, 1, dk, dv, o, ww=ww)
+    headnorm_gate(o, gate, weight, eps, 1.0, out)
+
+
+def state_space(ctx, u: torch.Tensor, dt: torch.Tensor, z: torch.Tensor, H: int, G: int, N: int, dv: int, dt_bias: torch.Tensor,
+                a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, weight: torch.Tensor, eps: float, parts: int,
+                scale: float, out: torch.Tensor, path: Optional[str] = None):
+    """A state-space mixer behind its convolution: ``u [T, H dv + 2 G N]`` float32 (columns x | B | C; head h reads group ``h //
+    (H / G)`` of B and C), step sizes ``d = softplus(dt + dt_bias)`` from ``dt [T, H]``, ``S <- exp(-exp(a_log) d) S + d B x^T; y =
+    S^T C + skip x`` from and into ``state [slots, H, dv, N]``, ``out = rms(y * silu(z) in ``parts`` equal parts) * weight * scale``
+    in the compute dtype.  ``dt`` and ``z [T, H dv]`` float32 with row strides of their own; ``path`` as in ``retention``."""
+    T, B, rep = u.shape[0], H * dv, H // G
+    assert u.dtype == torch.float32 and u.is_contiguous() and u.shape[1] == B + 2 * G * N
+    o = ctx.alloc((T, H, dv), torch.float32)
+    bg = ctx.alloc((T, 2 * H), torch.float32)
+    step_sizes(dt, dt_bias, a_log, bg)
+    recurrent_scan(SCAN_TOKEN, u[:, B + G * N:], u[:, B:B + G * N], u[:, :B], state, ctx, H, rep, N, dv, o, bg=bg, w0=skip)
+    part_norm_gate(o.view(T, B), z, weight, eps, parts, out, "silu", gate_first=True, scale=scale)
+
+
 def unit_removal(k: torch.Tensor, a: torch.Tensor, a_bias: Optional[torch.Tensor], unit_eps: float, H: int, dk: int,
                  ex: torch.Tensor):
     """What the generalized delta rule takes out of its state, per token and head: ``ex[:, h dk + i] = e_i = k_i /
@@ -1985,7 +2071,7 @@ def unit_removal(k: torch.Tensor, a: torch.Tensor, a_bias: Optional[torch.Tensor
                                     float(unit_eps), T, H, dk, _ptr(ex), _stream()), "unit_removal")
 
 
-LR_EXPEXP, LR_SOFTPLUS, LR_SIGMOID, LR_EXPSIG = 0, 1, 2, 3      # csrc/recurrent.cu: PRISM_LR_*
+LR_EXPEXP, LR_SOFTPLUS, LR_SIGMOID, LR_EXPSIG, LR_SIGPOW, LR_LOGSIGPOW = 0, 1, 2, 3, 4, 5      # csrc/recurrent.cu: PRISM_LR_*
 
 
 def lowrank_decay(low: torch.Tensor, w2t: torch.Tensor, w0: Optional[torch.Tensor], out: torch.Tensor, inner_tanh: bool = True,
@@ -1994,7 +2080,7 @@ def lowrank_decay(low: torch.Tensor, w2t: torch.Tensor, w0: Optional[torch.Tenso
     and in float32 throughout.  ``inner``: tanh or nothing.  ``epilogue``: ``LR_EXPEXP`` ``exp(-exp(z))`` (a per-channel
     decay from its double exponent), ``LR_SOFTPLUS`` ``exp(-exp(rate_log[n // per]) softplus(z))`` (a per-channel decay
     with one rate per ``per`` channels), ``LR_SIGMOID`` (a gate), ``LR_EXPSIG`` ``exp(-rate sigmoid(z))`` (a per-channel
-    decay that stays above ``exp(-rate)``).  ``low [T, R]`` float32 (row stride free), ``w2t [R,
+    decay that stays above ``exp(-rate)``), ``LR_SIGPOW`` ``sigmoid(z)^rate`` and ``LR_LOGSIGPOW`` its logarithm.  ``low [T, R]`` float32 (row stride free), ``w2t [R,
     N]`` float32 (the second matrix, transposed), ``w0 [N]`` or None, ``out [T, N]`` float32."""
     _cuda(low, w2t, w0, out, rate_log)
     T, R = low.shape
@@ -2053,12 +2139,12 @@ def hyper_norm(x: torch.Tensor, streams: int, x_out: Optional[torch.Tensor], del
 
 
 def causal_conv(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor], tail: torch.Tensor, ctx, out: torch.Tensor,
-                move_tail: bool = False, add_input: bool = False, taps_t: Optional[torch.Tensor] = None):
+                move_tail: bool = False, add_input: bool = False, taps_t: Optional[torch.Tensor] = None, silu: bool = False):
     """``out[t, c] = bias[c] + sum_j taps[c, K-1-j] x[t-j, c]``: a short causal convolution over time per channel,
     float32; ``x [T, C]`` (row stride free), ``taps [C, K]`` (last column: the current token's), ``tail [slots, K - 1,
     C]`` the request's last inputs before this step.  ``move_tail``: every request brings one token, and the kernel
     moves the tail up itself (else ``state_tail`` follows).  ``add_input``: ``out = x + conv(x)``.  ``out``: float32
-    or the compute dtype (rounded once).  ``taps_t``: the same taps as float32 ``[K, C]`` (made once by the caller), read
+    or the compute dtype (rounded once).  ``silu``: through silu at the end.  ``taps_t``: the same taps as float32 ``[K, C]`` (made once by the caller), read
     128 bits at a time where the sizes allow."""
     _cuda(x, taps, bias, tail, out, taps_t)
     assert taps_t is None or (taps_t.dtype == torch.float32 and taps_t.is_contiguous() and taps_t.shape == (taps.shape[1], taps.shape[0]))
@@ -2070,7 +2156,8 @@ def causal_conv(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor
     assert bias is None or (bias.shape == (C,) and bias.is_contiguous())
     _check(lib().prism_causal_conv(_ptr(x), x.stride(0), _ptr(taps), _dt(taps), _ptr(bias), F32 if bias is None else _dt(bias),
                                    K, C, _ptr(tail), _ptr(ctx.tok_seg), _ptr(ctx.seg_start), _ptr(ctx.state_slots), T, _ptr(out),
-                                   _dt(out), out.stride(0), 1 if move_tail else 0, 1 if add_input else 0, _ptr(taps_t), _stream()), "causal_conv")
+                                   _dt(out), out.stride(0), 1 if move_tail else 0, 1 if add_input else 0, _ptr(taps_t),
+                                   1 if silu else 0, _stream()), "causal_conv")
 
 
 def block_gates(u: torch.Tensor, wr: torch.Tensor, wi: torch.Tensor, br: torch.Tensor, bi: torch.Tensor, lam: torch.Tensor,
@@ -2120,7 +2207,7 @@ def rglru_scan(a: torch.Tensor, g: torch.Tensor, y: torch.Tensor, state: torch.T
                                   _stream()), "rglru_scan")
 
 
-MOE_ACTS = {"silu": 0, "gelu_tanh": 1, "relu": 2, "relu2": 3}      # csrc/moe.cu: moe_act
+MOE_ACTS = {"silu": 0, "gelu_tanh": 1, "relu": 2, "relu2": 3, "clamped": 4}      # csrc/moe.cu: moe_act, moe_glu
 moe_tensor_cores = True                                 # bf16 experts on tcgen05 (csrc/moe_tcgen05.cu); False: CUDA cores
 
 
@@ -2175,7 +2262,8 @@ def _moe_route_place(L, logits, T, E, top, softmax, renorm, pad, counts, offs, s
 
 def moe_feed_forward(ctx, x: torch.Tensor, logits: torch.Tensor, gate_up_w: torch.Tensor, down_w: torch.Tensor, top: int,
                      softmax: bool = False, renorm: bool = False, scale_input: bool = True, act: str = "silu",
-                     gated: bool = True, choice: Optional[MoeChoice] = None, extra_planes: int = 0, shared=None) -> torch.Tensor:
+                     gated: bool = True, choice: Optional[MoeChoice] = None, extra_planes: int = 0, shared=None, limit: float = 0.0,
+                     own: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Mixture of experts on the step's rows: ``x [T, W]`` (compute dtype), router ``logits [T, E]`` float32,
     ``gate_up_w [E, 2 F, W]`` (an expert's gate rows, then its up rows), ``down_w [E, W, F]``.  Each token takes the
     ``top`` experts with the largest scores (sigmoid of the logits, or their softmax); a choice's weight is its score
@@ -2185,7 +2273,8 @@ def moe_feed_forward(ctx, x: torch.Tensor, logits: torch.Tensor, gate_up_w: torc
     choices' for the caller to fill (a shared expert's result), so that nothing is copied together afterwards.
     ``shared``: ``(gate_up [2 Fs, W], down [W, Fs])`` of a gated expert with the same activation that every token goes
     through: its result is the stack's last plane (one more than ``extra_planes``); a step of up to ``MOE_SHARED_TOKENS`` tokens
-    runs it in the experts' own launches.
+    runs it in the experts' own launches.  ``limit``: of the clamped form.  ``own [T, W]`` float32: ``logits`` may have more columns
+    than there are experts, the last ones identity experts, whose output is the token's row of ``own`` (times the weight).
     Returns float32 ``[top, T, W]``: one plane per choice, which the next norm adds up.  The rows are sorted by
     expert on the device and run as grouped products; the host never learns the counts.  bf16 with rows of 16-byte
     multiples: tcgen05 tiles of one expert each (``csrc/moe_tcgen05.cu``); otherwise CUDA cores (``csrc/moe.cu``)."""
@@ -2194,9 +2283,15 @@ def moe_feed_forward(ctx, x: torch.Tensor, logits: torch.Tensor, gate_up_w: torc
     E, F2, _ = gate_up_w.shape
     F = F2 // 2 if gated else F2
     gt = 1 if gated else 0
-    assert logits.dtype == torch.float32 and logits.shape == (T, E) and logits.stride(1) == 1 and x.stride(1) == 1
+    Z = logits.shape[1]                                     # experts and identity experts
+    assert logits.dtype == torch.float32 and logits.shape == (T, Z) and logits.stride(1) == 1 and x.stride(1) == 1
+    assert Z == E or (Z > E and own is not None and own.dtype == torch.float32 and own.shape == (T, W) and own.is_contiguous()
+                      and not scale_input)
+    assert act != "clamped" or gated
     assert gate_up_w.shape == (E, (2 if gated else 1) * F, W) and down_w.shape == (E, W, F) and gate_up_w.is_contiguous() and down_w.is_contiguous()
-    assert gate_up_w.dtype == x.dtype and down_w.dtype == x.dtype and 1 <= top <= E
+    assert gate_up_w.dtype == x.dtype and down_w.dtype == x.dtype and 1 <= top <= Z
+    if Z == E:
+        own = None
     rows = T * top
     dev = x.device
     L = lib()
@@ -2210,22 +2305,22 @@ def moe_feed_forward(ctx, x: torch.Tensor, logits: torch.Tensor, gate_up_w: torc
                 and sdn.data_ptr() % 16 == 0 and x.data_ptr() % 16 == 0)
         if not ride:
             y = moe_feed_forward(ctx, x, logits, gate_up_w, down_w, top, softmax, renorm, scale_input, act, gated, choice,
-                                 extra_planes + 1)
-            linear(glu_hidden(ctx, x, sgu, act), sdn, None, out=y[-1])
+                                 extra_planes + 1, limit=limit, own=own)
+            linear(glu_hidden(ctx, x, sgu, act, limit), sdn, None, out=y[-1])
             return y
     if x.dtype == torch.bfloat16 and moe_tensor_cores and L.prism_moe_tcgen05_supported(W, F) and x.stride(0) % 8 == 0:
         # tensor cores: every expert's rows start at a multiple of the token tile, one tile has one expert
         ntok = 16 if T <= 16 else (32 if T <= 32 else 64)
         tiles = min(rows, (rows + E * (ntok - 1)) // ntok)          # no more tiles than this, whatever the choice
         padded = tiles * ntok
-        ints = torch.empty(E + (E + 1) + 2 * rows + padded, dtype=torch.int32, device=dev)
-        counts, offs = ints[:E], ints[E:2 * E + 1]
-        o = 2 * E + 1
+        ints = torch.empty(Z + (Z + 1) + 2 * rows + padded, dtype=torch.int32, device=dev)
+        counts, offs = ints[:Z], ints[Z:2 * Z + 1]
+        o = 2 * Z + 1
         sel_e, sel_rank, row_dst = ints[o:o + rows], ints[o + rows:o + 2 * rows], ints[o + 2 * rows:]
         flt = torch.empty(rows + padded, dtype=torch.float32, device=dev)
         sel_w, row_w = flt[:rows], flt[rows:]
         err = _tc_err_word(dev)
-        _moe_route_place(L, logits, T, E, top, softmax, renorm, ntok, counts, offs, sel_e, sel_w, sel_rank, None, None, None, choice)
+        _moe_route_place(L, logits, T, Z, top, softmax, renorm, ntok, counts, offs, sel_e, sel_w, sel_rank, None, None, None, choice)
         sT, s1, s2, k1, k2 = 0, (None, None, 0, 0, 0, 0, None, 0), (None, None, 0, 0, 0, 0, None, 0), 1, 1
         y = ctx.alloc((top + extra_planes + (1 if shared is not None else 0), T, W), torch.float32)
         if shared is not None:
@@ -2242,26 +2337,28 @@ def moe_feed_forward(ctx, x: torch.Tensor, logits: torch.Tensor, gate_up_w: torc
             ws, cnt = _tc_workspace(dev, max(tx1 * k1 * (2 if gated else 1), tx2 * k2) * ty * ntok * 128, max(tx1, tx2) * ty)
         xs = ctx.alloc((padded, W), x.dtype)
         _check(L.prism_moe_gather(_ptr(x), x.stride(0), _ptr(offs), _ptr(sel_e), _ptr(sel_w), _ptr(sel_rank), T, int(top), W, si,
-                                  _ptr(xs), _ptr(row_dst), _ptr(row_w), _stream()), "moe_gather")
+                                  E, _ptr(own), _ptr(y), _ptr(xs), _ptr(row_dst), _ptr(row_w), _stream()), "moe_gather")
         hidden = ctx.alloc((padded, F), x.dtype)
         _check(L.prism_moe_gemm_tcgen05(_ptr(xs), W, _ptr(gate_up_w), _ptr(offs), _ptr(counts), None, None, ntok, tiles, E, F, W,
-                                        gt, MOE_ACTS[act], _ptr(hidden), F, _ptr(err), *s1, k1, _ptr(ws), _ptr(cnt), _stream()),
+                                        gt, MOE_ACTS[act], _ptr(hidden), F, _ptr(err), *s1, k1, _ptr(ws), _ptr(cnt), float(limit), _stream()),
                "moe_gemm_tcgen05")
         _check(L.prism_moe_gemm_tcgen05(_ptr(hidden), F, _ptr(down_w), _ptr(offs), _ptr(counts), _ptr(row_dst),
                                         None if scale_input else _ptr(row_w), ntok, tiles, E, W, F, 0, 0, _ptr(y), W, _ptr(err),
-                                        *s2, k2, _ptr(ws), _ptr(cnt), _stream()), "moe_gemm_tcgen05")
+                                        *s2, k2, _ptr(ws), _ptr(cnt), 0.0, _stream()), "moe_gemm_tcgen05")
         return y
-    ints = torch.empty(E + (E + 1) + 4 * rows, dtype=torch.int32, device=dev)
-    counts, offs = ints[:E], ints[E:2 * E + 1]
-    o = 2 * E + 1
+    ints = torch.empty(Z + (Z + 1) + 4 * rows, dtype=torch.int32, device=dev)
+    counts, offs = ints[:Z], ints[Z:2 * Z + 1]
+    o = 2 * Z + 1
     sel_e, sel_rank, row_tok, row_dst = (ints[o + i * rows:o + (i + 1) * rows] for i in range(4))
     flt = torch.empty(2 * rows, dtype=torch.float32, device=dev)
     sel_w, row_w = flt[:rows], flt[rows:]
-    _moe_route_place(L, logits, T, E, top, softmax, renorm, 1, counts, offs, sel_e, sel_w, sel_rank, row_tok, row_w, row_dst, choice)
+    _moe_route_place(L, logits, T, Z, top, softmax, renorm, 1, counts, offs, sel_e, sel_w, sel_rank, row_tok, row_w, row_dst, choice)
     hidden = ctx.alloc((rows, F), x.dtype)
     _check(L.prism_moe_gemm(_ptr(x), x.stride(0), _ptr(gate_up_w), _dt(x), _ptr(offs), _ptr(row_tok), _ptr(row_w), _ptr(row_dst),
-                            rows, E, F, W, 1, si, MOE_ACTS[act], _ptr(hidden), F, gt, _stream()), "moe_gemm")
+                            rows, E, F, W, 1, si, MOE_ACTS[act], _ptr(hidden), F, gt, float(limit), _stream()), "moe_gemm")
     y = ctx.alloc((top + extra_planes, T, W), torch.float32)
     _check(L.prism_moe_gemm(_ptr(hidden), F, _ptr(down_w), _dt(x), _ptr(offs), _ptr(row_tok), _ptr(row_w), _ptr(row_dst),
-                            rows, E, W, F, 0, si, 0, _ptr(y), W, 1, _stream()), "moe_gemm")
+                            rows, E, W, F, 0, si, 0, _ptr(y), W, 1, 0.0, _stream()), "moe_gemm")
+    if own is not None:
+        _check(L.prism_moe_identity(_ptr(own), _ptr(sel_e), _ptr(sel_w), T, int(top), W, E, _ptr(y), _stream()), "moe_identity")
     return y

@@ -60,7 +60,7 @@ class GQAAttention(Mixer):
     instead (all heads of q, or of k, at once, with weights of that size).  ``gate``: the concatenated heads are
     multiplied by ``sigmoid(W_g h)`` before the output projection; ``gate="head"``: one gate number per head.
     ``sink_value``: a constant sink, the same for every head (0: one is added to the softmax's denominator).  ``out_scale``: a constant on the layer's result (folded into
-    the gate).  A rotation with rescaled frequencies (``rotary_scaled``), the query/key norm and the gate
+    the gate, or into the stored values where a layer that works from the float32 projection has keys and values of its own).  A rotation with rescaled frequencies (``rotary_scaled``), the query/key norm and the gate
     work from the float32 result of the input projection; so may a layer without keys and values of its own.
     ``qk_norm_weight`` False: the query/key norm has no weights (q and k are divided by their root mean square and
     nothing else).  ``dist_bias``: a learned bias by distance on the scaled scores, ``dict(rows=B, far=D)``: a table
@@ -294,13 +294,14 @@ class GQAAttention(Mixer):
                                rot.inv_freq if rot and rot.rotary_dim else None, rot.rotary_dim if rot else 0, q,
                                cache.k if own else None, cache.v if own else None, cache.block_table, ctx.positions,
                                ctx.tok_seg, cache.num_pages, ctx.max_positions, ctx.err, whole=self.qk_norm_whole,
-                               halves=bool(rot and not rot.interleaved), nkv=self.nkv)
+                               halves=bool(rot and not rot.interleaved), nkv=self.nkv,
+                               v_scale=self.out_scale if own and not self.gate else 1.0)
         attn = ctx.alloc((T, self.nh * self.vhd), ctx.dtype) if self.gate else out
         ops.masked_attention(ctx, q, attn, cache.k, cache.v, cache.block_table, cache.num_pages, self.mask, self.scale,
                              self._sink(), self.bias_table)
         if self.gate:
             ops.gated_product(attn, proj[:, qs + kvs + vs:], out, "sigmoid", self.out_scale)
-        elif self.out_scale != 1.0:
+        elif self.out_scale != 1.0 and not own:
             out.mul_(self.out_scale)
 
     def _sink(self):

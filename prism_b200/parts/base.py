@@ -146,6 +146,11 @@ class NormedDelta:
     weight: object
     eps: float
 
+    def carry_out(self, residual, copy):
+        """The sum alone, in place on the float32 rows; ``copy`` (None: not wanted) receives the new rows in its dtype."""
+        from .. import ops
+        ops.add_normed_rmsnorm(residual, self.delta, self.weight, self.eps, None, 0.0, copy)
+
 
 @dataclass(frozen=True)
 class DetachedProjection:
@@ -304,6 +309,8 @@ class FeedForward(Part):
     category = "feed_forward"
     detachable_out = False
     detachable_in = False
+    # True: ``forward`` takes the float32 rows that ``x`` is the copy of as well (``rows32``), where the block has them
+    reads_float32_too = False
 
     def forward(self, ctx, x):
         raise NotImplementedError

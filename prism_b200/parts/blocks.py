@@ -7,6 +7,7 @@ feed-forward, a per-layer token input after the feed-forward.
 ``parallel``: one norm whose output both the mixer and the feed-forward read;
 their two results are added to the residual stream together.
 ``sandwich``: a norm before and after every sublayer.
+``outnorm``: a norm on every sublayer's result only; the sublayers read the stream itself.
 ``postnorm``: the residual stream itself is normed after every sum,
 ``x <- norm(alpha x + sublayer(x))``, and the sublayers read x as it is.
 ``hyper``: pre-norm sublayers around a residual stream kept in several
@@ -16,7 +17,7 @@ from __future__ import annotations
 
 from typing import Optional
 
-from .base import Block, CacheNeed, ParamSpec, PartSpec, StreamUpdate, WeightSource, build_part, register_part
+from .base import Block, CacheNeed, NormedDelta, ParamSpec, PartSpec, StreamUpdate, WeightSource, build_part, register_part
 from .. import ops
 
 
@@ -163,6 +164,45 @@ class SandwichBlock(Block):
         if self.feed_forward is not None:
             h = self.ff_norm.forward(ctx, residual, d)
             d = self.ff_post.leave_open(self.feed_forward.forward(ctx, h))
+        return residual, d
+
+
+@register_part("block", "outnorm")
+class OutputNormBlock(Block):
+    """``x += mixer_post(mixer(x))``, then ``x += ff_post(feed_forward(x))``: a norm on each sublayer's result and none on
+    what it reads, which is the residual stream itself (its copy in the compute dtype; a mixer with ``reads_float32`` gets
+    the float32 rows, a feed-forward with ``reads_float32_too`` both).  Each result is left open as a ``NormedDelta`` and
+    carried out - partial sums, norm, residual sum, copy - by one launch in front of the next sublayer, or by the norm that
+    follows the last block.  ``feed_forward`` None: the layer ends after its mixer (a file that still holds the second
+    norm's weight may: nothing reads it)."""
+
+    def __init__(self, mixer: PartSpec, mixer_post: PartSpec, feed_forward: Optional[PartSpec] = None,
+                 ff_post: Optional[PartSpec] = None):
+        self.mixer = self.add_child("mixer", build_part("mixer", mixer))
+        self.mixer_post = self.add_child("mixer_post", build_part("norm", mixer_post))
+        self.feed_forward = (self.add_child("feed_forward", build_part("feed_forward", feed_forward))
+                             if feed_forward is not None else None)
+        if self.feed_forward is not None and ff_post is None:
+            raise ValueError("an outnorm block with a feed-forward needs the norm behind it")
+        self.ff_post = self.add_child("ff_post", build_part("norm", ff_post)) if ff_post is not None else None
+
+    @staticmethod
+    def _rows(ctx, residual, delta):
+        """Carries out what is open and returns the rows in the compute dtype."""
+        copy = None if ctx.dtype == ops.torch.float32 else ctx.alloc(tuple(residual.shape), ctx.dtype)
+        if isinstance(delta, NormedDelta):
+            delta.carry_out(residual, copy)
+        elif delta is not None or copy is not None:
+            ops.add_rows(residual, delta, copy)
+        return residual if copy is None else copy
+
+    def forward(self, ctx, residual, delta, cache):
+        h = self._rows(ctx, residual, delta)
+        d = self.mixer_post.leave_open(self.mixer.forward(ctx, residual if self.mixer.reads_float32 else h, cache))
+        if self.feed_forward is not None:
+            h = self._rows(ctx, residual, d)
+            ff = self.feed_forward
+            d = self.ff_post.leave_open(ff.forward(ctx, h, rows32=residual) if ff.reads_float32_too else ff.forward(ctx, h))
         return residual, d
 
 

@@ -16,14 +16,15 @@ from .. import ops
 class SwiGLU(FeedForward):
     """``names``: the gate, up and down tensors' names in the model file.  ``activation``: what the gate goes
     through, ``silu`` or ``gelu_tanh``; or ``clamped``, the form with both projections limited by ``limit``
-    (``ops.glu``)."""
+    (``ops.glu``).  ``biases``: the names of the gate's, the up and the down projection's biases, or None."""
 
     def __init__(self, hidden_size: int, intermediate_size: int,
                  names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), activation: str = "silu",
-                 limit: Optional[float] = None):
+                 limit: Optional[float] = None, biases=None):
         self.hidden_size = int(hidden_size)
         self.intermediate_size = int(intermediate_size)
         self.names = tuple(names)
+        self.biases = None if biases is None else tuple(biases)
         if activation not in ops.GATED:
             raise ValueError(f"a gated feed-forward's activation is one of {ops.GATED}, got {activation!r}")
         if activation == "clamped" and limit is None:
@@ -36,15 +37,19 @@ class SwiGLU(FeedForward):
             ParamSpec("gate_up_w", (WeightSource(self.names[0], (I, H)),
                                     WeightSource(self.names[1], (I, H)))),
             ParamSpec("down_w", (WeightSource(self.names[2], (H, I)),)),
-        ]
+        ] + ([] if self.biases is None else [
+            ParamSpec("gate_up_b", (WeightSource(self.biases[0], (I,), "bias"), WeightSource(self.biases[1], (I,), "bias"))),
+            ParamSpec("down_b", (WeightSource(self.biases[2], (H,), "bias"),)),
+        ])
 
     def forward(self, ctx, x):
-        return ops.feed_forward_glu(ctx, x, self.w["gate_up_w"], self.w["down_w"], self.activation, self.limit)
+        return ops.feed_forward_glu(ctx, x, self.w["gate_up_w"], self.w["down_w"], self.activation, self.limit,
+                                    self.w.get("gate_up_b"), self.w.get("down_b"))
 
     def forward_to(self, ctx, x, out):
         """The layer's result into ``out [T, hidden]`` (float32, contiguous): a plane of a stack that the next norm adds up."""
-        act = ops.glu_hidden(ctx, x, self.w["gate_up_w"], self.activation, self.limit)
-        ops.linear(act, self.w["down_w"], None, out=out)
+        act = ops.glu_hidden(ctx, x, self.w["gate_up_w"], self.activation, self.limit, self.w.get("gate_up_b"))
+        ops.linear(act, self.w["down_w"], self.w.get("down_b"), out=out)
 
 
 @register_part("feed_forward", "mlp")
@@ -108,17 +113,29 @@ class MixtureOfExperts(FeedForward):
     experts of the best ``keep`` groups can be chosen.  ``weight_scale``: a constant on the weights; ``sum_eps``: added
     to the sum that ``renorm`` divides by.  ``shared``: a feed-forward part with ``forward_to`` (``mlp``, ``swiglu``) that
     every token goes through and whose result is added (its tensors under this part's prefix).  ``router_bias``: the name
-    of a tensor ``[experts]`` added to the router's logits."""
+    of a tensor ``[experts]`` added to the router's logits.  ``activation`` ``clamped`` (with ``limit``): the form of ``ops.glu``
+    with gate and up limited.  ``identity``: that many further rows of the router (and entries of the tensors above), behind
+    the experts' own: a choice of one of them adds the layer's input itself, times the weight (from the float32 rows where
+    the block has them); they have no other tensors, and their scores take part in the softmax and the choice."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int, softmax: bool = False,
                  renorm: bool = False, scale_input: bool = True, activation: str = "silu",
                  names=("router", "e{e}.", "gate", "up", "down"), gated: bool = True, correction: Optional[str] = None,
                  groups: int = 1, keep: Optional[int] = None, weight_scale: float = 1.0, sum_eps: float = 0.0,
-                 shared: Optional[PartSpec] = None, router_bias: Optional[str] = None):
+                 shared: Optional[PartSpec] = None, router_bias: Optional[str] = None, limit: Optional[float] = None,
+                 identity: int = 0):
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.experts, self.top = int(experts), int(top)
-        if not 1 <= self.top <= self.experts:
-            raise ValueError(f"a token uses {self.top} of {self.experts} experts: between 1 and all of them")
+        self.identity = int(identity)
+        self.routed = self.experts + self.identity              # what the router chooses among
+        if self.identity < 0 or not 1 <= self.top <= self.routed:
+            raise ValueError(f"a token uses {self.top} of {self.routed} experts: between 1 and all of them")
+        if activation == "clamped" and (limit is None or not gated):
+            raise ValueError("the clamped form needs its limit and a gate")
+        if self.identity and (scale_input or groups != 1):
+            raise ValueError("identity experts: the weight multiplies an expert's output, and there are no groups")
+        self.limit = float(limit or 0.0)
+        self.reads_float32_too = self.identity > 0
         if activation not in ops.MOE_ACTS:
             raise ValueError(f"activation {activation!r}: one of {sorted(ops.MOE_ACTS)}")
         self.softmax, self.renorm, self.scale_input, self.activation = bool(softmax), bool(renorm), bool(scale_input), activation
@@ -141,26 +158,28 @@ class MixtureOfExperts(FeedForward):
             p = pat.format(e=e)
             gu += ([WeightSource(p + gate, (I, H))] if self.gated else []) + [WeightSource(p + up, (I, H))]
             dn.append(WeightSource(p + down, (H, I)))
-        ps = [ParamSpec("router_w", (WeightSource(router, (self.experts, H)),)),
+        ps = [ParamSpec("router_w", (WeightSource(router, (self.routed, H)),)),
               ParamSpec("gate_up_w", tuple(gu)), ParamSpec("down_w", tuple(dn))]
         if self.router_bias is not None:
-            ps.append(ParamSpec("router_b", (WeightSource(self.router_bias, (self.experts,), "bias"),)))
+            ps.append(ParamSpec("router_b", (WeightSource(self.router_bias, (self.routed,), "bias"),)))
         if self.correction is not None:
-            ps.append(ParamSpec("correction", (WeightSource(self.correction, (self.experts,), "bias"),)))
+            ps.append(ParamSpec("correction", (WeightSource(self.correction, (self.routed,), "bias"),)))
         return ps
 
     def on_bound(self):
         self.choice = ops.MoeChoice(self.w.get("correction"), self.groups, self.keep, self.weight_scale, self.sum_eps)
 
-    def forward(self, ctx, x):
+    def forward(self, ctx, x, rows32=None):
         H, I, E = self.hidden_size, self.intermediate_size, self.experts
         # a gated shared expert with the experts' own activation runs with them
-        alike = isinstance(self.shared, SwiGLU) and self.gated and self.shared.activation == self.activation
+        alike = (isinstance(self.shared, SwiGLU) and self.gated and self.shared.activation == self.activation
+                 and self.shared.biases is None and self.shared.limit == self.limit)
         logits = ops.linear(x, self.w["router_w"], self.w.get("router_b"), out_dtype=ops.torch.float32)
         y = ops.moe_feed_forward(ctx, x, logits, self.w["gate_up_w"].view(E, (2 if self.gated else 1) * I, H),
                                  self.w["down_w"].view(E, H, I), self.top, self.softmax, self.renorm, self.scale_input,
                                  self.activation, self.gated, self.choice, extra_planes=0 if self.shared is None or alike else 1,
-                                 shared=(self.shared.w["gate_up_w"], self.shared.w["down_w"]) if alike else None)
+                                 shared=(self.shared.w["gate_up_w"], self.shared.w["down_w"]) if alike else None,
+                                 limit=self.limit, own=None if not self.identity else (x.float() if rows32 is None else rows32))
         if self.shared is not None and not alike:
             self.shared.forward_to(ctx, x, y[self.top])          # the shared expert's result is the stack's last plane
         return y

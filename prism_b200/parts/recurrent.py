@@ -14,6 +14,10 @@ low-rank product, and a low-rank sigmoid gate on the read-out.
 ``general_delta``: the generalized delta rule: a decay and a removal rate per
 key channel; what is removed is read along the unit key.
 ``retention``: a sum of outer products under one constant decay per head, of rotated queries and keys.
+``lightning``: the same of queries, keys and values behind silu, with one norm over all heads.
+``gated_linear``: a sum of outer products under a decay per key channel from a low-rank product.
+``state_space``: a sum of outer products with a step size per head and token that also sets the decay, behind a short
+convolution, with a skip path and a norm behind the gate.
 ``rglru``: a recurrence with one number of state per channel whose gates are
 block-diagonal products, behind a short convolution, beside a gelu branch.
 ``sum``: several mixers side by side on the same input, their results scaled
@@ -339,6 +343,203 @@ class RetentionMixer(Mixer):
         proj = ops.linear(x, self.w["in_w"], None, out_dtype=torch.float32)          # q | k | v | g
         inner = ctx.alloc((T, B), ctx.dtype)
         ops.retention(ctx, proj, H, dk, dv, self.rot, self.decays, self.powers, state.state, self.eps, self.ones, inner)
+        return ops.linear_delta(inner, self.w["o_w"], None, f32=True)
+
+
+@register_part("mixer", "lightning")
+class LightningMixer(Mixer):
+    """Linear attention with a fixed decay per head behind silu, without softmax, denominator or scale.  With h the input,
+    per token and head (``num_heads`` heads of ``head_dim`` key and ``v_head_dim`` value channels)::
+
+        q, k, v = silu(W_q h), silu(W_k h), silu(W_v h)
+        S <- decay S + k v^T;   o = S^T q                    the head's entry of ``decay``
+        out = W_o [o / rms(o) * norm * sigmoid(W_g h)]       one root mean square over all heads
+
+    State per request: S ``[H, v_head_dim, head_dim]`` (stored column by column), float32, starting at zero.  All input
+    projections are one product with float32 results.  ``names``: keys q, k, v, g, norm, o."""
+
+    NAMES = dict(q="q", k="k", v="v", g="g", norm="norm", o="o")
+    graph_safe = True
+    float32_projection = True
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, decay: Sequence[float], eps: float,
+                 names: Optional[dict] = None):
+        self.hidden_size, self.H, self.dk, self.dv = int(hidden_size), int(num_heads), int(head_dim), int(v_head_dim)
+        if min(self.H, self.dk, self.dv) < 1 or self.dk > 1024:
+            raise ConfigError("lightning: heads and sizes must be positive, head_dim at most 1024")
+        self.decay = [float(d) for d in decay]
+        if len(self.decay) != self.H:
+            raise ConfigError(f"lightning: {len(self.decay)} decays for {self.H} heads")
+        self.eps = float(eps)
+        self.names = dict(self.NAMES, **(names or {}))
+
+    def cache_needs(self):
+        return (CacheNeed("state", state_shape=(self.H, self.dv, self.dk)),)
+
+    def cache_need(self):
+        return self.cache_needs()[0]
+
+    def params(self):
+        W, n, A, B = self.hidden_size, self.names, self.H * self.dk, self.H * self.dv
+        return [ParamSpec("in_w", (WeightSource(n["q"], (A, W)), WeightSource(n["k"], (A, W)), WeightSource(n["v"], (B, W)),
+                                   WeightSource(n["g"], (B, W)))),
+                ParamSpec("norm", (WeightSource(n["norm"], (B,), "norm"),)),
+                ParamSpec("o_w", (WeightSource(n["o"], (W, B)),))]
+
+    def on_bound(self):
+        self.decays = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(self.device)
+        self.powers = ops.decay_powers(self.decays)
+
+    def forward(self, ctx, x, cache):
+        state = cache[0] if isinstance(cache, tuple) else cache
+        proj = ops.linear(x, self.w["in_w"], None, out_dtype=torch.float32)          # q | k | v | g
+        inner = ctx.alloc((x.shape[0], self.H * self.dv), ctx.dtype)
+        ops.lightning(ctx, proj, self.H, self.dk, self.dv, self.decays, self.powers, state.state, self.w["norm"], self.eps, inner)
+        return ops.linear_delta(inner, self.w["o_w"], None, f32=True)
+
+
+@register_part("mixer", "gated_linear")
+class GatedLinearMixer(Mixer):
+    """Gated linear attention: a decay of its own for every key channel, without softmax or denominator.  With h the
+    input, per token and head (``num_heads`` heads of ``head_dim`` key and ``v_head_dim`` value channels)::
+
+        q, k, v = W_q h / sqrt(head_dim), W_k h, W_v h
+        w = sigmoid(W_a2 (W_a1 h) + a2_b)^(1 / tau)          per head and key channel
+        S <- diag(w) S + k v^T;   o = S^T q
+        out = W_o [o / rms(o) * norm * silu(W_g h)]          norm per head, one weight vector for all heads
+
+    State per request: S ``[H, v_head_dim, head_dim]`` (stored column by column), float32, starting at zero.  All input
+    projections, the decay's first product among them, are one product with float32 results; the decay's second product
+    runs in float32 with its epilogue.  The decay's rank is the shape of ``a1``.  ``names``: keys q, k, v, g, a1, a2, a2_b,
+    norm, o."""
+
+    NAMES = dict(q="q", k="k", v="v", g="g", a1="a1", a2="a2", a2_b="a2.b", norm="norm", o="o")
+    graph_safe = True
+    float32_projection = True
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, decay_rank: int, tau: float, eps: float,
+                 names: Optional[dict] = None):
+        self.hidden_size, self.H, self.dk, self.dv = int(hidden_size), int(num_heads), int(head_dim), int(v_head_dim)
+        self.rank, self.tau, self.eps = int(decay_rank), float(tau), float(eps)
+        if min(self.H, self.dk, self.dv, self.rank) < 1 or self.dk > 1024 or not self.tau > 0:
+            raise ConfigError("gated linear attention: heads, sizes, the decay's rank and tau must be positive, head_dim at most 1024")
+        self.names = dict(self.NAMES, **(names or {}))
+
+    def cache_needs(self):
+        return (CacheNeed("state", state_shape=(self.H, self.dv, self.dk)),)
+
+    def cache_need(self):
+        return self.cache_needs()[0]
+
+    def params(self):
+        W, n, A, B = self.hidden_size, self.names, self.H * self.dk, self.H * self.dv
+        return [ParamSpec("in_w", (WeightSource(n["q"], (A, W)), WeightSource(n["k"], (A, W)), WeightSource(n["v"], (B, W)),
+                                   WeightSource(n["g"], (B, W)), WeightSource(n["a1"], (self.rank, W)))),
+                ParamSpec("a2", (WeightSource(n["a2"], (A, self.rank)),)),
+                ParamSpec("a2_b", (WeightSource(n["a2_b"], (A,), "bias"),)),
+                ParamSpec("norm", (WeightSource(n["norm"], (self.dv,), "norm"),)),
+                ParamSpec("o_w", (WeightSource(n["o"], (W, B)),))]
+
+    def on_bound(self):
+        # the decay's second product runs in float32 whatever the engine's dtype; transposed, so that the kernels'
+        # neighbouring threads read neighbouring floats
+        self.a2t = self.w["a2"].float().t().contiguous() if self.w["a2"] is not None else None
+
+    def forward(self, ctx, x, cache):
+        state = cache[0] if isinstance(cache, tuple) else cache
+        proj = ops.linear(x, self.w["in_w"], None, out_dtype=torch.float32)          # q | k | v | g | a1
+        inner = ctx.alloc((x.shape[0], self.H * self.dv), ctx.dtype)
+        ops.gated_linear(ctx, proj, self.H, self.dk, self.dv, self.a2t, self.w["a2_b"], 1.0 / self.tau, state.state, self.w["norm"],
+                         self.eps, inner)
+        return ops.linear_delta(inner, self.w["o_w"], None, f32=True)
+
+
+@register_part("mixer", "state_space")
+class StateSpaceMixer(Mixer):
+    """A selective state-space mixer with one decay per head and token (Mamba-2's form).  With h the input, ``num_heads``
+    heads of ``v_head_dim`` channels, ``groups`` groups of B and C with ``state`` entries each (head i reads group ``i //
+    (heads / groups)``)::
+
+        [z | x | B | C | dt] = W_in h;   [x | B | C] <- silu(conv([x | B | C]) + conv_b)      conv: causal, per channel
+        d = softplus(dt + dt_bias)                                                         per head
+        S <- exp(-exp(A_log) d) S + d B x^T;   y = S^T C + D x                              per head, S [state, v_head_dim]
+        out = W_o [y silu(z), normed in ``norm_groups`` equal parts, * norm]
+
+    State per request: S ``[H, v_head_dim, state]`` (stored column by column) and the convolution's last ``conv - 1`` inputs,
+    both float32, both starting at zero.  The input projection gives float32; convolution, step sizes, decays, state,
+    gate and norm are float32.  ``names``: keys in, conv, conv_b, dt_bias, A_log, D, norm, o."""
+
+    NAMES = {"in": "in", "conv": "conv", "conv_b": "conv.b", "dt_bias": "dt_bias", "A_log": "A_log", "D": "D", "norm": "norm", "o": "o"}
+    graph_safe = True
+    float32_projection = True
+    detachable_out = detachable_in = True
+
+    def __init__(self, hidden_size: int, num_heads: int, v_head_dim: int, state: int, groups: int, conv: int, norm_groups: int,
+                 eps: float, out_scale: float = 1.0, names: Optional[dict] = None):
+        self.hidden_size, self.H, self.dv, self.N = int(hidden_size), int(num_heads), int(v_head_dim), int(state)
+        self.G, self.K, self.parts = int(groups), int(conv), int(norm_groups)
+        self.inner = self.H * self.dv
+        if min(self.H, self.dv, self.N, self.G, self.K, self.parts) < 1 or self.H % self.G or self.inner % self.parts:
+            raise ConfigError(f"state-space mixer: heads ({self.H}) must be a multiple of groups ({self.G}), heads times vdim "
+                              f"({self.inner}) a multiple of norm_groups ({self.parts}), and every size positive")
+        if self.N > 1024:
+            raise ConfigError(f"state-space mixer: state {self.N} exceeds the scan kernel's 1024")
+        self.eps, self.out_scale = float(eps), float(out_scale)
+        self.names = dict(self.NAMES, **(names or {}))
+        self.C = self.inner + 2 * self.G * self.N                 # channels of the convolution: x | B | C
+        self._own_in = self._own_out = True
+
+    def cache_needs(self):
+        return (CacheNeed("state", state_shape=(self.H, self.dv, self.N)),
+                CacheNeed("state", state_shape=(self.K - 1, self.C)))
+
+    def _in_source(self):
+        return WeightSource(self.names["in"], (self.inner + self.C + self.H, self.hidden_size))
+
+    def _out_source(self):
+        return WeightSource(self.names["o"], (self.hidden_size, self.inner))
+
+    def params(self):
+        n, H = self.names, self.H
+        return (([ParamSpec("in_w", (self._in_source(),))] if self._own_in else [])
+                + [ParamSpec("taps", (WeightSource(n["conv"], (self.C, self.K)),)),
+                   ParamSpec("conv_b", (WeightSource(n["conv_b"], (self.C,), "bias"),)),
+                   ParamSpec("dt_bias", (WeightSource(n["dt_bias"], (H,), "bias"),)),
+                   ParamSpec("A_log", (WeightSource(n["A_log"], (H,), "bias"),)),
+                   ParamSpec("D", (WeightSource(n["D"], (H,), "norm"),)),
+                   ParamSpec("norm", (WeightSource(n["norm"], (self.inner,), "norm"),))]
+                + ([ParamSpec("o_w", (self._out_source(),))] if self._own_out else []))
+
+    def detach_out_projection(self):
+        self._own_out = False
+        return DetachedProjection(self.handed_over(self._out_source()), (), self.inner)
+
+    def detach_in_projection(self):
+        self._own_in = False
+        return DetachedProjection(self.handed_over(self._in_source()), (), self.inner + self.C + self.H, float32=True)
+
+    def on_bound(self):
+        # the taps once more as float32 [K, channels]: the kernels' neighbouring threads read neighbouring floats
+        self.taps_t = self.w["taps"].float().t().contiguous() if self.w.get("taps") is not None else None
+
+    def forward_inner(self, ctx, x, cache, out, proj=None):
+        state, tail = cache
+        T, inner, C = x.shape[0], self.inner, self.C
+        if proj is None:
+            proj = ops.linear(x, self.w["in_w"], None, out_dtype=torch.float32)        # z | x | B | C | dt
+        xbc = proj[:, inner:inner + C]
+        u = ctx.alloc((T, C), torch.float32)
+        single = ctx.decode_only          # one token per request: the kernel that reads the tail also moves it up
+        ops.causal_conv(xbc, self.w["taps"], self.w["conv_b"], tail.state, ctx, u, move_tail=single, taps_t=self.taps_t, silu=True)
+        if not single:
+            ops.state_tail(xbc, tail.state, ctx)
+        ops.state_space(ctx, u, proj[:, inner + C:inner + C + self.H], proj[:, :inner], self.H, self.G, self.N, self.dv,
+                        self.w["dt_bias"], self.w["A_log"], self.w["D"], state.state, self.w["norm"], self.eps, self.parts,
+                        self.out_scale, out)
+
+    def forward(self, ctx, x, cache):
+        inner = ctx.alloc((x.shape[0], self.inner), ctx.dtype)
+        self.forward_inner(ctx, x, cache, inner)
         return ops.linear_delta(inner, self.w["o_w"], None, f32=True)
 
 
