@@ -721,7 +721,7 @@ def limatar_kernel_numbers(s, pk, once=None):
     freq = (10000.0 ** (-torch.arange(0, dk, 2).float() / dk)).to(DEV)
     rot = RotaryParams(freq, dk, False)
     decay = torch.tensor([1.0 - 2.0 ** (-5 - i % 8) for i in range(H)], device=DEV)
-    powers, ones = ops.decay_powers(decay), torch.ones(dv, device=DEV)
+    powers = ops.decay_powers(decay)
     for label, batch, cached, q_len in shapes:
         Tt = batch * q_len
         c = types.SimpleNamespace(seg_start=(torch.arange(batch + 1, dtype=torch.int32) * q_len).to(DEV), S=batch, max_q_len=q_len,
@@ -731,7 +731,7 @@ def limatar_kernel_numbers(s, pk, once=None):
         state = torch.zeros(batch + 1, H, dv, dk, device=DEV)
         proj = torch.randn(Tt, 2 * H * (dk + dv), device=DEV) * 0.3
         o = torch.empty(Tt, H * dv, device=DEV, dtype=torch.bfloat16)
-        run(f"retention_{label}", lambda: ops.retention(c, proj, H, dk, dv, rot, decay, powers, state, 1e-6, ones, o), 4 * Tt * H * dk * dv,
+        run(f"retention_{label}", lambda: ops.retention(c, proj, H, dk, dv, rot, decay, powers, state, 1e-6, o), 4 * Tt * H * dk * dv,
             4 * (2 * batch * H * dk * dv + Tt * H * (2 * dk + 2 * dv)) + 2 * Tt * H * dv, fp32=True)
         x = torch.nn.functional.normalize(torch.randn(Tt, 3 * H, dk, device=DEV), dim=-1).view(Tt, -1)
         bg = torch.rand(Tt, 2 * H, device=DEV) * 0.5 + 0.5

@@ -110,10 +110,12 @@ class _Sig:
     prism_shift_mix = [_p, _i, _p, _p, _i, _i, _p, _p, _p, _i, _p, _i, _ll, _i, _p]
     prism_headnorm_gate = [_p, _p, _ll, _p, _i, _i, _f, _f, _i, _i, _i, _p, _i, _ll, _i, _p]
     prism_recurrent_scan = [_i, _p, _ll, _ll, _ll, _ll, _p, _p, _ll, _p, _i, _p, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _i, _p, _ll, _p]
-    prism_retention_step_supported = [_i, _i]
-    prism_retention_chunks_supported = [_i, _i, _i, _i]
-    prism_retention_step = [_p, _ll, _i, _i, _i, _i, _i, _i, _i, _p, _i, _i, _f, _f, _p, _p, _p, _p, _f, _p, _i, _ll, _p]
-    prism_retention_chunks = [_p, _ll, _i, _i, _i, _i, _i, _i, _i, _i, _p, _i, _i, _f, _f, _p, _p, _p, _p, _f, _p, _p, _ll, _p]
+    prism_decay_step_supported = [_i, _i]
+    prism_decay_chunks_supported = [_i, _i, _i, _i]
+    prism_decay_step = [_i, _p, _p, _p, _ll, _i, _i, _i, _i, _i, _i, _p, _i, _i, _f, _f, _f, _p, _p, _ll, _p, _i, _p, _i, _p, _i,
+                        _p, _ll, _i, _p, _p, _i, _f, _p, _p, _p, _p, _ll, _p, _i, _f, _p, _i, _ll, _p]
+    prism_decay_chunks = [_i, _p, _p, _p, _ll, _i, _i, _i, _i, _i, _i, _i, _p, _i, _i, _f, _f, _f, _p, _p, _ll, _p, _i, _p, _i, _p, _i,
+                          _p, _p, _p, _p, _p, _ll, _p, _i, _f, _p, _p, _p, _ll, _p]
     prism_unit_removal = [_p, _p, _ll, _p, _i, _f, _i, _i, _i, _p, _p]
     prism_decay_from_exponent = [_p, _ll, _p, _i, _i, _i, _p]
     prism_lowrank_decay = [_p, _ll, _i, _p, _p, _i, _i, _i, _p, _ll, _i, _i, _p, _i, _i, _f, _p]
@@ -1940,87 +1942,184 @@ def recurrent_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
         "recurrent_scan")
 
 
-RETENTION_CHUNK = 64           # csrc/retention.cu: RET_CHUNK
-RETENTION_CHUNKED_FROM = int(os.environ.get("PRISM_RETENTION_CHUNKED_FROM", "16"))      # tokens of one request in a step
+DECAY_CHUNK = 64               # csrc/decayed_sum.cu: DS_CHUNK
+DECAY_CHUNKED_FROM = int(os.environ.get("PRISM_DECAY_CHUNKED_FROM", "16"))      # tokens of one request in a step
+DECAY_HEAD, DECAY_TOKEN, DECAY_CHANNEL = 0, 1, 2      # csrc/decayed_sum.cu: PRISM_DS_*
 
 
 def decay_powers(decay: torch.Tensor) -> torch.Tensor:
-    """``[H, RETENTION_CHUNK + 1]`` float32: powers 0, 1, .. of the float32 decays ``[H]``, formed in float64."""
-    n = torch.arange(RETENTION_CHUNK + 1, dtype=torch.float64, device=decay.device)
+    """``[H, DECAY_CHUNK + 1]`` float32: powers 0, 1, .. of the float32 decays ``[H]``, formed in float64."""
+    n = torch.arange(DECAY_CHUNK + 1, dtype=torch.float64, device=decay.device)
     return (decay.double()[:, None] ** n[None, :]).to(torch.float32).contiguous()
 
 
+class DecayedSum:
+    """One step of ``S <- D S + k v^T; o = S^T q`` for ``csrc/decayed_sum.cu``: ``q``, ``k`` (``[T, (H / rep) dk]``) and ``v [T, H dv]``
+    float32 column blocks with one row stride, ``state [slots, H, dv, dk]``, and what surrounds the recurrence.  ``kind``:
+    ``DECAY_HEAD`` with ``decay [H]`` and ``powers`` (``decay_powers``); ``DECAY_TOKEN`` with ``dt [T, H]``, ``dt_bias``, ``a_log``,
+    ``skip [H]``; ``DECAY_CHANNEL`` with ``low [T, R]``, ``a2t [R, H dk]``, ``a2_bias``, ``rate``.  ``silu``: q, k and v go through silu first; ``rot`` (a
+    ``RotaryParams`` or None) turns q and k; ``qmul`` / ``kmul``: factors on them.  With ``gate [T, H dv]`` the result is ``o / rms(o)
+    * weight * silu(gate)`` per head in the dtype of ``out [T, H dv]`` (``weight [dv]`` or None), without one ``o`` itself in float32."""
+
+    def __init__(self, kind: int, q, k, v, H: int, rep: int, dk: int, dv: int, state, out, gate=None, weight=None, eps: float = 0.0,
+                 silu: bool = False, rot=None, qmul: float = 1.0, kmul: float = 1.0, decay=None, powers=None, dt=None, dt_bias=None,
+                 a_log=None, skip=None, low=None, a2t=None, a2_bias=None, rate: float = 1.0):
+        T = q.shape[0]
+        _cuda(q, k, v, state, out, gate, weight, decay, powers, dt, dt_bias, a_log, skip, low, a2t, a2_bias)
+        for t in (q, k, v):
+            assert t.dtype == torch.float32 and t.dim() == 2 and t.shape[0] == T and t.stride(1) == 1
+            assert T == 1 or t.stride(0) == q.stride(0), "q, k and v rows must be equally far apart"
+        assert H % rep == 0 and q.shape[1] == k.shape[1] == (H // rep) * dk and v.shape[1] == H * dv
+        assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dv, dk)
+        assert out.shape == (T, H * dv) and out.stride(1) == 1
+        if gate is None:
+            assert out.dtype == torch.float32 and weight is None
+        else:
+            assert gate.dtype == torch.float32 and gate.shape == (T, H * dv) and gate.stride(1) == 1
+            assert weight is None or (weight.shape == (dv,) and weight.is_contiguous())
+        if kind == DECAY_HEAD:
+            assert decay.dtype == powers.dtype == torch.float32 and decay.shape == (H,) and powers.shape == (H, DECAY_CHUNK + 1)
+            assert powers.is_contiguous() and decay.is_contiguous()
+        elif kind == DECAY_TOKEN:
+            assert dt.dtype == torch.float32 and dt.shape == (T, H) and dt.stride(1) == 1 and not silu
+            assert all(x.shape == (H,) and x.is_contiguous() for x in (dt_bias, a_log)) and (skip is None or skip.shape == (H,))
+        else:
+            assert a2t.dtype == torch.float32 and a2t.is_contiguous() and a2t.shape[1] == H * dk and low.shape == (T, a2t.shape[0])
+            assert low.dtype == torch.float32 and low.stride(1) == 1 and (a2_bias is None or a2_bias.numel() == H * dk)
+        assert rot is None or kind == DECAY_HEAD
+        self.kind, self.q, self.k, self.v, self.T, self.H, self.rep, self.dk, self.dv = kind, q, k, v, T, H, rep, dk, dv
+        self.state, self.out, self.gate, self.weight, self.eps, self.silu = state, out, gate, weight, float(eps), bool(silu)
+        self.rd, self.freq = (rot.rotary_dim, rot.inv_freq) if rot is not None and rot.rotary_dim else (0, None)
+        self.il, self.amp = (rot.interleaved, rot.amplitude) if self.rd else (False, 1.0)
+        self.qmul, self.kmul = float(qmul), float(kmul)
+        self.decay, self.powers, self.dt, self.dt_bias, self.a_log, self.skip = decay, powers, dt, dt_bias, a_log, skip
+        self.low, self.a2t, self.a2_bias, self.rate = low, a2t, a2_bias, float(rate)
+
+    def path(self, ctx) -> str:
+        """``"step"``: one launch for a step of single tokens (it asks for the state before the kernel before it has ended, so
+        something that is not a kernel of this library - the copy of the step's descriptor - has to lie between two calls
+        on one state); ``"chunks"``: long stretches in bfloat16, on tensor cores; ``"scan"``: any size, token after token."""
+        L = lib()
+        if ctx.decode_only and L.prism_decay_step_supported(self.dk, self.dv) and self.state.data_ptr() % 16 == 0:
+            return "step"
+        ptrs = (self.q, self.k, self.v, self.out) + (() if self.gate is None else (self.gate,))
+        if (ctx.max_q_len >= DECAY_CHUNKED_FROM and (self.out.dtype if self.gate is not None else ctx.dtype) == torch.bfloat16
+                and L.prism_decay_chunks_supported(self.dk, self.dv, self.rd, 1 if self.il else 0) and not (self.rd and self.silu)
+                and all(t.data_ptr() % 16 == 0 for t in ptrs) and (self.T == 1 or self.q.stride(0) % 4 == 0)
+                and self.out.stride(0) % 2 == 0 and (self.gate is None or self.gate.stride(0) % 2 == 0)):
+            return "chunks"
+        return "scan"
+
+    def _dt(self, t):
+        return F32 if t is None else _dt(t)
+
+    def step(self, ctx):
+        assert self.T == ctx.S
+        one = self.T == 1
+        st = lambda t: 0 if t is None else t.stride(0)
+        _check(lib().prism_decay_step(
+            self.kind, _ptr(self.q), _ptr(self.k), _ptr(self.v), st(self.q), self.T, self.H, self.rep, self.dk, self.dv,
+            1 if self.silu else 0, _ptr(self.freq), self.rd, 1 if self.il else 0, float(self.amp), self.qmul, self.kmul, _ptr(self.decay),
+            _ptr(self.dt), st(self.dt), _ptr(self.dt_bias), self._dt(self.dt_bias), _ptr(self.a_log), self._dt(self.a_log),
+            _ptr(self.skip), self._dt(self.skip), _ptr(self.low), st(self.low), 0 if self.a2t is None else self.a2t.shape[0], _ptr(self.a2t),
+            _ptr(self.a2_bias), self._dt(self.a2_bias), self.rate, _ptr(self.state), _ptr(ctx.positions), _ptr(ctx.state_slots),
+            _ptr(self.gate), st(self.gate), _ptr(self.weight), self._dt(self.weight), self.eps, _ptr(self.out), _dt(self.out),
+            self.H * self.dv if one else self.out.stride(0), _stream()), "decay_step")
+
+    def chunks(self, ctx):
+        global launch_count
+        T, H = self.T, self.H
+        table = cum = fac = None
+        if self.rd:
+            key = ("rotary_table", self.freq.data_ptr())          # one table per step for all layers
+            table = ctx.scratch.get(key)
+            if table is None:
+                table = ctx.scratch[key] = ctx.alloc((T, self.rd // 2, 2), torch.float32)
+                rope_table(ctx.positions, self.freq, table)
+        n = T // DECAY_CHUNK + ctx.S
+        ws = ctx.alloc((n * H * self.dv * self.dk,), torch.float32)
+        if self.kind == DECAY_TOKEN:
+            fac = ctx.alloc((n * H,), torch.float32)
+        elif self.kind == DECAY_CHANNEL:
+            cum = ctx.alloc((T, H * self.dk), torch.float32)
+            lowrank_decay(self.low, self.a2t, self.a2_bias, cum, inner_tanh=False, epilogue=LR_LOGSIGPOW, rate=self.rate)
+        st = lambda t: 0 if t is None else t.stride(0)
+        _check(lib().prism_decay_chunks(
+            self.kind, _ptr(self.q), _ptr(self.k), _ptr(self.v), self.q.stride(0), T, ctx.S, H, self.rep, self.dk, self.dv,
+            1 if self.silu else 0, _ptr(table), self.rd, 1 if self.il else 0, float(self.amp), self.qmul, self.kmul, _ptr(self.powers),
+            _ptr(self.dt), st(self.dt), _ptr(self.dt_bias), self._dt(self.dt_bias), _ptr(self.a_log), self._dt(self.a_log),
+            _ptr(self.skip), self._dt(self.skip), _ptr(cum), _ptr(self.state), _ptr(ctx.seg_start), _ptr(ctx.state_slots),
+            _ptr(self.gate), st(self.gate), _ptr(self.weight), self._dt(self.weight), self.eps, _ptr(ws), _ptr(fac), _ptr(self.out),
+            self.out.stride(0), _stream()), "decay_chunks")
+        launch_count += 2
+
+    def scan(self, ctx):
+        """Token after token by ``recurrent_scan``; q, k and v are prepared in place."""
+        T, H, dk, dv, G = self.T, self.H, self.dk, self.dv, self.H // self.rep
+        q, k, v = self.q, self.k, self.v
+        if self.silu:
+            for t in (q, k, v):
+                activation(t, t, "silu")
+        for t, f in ((q, self.qmul), (k, self.kmul)):
+            if self.rd or f != 1.0:
+                t3 = t.view(T, G, dk)
+                rotate_slice(t3, t3, self.rd, self.freq, ctx.positions, self.il, self.amp, f)
+        o = self.out.view(T, H, dv) if self.gate is None and self.out.is_contiguous() else ctx.alloc((T, H, dv), torch.float32)
+        if self.kind == DECAY_HEAD:
+            recurrent_scan(SCAN_RETAIN, q, k, v, self.state, ctx, H, 1, dk, dv, o, w0=self.decay)
+        elif self.kind == DECAY_TOKEN:
+            bg = ctx.alloc((T, 2 * H), torch.float32)
+            step_sizes(self.dt, self.dt_bias, self.a_log, bg)
+            recurrent_scan(SCAN_TOKEN, q, k, v, self.state, ctx, H, self.rep, dk, dv, o, bg=bg, w0=self.skip)
+        else:
+            ww = ctx.alloc((T, H * dk), torch.float32)
+            lowrank_decay(self.low, self.a2t, self.a2_bias, ww, inner_tanh=False, epilogue=LR_SIGPOW, rate=self.rate)
+            recurrent_scan(SCAN_GATED, q, k, v, self.state, ctx, H, 1, dk, dv, o, ww=ww)
+        if self.gate is not None:
+            headnorm_gate(o, self.gate, self.weight if self.weight is not None else _ones(dv, q.device), self.eps, 1.0, self.out)
+        elif o.data_ptr() != self.out.data_ptr():
+            self.out.copy_(o.view(T, H * dv))
+
+    def run(self, ctx, path: Optional[str] = None):
+        """``path``: one of the three (tests and timing); None: chosen here."""
+        path = path or self.path(ctx)
+        {"step": self.step, "chunks": self.chunks, "scan": self.scan}[path](ctx)
+
+
+_ones_of = {}
+
+
+def _ones(n: int, device) -> torch.Tensor:
+    """A float32 vector of ones, made once per size and device."""
+    key = (n, str(device))
+    if key not in _ones_of:
+        _ones_of[key] = torch.ones(n, dtype=torch.float32, device=device)
+    return _ones_of[key]
+
+
 def retention(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, rot, decay: torch.Tensor, powers: torch.Tensor,
-              state: torch.Tensor, eps: float, ones: torch.Tensor, out: torch.Tensor, path: Optional[str] = None):
+              state: torch.Tensor, eps: float, out: torch.Tensor, path: Optional[str] = None):
     """Retention between its input and its output projection, for the step's tokens: from the float32 product ``proj [T,
     H (2 dk + 2 dv)]`` (columns q | k | v | gate), q and k rotated by ``rot`` (a ``RotaryParams`` or None) and k multiplied
     by ``dk^-1/2``, ``S <- decay[h] S + k v^T; o = S^T q`` from and into ``state [slots, H, dv, dk]``, ``out = o / rms(o) *
-    silu(gate)`` in the compute dtype.  ``powers``: ``decay_powers(decay)``; ``ones [dv]``.
-
-    ``path`` (None: chosen here): ``"step"`` one launch for a step of single tokens (it asks for the state before the kernel
-    before it has ended, so something that is not a kernel of this library - the copy of the step's descriptor - has to lie
-    between two calls on one state); ``"chunks"`` long stretches in bfloat16, on tensor cores; ``"scan"`` any
-    size, token after token (rotates q and k in place)."""
-    T, A, B = proj.shape[0], H * dk, H * dv
-    _cuda(proj, decay, powers, state, out)
-    assert proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[1] == 2 * A + 2 * B
-    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dv, dk)
-    assert decay.dtype == powers.dtype == torch.float32 and decay.shape == (H,) and powers.shape == (H, RETENTION_CHUNK + 1)
-    assert out.shape == (T, B) and out.stride(1) == 1 and powers.is_contiguous() and decay.is_contiguous()
-    rd, freq = (rot.rotary_dim, rot.inv_freq) if rot is not None and rot.rotary_dim else (0, None)
-    il, amp = (rot.interleaved, rot.amplitude) if rd else (False, 1.0)
-    L = lib()
-    if path is None:
-        if ctx.decode_only and L.prism_retention_step_supported(dk, dv):
-            path = "step"
-        elif (ctx.max_q_len >= RETENTION_CHUNKED_FROM and out.dtype == torch.bfloat16
-              and L.prism_retention_chunks_supported(dk, dv, rd, 1 if il else 0)):
-            path = "chunks"
-        else:
-            path = "scan"
-    if path == "step":
-        assert T == ctx.S
-        _check(L.prism_retention_step(_ptr(proj), proj.stride(0), A, 2 * A, 2 * A + B, T, H, dk, dv, _ptr(freq), rd, 1 if il else 0,
-                                      float(amp), dk ** -0.5, _ptr(decay), _ptr(state), _ptr(ctx.positions), _ptr(ctx.state_slots),
-                                      float(eps), _ptr(out), _dt(out), out.stride(0), _stream()), "retention_step")
-        return
-    if path == "chunks":
-        global launch_count
-        table = None
-        if rd:
-            key = ("rotary_table", freq.data_ptr())          # one table per step for all layers
-            table = ctx.scratch.get(key)
-            if table is None:
-                table = ctx.scratch[key] = ctx.alloc((T, rd // 2, 2), torch.float32)
-                rope_table(ctx.positions, freq, table)
-        ws = ctx.alloc(((T // RETENTION_CHUNK + ctx.S) * H * dv * dk,), torch.float32)
-        _check(L.prism_retention_chunks(_ptr(proj), proj.stride(0), A, 2 * A, 2 * A + B, T, ctx.S, H, dk, dv, _ptr(table), rd,
-                                        1 if il else 0, float(amp), dk ** -0.5, _ptr(powers), _ptr(state), _ptr(ctx.seg_start),
-                                        _ptr(ctx.state_slots), float(eps), _ptr(ws), _ptr(out), out.stride(0), _stream()),
-               "retention_chunks")
-        launch_count += 2
-        return
-    q, k = proj[:, :A].view(T, H, dk), proj[:, A:2 * A].view(T, H, dk)
-    if rd:
-        rotate_slice(q, q, rd, freq, ctx.positions, il, amp)
-    rotate_slice(k, k, rd, freq, ctx.positions, il, amp, dk ** -0.5)
-    o = ctx.alloc((T, H, dv), torch.float32)
-    recurrent_scan(SCAN_RETAIN, proj[:, :A], proj[:, A:2 * A], proj[:, 2 * A:2 * A + B], state, ctx, H, 1, dk, dv, o, w0=decay)
-    headnorm_gate(o, proj[:, 2 * A + B:], ones, eps, 1.0, out)
+    silu(gate)`` in the compute dtype.  ``powers``: ``decay_powers(decay)``; ``path``: see ``DecayedSum``."""
+    A, B = H * dk, H * dv
+    assert proj.shape[1] == 2 * A + 2 * B
+    DecayedSum(DECAY_HEAD, proj[:, :A], proj[:, A:2 * A], proj[:, 2 * A:2 * A + B], H, 1, dk, dv, state, out, gate=proj[:, 2 * A + B:],
+               eps=eps, rot=rot, kmul=dk ** -0.5, decay=decay, powers=powers).run(ctx, path)
 
 
 def lightning(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, decay: torch.Tensor, powers: torch.Tensor, state: torch.Tensor,
               weight: torch.Tensor, eps: float, out: torch.Tensor, path: Optional[str] = None):
     """Lightning attention between its input and its output projection: from the float32 product ``proj [T, H (2 dk + 2 dv)]``
     (columns q | k | v | gate), q, k and v through silu, ``S <- decay[h] S + k v^T; o = S^T q`` from and into ``state [slots,
-    H, dv, dk]``, ``out = rms(o over all heads) * weight * sigmoid(gate)`` in the compute dtype.  ``powers`` and ``path`` as in
-    ``retention`` (``"scan"`` puts q, k and v through silu in place)."""
-    T, A, B = proj.shape[0], H * dk, H * dv
-    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] == 2 * A + 2 * B
-    o = ctx.alloc((T, H, dv), torch.float32)
-    activation(proj[:, :2 * A + B], proj[:, :2 * A + B], "silu")
-    recurrent_scan(SCAN_RETAIN, proj[:, :A], proj[:, A:2 * A], proj[:, 2 * A:2 * A + B], state, ctx, H, 1, dk, dv, o, w0=decay)
-    part_norm_gate(o.view(T, B), proj[:, 2 * A + B:], weight, eps, 1, out, "sigmoid")
+    H, dv, dk]``, ``out = rms(o over all heads) * weight * sigmoid(gate)`` in the compute dtype.  ``powers``, ``path``: as above."""
+    A, B = H * dk, H * dv
+    assert proj.shape[1] == 2 * A + 2 * B
+    o = ctx.alloc((proj.shape[0], B), torch.float32)
+    DecayedSum(DECAY_HEAD, proj[:, :A], proj[:, A:2 * A], proj[:, 2 * A:2 * A + B], H, 1, dk, dv, state, o, silu=True, decay=decay,
+               powers=powers).run(ctx, path)
+    part_norm_gate(o, proj[:, 2 * A + B:], weight, eps, 1, out, "sigmoid")
 
 
 def gated_linear(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, a2t: torch.Tensor, a2_bias: torch.Tensor, rate: float,
@@ -2028,16 +2127,12 @@ def gated_linear(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, a2t: torch.T
     """Gated linear attention between its input and its output projection: from the float32 product ``proj [T, H (2 dk + 2
     dv) + R]`` (columns q | k | v | gate | the decay's low-rank part), ``w = sigmoid(low @ a2t + a2_bias)^rate``, ``S <- diag(w) S
     + k v^T; o = S^T q dk^-1/2`` from and into ``state [slots, H, dv, dk]``, ``out = rms(o per head) * weight * silu(gate)`` in
-    the compute dtype.  ``a2t [R, H dk]`` float32, ``weight [dv]``; ``path`` as in ``retention``."""
-    T, A, B, R = proj.shape[0], H * dk, H * dv, a2t.shape[0]
-    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] == 2 * A + 2 * B + R
-    q, k, v, gate, low = proj[:, :A], proj[:, A:2 * A], proj[:, 2 * A:2 * A + B], proj[:, 2 * A + B:2 * A + 2 * B], proj[:, 2 * A + 2 * B:]
-    ww = ctx.alloc((T, A), torch.float32)
-    lowrank_decay(low, a2t, a2_bias, ww, inner_tanh=False, epilogue=LR_SIGPOW, rate=rate)
-    rotate_slice(q.view(T, H, dk), q.view(T, H, dk), 0, None, ctx.positions, False, 1.0, dk ** -0.5)
-    o = ctx.alloc((T, H, dv), torch.float32)
-    recurrent_scan(SCAN_GATED, q, k, v, state, ctx, H, 1, dk, dv, o, ww=ww)
-    headnorm_gate(o, gate, weight, eps, 1.0, out)
+    the compute dtype.  ``a2t [R, H dk]`` float32, ``weight [dv]``; ``path``: as above."""
+    A, B = H * dk, H * dv
+    assert proj.shape[1] == 2 * A + 2 * B + a2t.shape[0]
+    DecayedSum(DECAY_CHANNEL, proj[:, :A], proj[:, A:2 * A], proj[:, 2 * A:2 * A + B], H, 1, dk, dv, state, out,
+               gate=proj[:, 2 * A + B:2 * A + 2 * B], weight=weight, eps=eps, qmul=dk ** -0.5, low=proj[:, 2 * A + 2 * B:], a2t=a2t,
+               a2_bias=a2_bias, rate=rate).run(ctx, path)
 
 
 def state_space(ctx, u: torch.Tensor, dt: torch.Tensor, z: torch.Tensor, H: int, G: int, N: int, dv: int, dt_bias: torch.Tensor,
@@ -2046,14 +2141,13 @@ def state_space(ctx, u: torch.Tensor, dt: torch.Tensor, z: torch.Tensor, H: int,
     """A state-space mixer behind its convolution: ``u [T, H dv + 2 G N]`` float32 (columns x | B | C; head h reads group ``h //
     (H / G)`` of B and C), step sizes ``d = softplus(dt + dt_bias)`` from ``dt [T, H]``, ``S <- exp(-exp(a_log) d) S + d B x^T; y =
     S^T C + skip x`` from and into ``state [slots, H, dv, N]``, ``out = rms(y * silu(z) in ``parts`` equal parts) * weight * scale``
-    in the compute dtype.  ``dt`` and ``z [T, H dv]`` float32 with row strides of their own; ``path`` as in ``retention``."""
-    T, B, rep = u.shape[0], H * dv, H // G
-    assert u.dtype == torch.float32 and u.is_contiguous() and u.shape[1] == B + 2 * G * N
-    o = ctx.alloc((T, H, dv), torch.float32)
-    bg = ctx.alloc((T, 2 * H), torch.float32)
-    step_sizes(dt, dt_bias, a_log, bg)
-    recurrent_scan(SCAN_TOKEN, u[:, B + G * N:], u[:, B:B + G * N], u[:, :B], state, ctx, H, rep, N, dv, o, bg=bg, w0=skip)
-    part_norm_gate(o.view(T, B), z, weight, eps, parts, out, "silu", gate_first=True, scale=scale)
+    in the compute dtype.  ``dt`` and ``z [T, H dv]`` float32 with row strides of their own; ``path``: as above."""
+    B = H * dv
+    assert u.shape[1] == B + 2 * G * N
+    o = ctx.alloc((u.shape[0], B), torch.float32)
+    DecayedSum(DECAY_TOKEN, u[:, B + G * N:], u[:, B:B + G * N], u[:, :B], H, H // G, N, dv, state, o, dt=dt, dt_bias=dt_bias,
+               a_log=a_log, skip=skip).run(ctx, path)
+    part_norm_gate(o, z, weight, eps, parts, out, "silu", gate_first=True, scale=scale)
 
 
 def unit_removal(k: torch.Tensor, a: torch.Tensor, a_bias: Optional[torch.Tensor], unit_eps: float, H: int, dk: int,

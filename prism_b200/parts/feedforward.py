@@ -145,7 +145,7 @@ class MixtureOfExperts(FeedForward):
         if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups:
             raise ValueError(f"{self.experts} experts in {self.groups} groups of which {self.keep} are kept: the groups must "
                              f"be equal and at least one kept")
-        if self.keep * (self.experts // self.groups) < self.top:
+        if self.keep * (self.routed // self.groups) < self.top:
             raise ValueError(f"{self.keep} groups of {self.experts // self.groups} experts hold fewer than the {self.top} "
                              f"experts a token uses")
         self.weight_scale, self.sum_eps = float(weight_scale), float(sum_eps)

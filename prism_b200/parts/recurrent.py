@@ -332,7 +332,6 @@ class RetentionMixer(Mixer):
     def on_bound(self):
         self.decays = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(self.device)
         self.powers = ops.decay_powers(self.decays)
-        self.ones = torch.ones(self.dv, dtype=torch.float32, device=self.device)
         self.rot = self.position.rotary() if self.position is not None else None
         if self.position is not None and (self.rot is None or self.rot.rotary_dim > self.dk):
             raise ConfigError(f"retention takes a rotary position encoding of at most head_dim {self.dk} entries")
@@ -342,7 +341,7 @@ class RetentionMixer(Mixer):
         T, H, dk, dv, A, B = x.shape[0], self.H, self.dk, self.dv, self.H * self.dk, self.H * self.dv
         proj = ops.linear(x, self.w["in_w"], None, out_dtype=torch.float32)          # q | k | v | g
         inner = ctx.alloc((T, B), ctx.dtype)
-        ops.retention(ctx, proj, H, dk, dv, self.rot, self.decays, self.powers, state.state, self.eps, self.ones, inner)
+        ops.retention(ctx, proj, H, dk, dv, self.rot, self.decays, self.powers, state.state, self.eps, inner)
         return ops.linear_delta(inner, self.w["o_w"], None, f32=True)
 
 

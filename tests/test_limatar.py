@@ -191,6 +191,6 @@ def test_k_shares_of_paired_products_and_experts():
 def test_powers_of_a_decay():
     from prism_b200 import ops
     p = ops.decay_powers(torch.tensor([0.0, 0.5, 1.0, 0.99951171875]))
-    assert p.shape == (4, ops.RETENTION_CHUNK + 1) and p.dtype == torch.float32
-    assert p[0].tolist() == [1.0] + [0.0] * ops.RETENTION_CHUNK and float(p[1, 3]) == 0.125 and float(p[2].min()) == 1.0
+    assert p.shape == (4, ops.DECAY_CHUNK + 1) and p.dtype == torch.float32
+    assert p[0].tolist() == [1.0] + [0.0] * ops.DECAY_CHUNK and float(p[1, 3]) == 0.125 and float(p[2].min()) == 1.0
     assert abs(float(p[3, 64]) - 0.99951171875 ** 64) < 1e-7

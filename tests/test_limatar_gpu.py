@@ -201,9 +201,9 @@ def test_retention_in_pieces_on_every_path(H, dk, dv, rot, pairs, sizes):
         q, k, v = turn(x[:, :A].view(n, H, dk)), turn(x[:, A:2 * A].view(n, H, dk)) * dk ** -0.5, x[:, 2 * A:2 * A + B].view(n, H, dv)
         o = torch.stack([LP.rms(LP.retain(q[:, i], k[:, i], v[:, i], decay[i]), 1e-6) for i in range(H)], 1)
         refs.append(o.reshape(n, B) * LP.silu(x[:, 2 * A + B:]))
-    dd, ones = torch.tensor(decay, device=DEV), torch.ones(dv, device=DEV)
+    dd = torch.tensor(decay, device=DEV)
     powers = ops.decay_powers(dd)
-    chunks = bool(ops.lib().prism_retention_chunks_supported(dk, dv, rot, 1 if pairs else 0))
+    chunks = bool(ops.lib().prism_decay_chunks_supported(dk, dv, rot, 1 if pairs else 0))
     for path, dt in (("scan", torch.float32), ("scan", torch.bfloat16), (None, torch.float32), (None, torch.bfloat16)) + \
             ((("chunks", torch.bfloat16),) if chunks else ()):
         state = torch.zeros(4, H, dv, dk, device=DEV)
@@ -213,7 +213,7 @@ def test_retention_in_pieces_on_every_path(H, dk, dv, rot, pairs, sizes):
             ctx = step_ctx([n for _, _, n in live], [(2, 0, 3)[s] for s, _, _ in live], [a for _, a, _ in live])
             x = torch.cat([xs[s][a:a + n] for s, a, n in live]).to(DEV)
             out = torch.empty(x.shape[0], B, dtype=dt, device=DEV)
-            ops.retention(ctx, x, H, dk, dv, rp, dd, powers, state, 1e-6, ones, out, path=path)
+            ops.retention(ctx, x, H, dk, dv, rp, dd, powers, state, 1e-6, out, path=path)
             o = 0
             for s, a, n in live:
                 got[s][a:a + n] = out[o:o + n].float().cpu()
@@ -242,8 +242,7 @@ def test_an_old_token_comes_back_through_the_state_of_many_chunks():
     for path, dt in (("scan", torch.float32), ("chunks", torch.bfloat16)):
         state = torch.zeros(1, H, d, d, device=DEV)
         out = torch.empty(n, d, dtype=dt, device=DEV)
-        ops.retention(step_ctx([n], [0]), x.to(DEV), H, d, d, None, decay, ops.decay_powers(decay), state, 1e-12, torch.ones(d, device=DEV), out,
-                      path=path)
+        ops.retention(step_ctx([n], [0]), x.to(DEV), H, d, d, None, decay, ops.decay_powers(decay), state, 1e-12, out, path=path)
         for t in (3, 63, 64, 200, 329):
             assert float((out[t].cpu().double() - ref).abs().max()) <= 1e-2, (path, t)
         assert float(out[2].abs().max()) == 0.0              # nothing to read before token 3
