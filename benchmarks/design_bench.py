@@ -1,10 +1,10 @@
-"""Prefill and decode throughput of the Dolezen, the Pofazen, the Zuvulorn, the Tagelorn or the Limatar design at layer sizes that resemble real models
+"""Prefill and decode throughput of the Dolezen, the Pofazen, the Zuvulorn, the Tagelorn, the Limatar or the Nivotar design at layer sizes that resemble real models
 (random weights, bf16), beside the Qwen2 architecture at equal width, depth and parameter count (Tagelorn also beside
 Zuvulorn, the closest of the other designs: attention with a sink, a delta rule with a decay per key channel, experts; Limatar
-beside Dolezen: latent attention), and the
+beside Dolezen: latent attention; Nivotar beside Limatar: decayed sums of outer products, limited experts), and the
 design's own kernels beside the like kernels on the same problem with their fractions of the measured peaks.
 
-    python bench.py --design dolezen|pofazen|zuvulorn|tagelorn|limatar [--sizes 2k,4k] [--steps K] [--warmup W]
+    python bench.py --design dolezen|pofazen|zuvulorn|tagelorn|limatar|nivotar [--sizes 2k,4k] [--steps K] [--warmup W]
     python benchmarks/design_bench.py [--design pofazen] [--sizes 2k] [--kernels-only] [--once KERNEL]
 
 One JSON line.  Timing: CUDA events after W >= 3 warm-up runs; every timed step reads all weights (more than
@@ -766,11 +766,164 @@ def limatar_kernel_numbers(s, pk, once=None):
     return out
 
 
+GLA_RANK = 16
+NIV_IDENTITY = 2
+
+
+def nivotar_ssm(s):
+    """The state-space half of a side-by-side layer: as many inner channels as the model is wide, heads of 64, a state of 128."""
+    return dict(heads=s["width"] // 64, vdim=64, state=128, groups=4, conv=4, norm_groups=4)
+
+
+def nivotar_config(s):
+    """Layers: gated linear attention, windowed attention beside a state-space mixer, gated linear attention, lightning
+    attention, ...; dense feed-forwards with biases and 8 limited experts beside 2 identity experts (2 a token) in turn."""
+    left = dict(heads=s["heads"], kv_heads=s["kv_heads"], dim=s["dim"], vdim=s["vdim"], scale=s["dim"] ** -0.5, mask=dict(size=s["window"]),
+                rot=dict(base=10000.0, dims=s["dim"]))
+    par = dict(left=left, right=nivotar_ssm(s), left_scale=0.7, right_scale=0.7)
+    gl = dict(heads=s["heads"], dim=s["dim"], vdim=s["vdim"], tau=16.0, decay_rank=GLA_RANK)
+    lightning = dict(heads=s["heads"], dim=s["dim"], vdim=s["vdim"], decay=[1.0 - 2.0 ** (-5 - i % 8) for i in range(s["heads"])])
+    dense = dict(kind="dense", ff=s["ff"] * 2 // 3 // 256 * 256)
+    routed = dict(kind="moe", expert=dict(ff=moe_ff(s), limit=7.0), router=dict(experts=MOE_EXPERTS, top=MOE_TOP, identity=NIV_IDENTITY))
+    layers = []
+    for i in range(s["layers"]):
+        kind, mixer = (("gla", gl), ("parallel", par), ("gla", gl), ("lightning", lightning))[i % 4]
+        layers.append(dict(type=kind, mixer=dict(mixer), mlp=dense if i % 2 == 0 else routed))
+    return dict(architecture="Nivotar", vocab=s["vocab"], width=s["width"], norm=dict(eps=1e-6), layers=layers, max_positions=8192)
+
+
+def nivotar_kernel_numbers(s, pk, once=None):
+    """The design's kernels alone, each beside the like kernel of the closest model on the same problem: the three decayed
+    sums between their projections beside retention (Limatar's); windowed attention on its own plane beside Qwen2's kernels; limited experts
+    with identity experts beside gated experts; the dense layer with biases beside the one without; norm of a result and sum beside norm,
+    sum and norm; the convolution with bias and silu beside the one without."""
+    from prism_b200 import ops
+    from prism_b200.parts.base import RotaryParams
+    out = {}
+    T = 2048
+    W = s["width"]
+    shapes = (("prefill_2048", 1, 0, T), ("decode_b8", 8, T - 1, 1), ("decode_b64", 64, T - 1, 1))
+
+    def run(name, fn, flops, nbytes, fp32=False):
+        if once:
+            if once == name:
+                for _ in range(3):
+                    fn()
+                torch.cuda.synchronize()
+            return
+        ms = timeit(graphed(fn))          # as in a decode step; several launches make up some of these
+        if fp32:
+            out[name] = dict(us=round(ms * 1e3, 1), fp32_tflops=round(flops / ms / 1e9, 2), gbs=round(nbytes / ms / 1e6, 1),
+                             frac_hbm_of_measured=round(nbytes / ms / 1e6 / pk["hbm_gbs"], 4))
+        else:
+            out[name] = _rates(ms, flops, nbytes, pk)
+
+    # the decayed sums: everything between the input and the output projection
+    H, dk, dv = s["heads"], s["dim"], s["vdim"]
+    A, B, R = H * dk, H * dv, GLA_RANK
+    rot = RotaryParams((10000.0 ** (-torch.arange(0, dk, 2).float() / dk)).to(DEV), dk, False)
+    decay = torch.tensor([1.0 - 2.0 ** (-5 - i % 8) for i in range(H)], device=DEV)
+    powers = ops.decay_powers(decay)
+    a2t, a2b = torch.randn(R, A, device=DEV) / R ** 0.5, torch.randn(A, device=DEV) + 2.0
+    wh, wb = torch.ones(dv, device=DEV), torch.ones(B, device=DEV)
+    m = nivotar_ssm(s)
+    Hs, ds, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+    C = Hs * ds + 2 * G * N
+    dtb, alog, skip, ws = torch.randn(Hs, device=DEV) - 3.0, torch.randn(Hs, device=DEV), torch.ones(Hs, device=DEV), torch.ones(Hs * ds, device=DEV)
+    taps, cb = torch.randn(C, m["conv"], device=DEV, dtype=torch.bfloat16), torch.zeros(C, device=DEV)
+    taps_t = taps.float().t().contiguous()
+    for label, batch, cached, q_len in shapes:
+        Tt = batch * q_len
+        c = types.SimpleNamespace(seg_start=(torch.arange(batch + 1, dtype=torch.int32) * q_len).to(DEV), S=batch, max_q_len=q_len,
+                                  tok_seg=torch.arange(batch, dtype=torch.int32).repeat_interleave(q_len).to(DEV),
+                                  state_slots=torch.arange(batch, dtype=torch.int32, device=DEV), decode_only=q_len == 1, scratch={},
+                                  positions=torch.arange(cached, cached + q_len, dtype=torch.int32).repeat(batch).to(DEV), dtype=torch.bfloat16,
+                                  alloc=lambda shape, dtype: torch.empty(shape, dtype=dtype, device=DEV))
+        state = torch.zeros(batch + 1, H, dv, dk, device=DEV)
+        proj = torch.randn(Tt, 2 * (A + B) + R, device=DEV) * 0.3
+        plain = torch.randn(Tt, 2 * (A + B), device=DEV) * 0.3
+        o = torch.empty(Tt, B, device=DEV, dtype=torch.bfloat16)
+        flops, nbytes = 4 * Tt * H * dk * dv, 4 * (2 * batch * H * dk * dv + Tt * 2 * (A + B)) + 2 * Tt * B
+        run(f"gated_linear_{label}", lambda: ops.gated_linear(c, proj, H, dk, dv, a2t, a2b, 1.0 / 16.0, state, wh, 1e-6, o), flops,
+            nbytes + 4 * Tt * R, fp32=True)
+        run(f"lightning_{label}", lambda: ops.lightning(c, plain, H, dk, dv, decay, powers, state, wb, 1e-6, o), flops, nbytes, fp32=True)
+        run(f"like_retention_{label}", lambda: ops.retention(c, plain, H, dk, dv, rot, decay, powers, state, 1e-6, o), flops, nbytes, fp32=True)
+        sstate = torch.zeros(batch + 1, Hs, ds, N, device=DEV)
+        u, z, dt = torch.randn(Tt, C, device=DEV) * 0.5, torch.randn(Tt, Hs * ds, device=DEV), torch.randn(Tt, Hs, device=DEV)
+        os_ = torch.empty(Tt, Hs * ds, device=DEV, dtype=torch.bfloat16)
+        run(f"state_space_{label}", lambda: ops.state_space(c, u, dt, z, Hs, G, N, ds, dtb, alog, skip, sstate, ws, 1e-6, m["norm_groups"], 0.7,
+                                                            os_), 4 * Tt * Hs * ds * N,
+            4 * (2 * batch * Hs * ds * N + Tt * (C + Hs * ds + Hs)) + 2 * Tt * Hs * ds, fp32=True)
+        tail = torch.zeros(batch + 1, m["conv"] - 1, C, device=DEV)
+        y = torch.empty(Tt, C, device=DEV)
+        cbytes = 8 * Tt * C + (8 * (m["conv"] - 1) * batch * C if q_len == 1 else 0)
+        run(f"conv_silu_{label}", lambda: ops.causal_conv(u, taps, cb, tail, c, y, move_tail=q_len == 1, taps_t=taps_t, silu=True), 0, cbytes, fp32=True)
+        run(f"like_conv_{label}", lambda: ops.causal_conv(u, taps, None, tail, c, y, move_tail=q_len == 1, taps_t=taps_t), 0, cbytes, fp32=True)
+    # windowed attention through the general path (float32 projection, norm over the whole projection, keys and values of one size)
+    nh, nkv, win = s["heads"], s["kv_heads"], s["window"]
+    mask = ops.KeyMask.window(win)
+    wq, wk = torch.ones(nh * dk, device=DEV), torch.ones(nkv * dk, device=DEV)
+    for label, batch, cached, q_len in shapes:
+        c, kc, vc, bt, npages = paged(batch, cached, q_len, nkv, dk, dk)
+        Tt = batch * q_len
+        q = torch.randn(Tt, nh, dk, device=DEV, dtype=torch.bfloat16)
+        o = torch.empty(Tt, nh * dk, device=DEV, dtype=torch.bfloat16)
+        pairs = batch * sum(min(p + 1, win) for p in range(cached, cached + q_len))
+        keys = batch * (min(cached + q_len, win) if q_len == 1 else cached + q_len)
+        flops, nbytes = 4 * pairs * nh * dk, 2 * (keys * nkv * 2 * dk + 2 * Tt * nh * dk)
+        run(f"window_{label}", lambda: ops.masked_attention(c, q, o, kc, vc, bt, npages, mask, dk ** -0.5), flops, nbytes)
+        if q_len == 1:
+            ns = ops.decode_splits(batch, nkv, cached + 1, win)
+            po, pml = torch.empty(batch, nh, ns, dk, device=DEV), torch.empty(batch, nh, ns, 2, device=DEV)
+            run(f"qwen2_window_{label}", lambda: ops.attention_decode_bf16(q, o, kc, vc, bt, c.positions, c.tok_seg, npages, win,
+                                                                           dk ** -0.5, ns, po, pml, c.err), flops, nbytes)
+        else:
+            run(f"qwen2_window_tcgen05_{label}", lambda: ops.attention_prefill_tc(q, o, kc, vc, bt, c.seg_start, c.cached_len, q_len,
+                                                                                  npages, win, dk ** -0.5, c.err), flops, nbytes)
+        x = torch.randn(Tt, (nh + 2 * nkv) * dk, device=DEV)
+        rbytes = 4 * x.numel() + 2 * x.numel()
+        run(f"norm_rope_store_{label}", lambda: ops.qk_norm_rope_store(
+            x[:, :nh * dk], x[:, nh * dk:(nh + nkv) * dk], x[:, (nh + nkv) * dk:], wq, wk, 1e-6, rot.inv_freq, dk, q, kc, vc, bt, c.positions,
+            c.tok_seg, npages, 8192, c.err, whole=True, halves=True, v_scale=0.7), 0, rbytes, fp32=True)
+        run(f"like_norm_rope_store_{label}", lambda: ops.qk_norm_rope_store(
+            x[:, :nh * dk], x[:, nh * dk:(nh + nkv) * dk], x[:, (nh + nkv) * dk:], wh, wh, 1e-6, rot.inv_freq, dk, q, kc, vc, bt, c.positions,
+            c.tok_seg, npages, 8192, c.err, halves=True), 0, rbytes, fp32=True)
+    # feed-forwards
+    E, top, F = MOE_EXPERTS, MOE_TOP, moe_ff(s)
+    Fd = s["ff"] * 2 // 3 // 256 * 256
+    mk = lambda *sh: torch.randn(*sh, device=DEV, dtype=torch.bfloat16) / sh[-1] ** 0.5
+    gu, dn, gud, dnd = mk(E, 2 * F, W), mk(E, W, F), mk(2 * Fd, W), mk(W, Fd)
+    gb, db = mk(2 * Fd), mk(W)
+    choice = ops.MoeChoice(torch.randn(E + NIV_IDENTITY, device=DEV) * 0.02)
+    actx = types.SimpleNamespace(alloc=lambda shape, dtype: torch.empty(shape, dtype=dtype, device=DEV))
+    for label, Tt in (("prefill_2048", T), ("decode_b8", 8), ("decode_b64", 64)):
+        xx, own = torch.randn(Tt, W, device=DEV, dtype=torch.bfloat16), torch.randn(Tt, W, device=DEV)
+        logits = torch.randn(Tt, E + NIV_IDENTITY, device=DEV)
+        chosen = torch.topk(torch.softmax(logits, -1) + choice.correction, top).indices
+        real, used = int((chosen < E).sum()), int(chosen[chosen < E].unique().numel())
+        run(f"limited_experts_with_identity_{label}", lambda: ops.moe_feed_forward(actx, xx, logits, gu, dn, top, True, False, False, "clamped",
+                                                                                   choice=choice, limit=7.0, own=own),
+            6 * real * F * W, 2 * 3 * used * F * W + Tt * W * (2 + 4 * top) + 4 * (Tt * top - real) * W)
+        few = logits[:, :E].contiguous()
+        run(f"like_gated_experts_{label}", lambda: ops.moe_feed_forward(actx, xx, few, gu, dn, top), 6 * Tt * top * F * W,
+            2 * (3 * min(E, Tt * top) * F * W + Tt * W * (1 + 2 * top)))
+        run(f"feed_forward_with_biases_{label}", lambda: ops.feed_forward_glu(actx, xx, gud, dnd, "silu", 0.0, gb, db), 6 * Tt * Fd * W,
+            2 * (3 * Fd * W + 3 * Tt * W))
+        run(f"qwen2_feed_forward_{label}", lambda: ops.feed_forward_swiglu(actx, xx, gud, dnd), 6 * Tt * Fd * W,
+            2 * (3 * Fd * W + 3 * Tt * W))
+    wn = torch.ones(W, device=DEV)
+    for label, Tt in (("prefill_2048", T), ("decode_b64", 64)):
+        h, d, x1 = torch.empty(Tt, W, device=DEV, dtype=torch.bfloat16), torch.randn(Tt, W, device=DEV), torch.randn(Tt, W, device=DEV)
+        run(f"norm_sum_copy_{label}", lambda: ops.add_normed_rmsnorm(x1, d, wn, 1e-6, None, 0.0, h), 0, 4 * Tt * W * 3 + 2 * Tt * W, fp32=True)
+        run(f"like_norm_sum_norm_{label}", lambda: ops.add_normed_rmsnorm(x1, d, wn, 1e-6, wn, 1e-6, h), 0, 4 * Tt * W * 3 + 2 * Tt * W, fp32=True)
+    return out
+
+
 DESIGNS = {"dolezen": (dolezen_config, kernel_numbers), "pofazen": (pofazen_config, pofazen_kernel_numbers),
            "zuvulorn": (zuvulorn_config, zuvulorn_kernel_numbers), "tagelorn": (tagelorn_config, tagelorn_kernel_numbers),
-           "limatar": (limatar_config, limatar_kernel_numbers)}
+           "limatar": (limatar_config, limatar_kernel_numbers), "nivotar": (nivotar_config, nivotar_kernel_numbers)}
 # designs measured beside another design as well as beside Qwen2: the closest of the models that ran before
-BESIDE = {"tagelorn": ("zuvulorn", zuvulorn_config), "limatar": ("dolezen", dolezen_config)}
+BESIDE = {"tagelorn": ("zuvulorn", zuvulorn_config), "limatar": ("dolezen", dolezen_config), "nivotar": ("limatar", limatar_config)}
 
 
 def run(sizes, steps, warmup, prompt_len=2048, batch=8, kernels_only=False, once=None, peaks=None, design="dolezen"):

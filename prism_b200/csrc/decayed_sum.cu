@@ -33,10 +33,17 @@
 namespace prism {
 
 constexpr int DS_CHUNK = 64;
-constexpr int DS_SUB = 16;                 // a sub-chunk: the rows one warp of the output kernel owns
-constexpr float DS_MAX_SPAN = 60.f;        // the most a sub-chunk's log decays may sum to before its scores are formed term by term
+constexpr int DS_SUB = 16;                 // a sub-chunk: the rows a pair of warps of the output kernel owns
+constexpr float DS_MAX_SPAN = 80.f;        // the most a sub-chunk's log decays (in units of ln 2) may sum to before its scores are formed
+                                           // term by term
 
 __device__ __forceinline__ float ds_silu(float z) { return z / (1.f + expf(-z)); }
+// 2^x by the special-function unit (results below 2^-126 are zero)
+__device__ __forceinline__ float ds_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ float ds_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // ---------------------------------------------------------------------------------------------------------
@@ -226,7 +233,15 @@ struct DecayChunks {
     long long dts;
     const void *dt_bias, *a_log, *skip;
     int dt_bias_bf16, a_log_bf16, skip_bf16;
-    float* cum;              // DS_CHANNEL: [T, H dk] log decays; the first kernel leaves their sums from each chunk's start on
+    const float* low;        // DS_CHANNEL: [T, R] (row stride ls); log decay = rate log sigmoid(low a2t + a2_bias), a2t [R, H dk]
+    long long ls;
+    int R;
+    const float* a2t;
+    const void* a2_bias;
+    int a2_bias_bf16;
+    float rate;
+    float* cum;              // DS_CHANNEL: [T, H dk]: the first kernel leaves the log decays' sums from each chunk's start on here,
+                             // in units of ln 2
     float* state;            // [slots, H, dv, dk]
     const int* seg_start;
     const int* slots;
@@ -395,21 +410,52 @@ __global__ void __launch_bounds__(DS_STATE_THREADS) decay_chunk_state_kernel(con
         const size_t cs = (size_t)a.H * dk;
         float sum = 0.f;
         constexpr int U = 8;
-        if (on)
-            for (int r = r0; r < r1; r += U) {
-                float x[U];
-#pragma unroll
-                for (int u = 0; u < U; ++u) x[u] = r + u < r1 ? cum[(size_t)(r + u) * cs] : 0.f;
-#pragma unroll
-                for (int u = 0; u < U; ++u) sum += x[u];
+        {
+            // the chunk's low-rank rows lie where the values' tile will be; eight tokens' products side by side
+            float* s_low = reinterpret_cast<float*>(vh);
+            const int RT = min(a.R, vs);                                  // entries of a row that fit (all of them but for large ranks)
+            const float* low = pdl_fresh(a.low) + (size_t)t0 * a.ls;
+            for (int i = tid; i < DS_CHUNK * RT; i += DS_STATE_THREADS) {
+                const int r = i / RT, c = i - r * RT;
+                s_low[c * DS_CHUNK + r] = r < n ? low[(size_t)r * a.ls + c] : 0.f;
             }
+            __syncthreads();
+            const float* w2 = a.a2t + (size_t)h * dk + d;
+            const float bias = on && a.a2_bias != nullptr ? load_param(a.a2_bias, a.a2_bias_bf16, (size_t)h * dk + d) : 0.f;
+            const float scale = -a.rate * 1.44269504f;
+            if (on)
+                for (int r = r0; r < r1; r += U) {
+                    float z[U];
+#pragma unroll
+                    for (int u = 0; u < U; ++u) z[u] = bias;
+                    for (int c = 0; c < RT; ++c) {
+                        const float w = w2[(size_t)c * cs];
+                        const float4 x0 = *reinterpret_cast<const float4*>(s_low + c * DS_CHUNK + r);
+                        const float4 x1 = *reinterpret_cast<const float4*>(s_low + c * DS_CHUNK + r + 4);
+                        z[0] += w * x0.x; z[1] += w * x0.y; z[2] += w * x0.z; z[3] += w * x0.w;
+                        z[4] += w * x1.x; z[5] += w * x1.y; z[6] += w * x1.z; z[7] += w * x1.w;
+                    }
+                    for (int c = RT; c < a.R; ++c) {
+                        const float w = w2[(size_t)c * cs];
+#pragma unroll
+                        for (int u = 0; u < U; ++u)
+                            if (r + u < r1) z[u] += w * low[(size_t)(r + u) * a.ls + c];
+                    }
+#pragma unroll
+                    for (int u = 0; u < U; ++u)
+                        if (r + u < r1) {
+                            sum += scale * ds_softplus(-z[u]);
+                            cum[(size_t)(r + u) * cs] = sum;                 // so far: from the run's first row on
+                        }
+                }
+        }
         s_part[tid] = sum;
         __syncthreads();
         if (on) {
-            float acc = 0.f, total = 0.f;
+            float before = 0.f, total = 0.f;
             for (int i = 0; i < runs; ++i) {
                 const float s = s_part[i * dkw + d];
-                if (i < g) acc += s;
+                if (i < g) before += s;
                 total += s;
             }
             for (int r = r0; r < min(DS_CHUNK, r0 + per); r += U) {
@@ -423,9 +469,9 @@ __global__ void __launch_bounds__(DS_STATE_THREADS) decay_chunk_state_kernel(con
 #pragma unroll
                 for (int u = 0; u < U; ++u) {
                     if (r + u >= min(DS_CHUNK, r0 + per)) continue;
-                    acc += x[u];
+                    const float acc = before + x[u];
                     if (r + u < r1) cum[(size_t)(r + u) * cs] = acc;
-                    const float w = r + u < r1 ? (a.act ? ds_silu(y[u]) : y[u]) * a.kmul * expf(total - acc) : 0.f;
+                    const float w = r + u < r1 ? (a.act ? ds_silu(y[u]) : y[u]) * a.kmul * ds_exp2(total - acc) : 0.f;
                     const __nv_bfloat16 hi = __float2bfloat16_rn(w);
                     kh[(r + u) * ks + d] = hi;
                     kl[(r + u) * ks + d] = __float2bfloat16_rn(w - __bfloat162float(hi));
@@ -452,7 +498,7 @@ __global__ void __launch_bounds__(DS_STATE_THREADS) decay_chunk_state_kernel(con
     ds_batches<8, DS_STATE_THREADS, float4>(DS_CHUNK, vq, [&](int r, int d) {
         return *reinterpret_cast<const float4*>(vx + (size_t)(t0 + min(r, n - 1)) * a.xs + (d < dv ? d : 0));
     }, [&](int r, int d, float4 v) {
-        ds_split4(r < n && d < dv ? ds_turn(a, v, d, 1.f) : ds_zero4(), vh + r * vs + d, vl + r * vs + d);
+        ds_split4(r < n && d < dv ? (ROT ? v : ds_turn(a, v, d, 1.f)) : ds_zero4(), vh + r * vs + d, vl + r * vs + d);
     });
     __syncthreads();
     float* U = a.ws + ((size_t)blockIdx.x * a.H + h) * (size_t)dv * dk;
@@ -551,7 +597,7 @@ __global__ void __launch_bounds__(256) decay_carry_kernel(const DecayChunks a) {
             if (c0 + j >= nc) continue;
             *reinterpret_cast<uint4*>(u + (size_t)(c0 + j) * stride) = make_uint4(ds_pack(s.x), ds_pack(s.y), ds_pack(s.z), ds_pack(s.w));
             if (DECAY == PRISM_DS_CHANNEL) {
-                w[j] = make_float4(expf(w[j].x), expf(w[j].y), expf(w[j].z), expf(w[j].w));
+                w[j] = make_float4(ds_exp2(w[j].x), ds_exp2(w[j].y), ds_exp2(w[j].z), ds_exp2(w[j].w));
             } else {
                 const float f = DECAY == PRISM_DS_TOKEN ? w[j].x : (c0 + j + 1 < nc ? whole : rest);
                 w[j] = make_float4(f, f, f, f);
@@ -565,12 +611,14 @@ __global__ void __launch_bounds__(256) decay_carry_kernel(const DecayChunks a) {
     *st = s;
 }
 
-constexpr int DS_OUT_THREADS = 128;
+constexpr int DS_OUT_THREADS = 256;
 
-// The outputs of one chunk and head.  Warp w owns tokens 16 w .. 16 w + 15 of the chunk; the operand on the other side
-// (64 value channels of the incoming state, the chunk's keys, its values) passes through one shared buffer.
+// The outputs of one chunk and head.  Warps w and w + 4 own tokens 16 w .. 16 w + 15 of the chunk and share their work - every
+// other k-step against the incoming state, every other sub-chunk of keys - and add up their sums at the end; the operand on
+// the other side (64 value channels of the incoming state, the chunk's keys, its values) passes through one shared buffer.  ROT:
+// rotated queries and keys, a head norm without weight and a gate behind it.
 template <int DVP, int DECAY, bool ROT>
-__global__ void __launch_bounds__(DS_OUT_THREADS, DVP <= 128 ? (DECAY == PRISM_DS_CHANNEL ? 2 : 3) : 1)
+__global__ void __launch_bounds__(DS_OUT_THREADS, DVP <= 128 ? 2 : 1)
 decay_chunk_out_kernel(const DecayChunks a) {
     pdl_trigger();
     int t0, n;
@@ -595,12 +643,12 @@ decay_chunk_out_kernel(const DecayChunks a) {
     const float* kx = pdl_fresh(a.k) + (size_t)(h / a.rep) * dk;
     const float* vx = pdl_fresh(a.v) + (size_t)h * dv;
     const float* pw = DECAY == PRISM_DS_HEAD ? a.pw + (size_t)h * (DS_CHUNK + 1) : nullptr;
-    const int kq = dkp / 4, mat = lane >> 3, lr = lane & 7, row0 = warp * DS_SUB;
+    const int kq = dkp / 4, mat = lane >> 3, lr = lane & 7, rw = warp & 3, grp = warp >> 2, row0 = rw * DS_SUB;
     const bool mine = row0 < n;                            // this warp has tokens
     if (DECAY == PRISM_DS_TOKEN) ds_token_sums(a, h, t0, n, s_b, s_d);       // read behind the barriers below
     // q or k rows of the chunk, prepared, as two terms
     auto load_rows = [&](const float* x, float mul, __nv_bfloat16* hi, __nv_bfloat16* lo) {
-        ds_batches<ROT ? 4 : 8, DS_OUT_THREADS, typename DsQuad<ROT>::type>(DS_CHUNK, kq, [&](int r, int d) {
+        ds_batches<ROT ? 2 : 4, DS_OUT_THREADS, typename DsQuad<ROT>::type>(DS_CHUNK, kq, [&](int r, int d) {
             const int t = t0 + min(r, n - 1);
             return ds_quad<ROT>(a, x + (size_t)t * a.xs, t, d < dk ? d : 0);
         }, [&](int r, int d, const typename DsQuad<ROT>::type& q) {
@@ -609,12 +657,12 @@ decay_chunk_out_kernel(const DecayChunks a) {
     };
     if constexpr (CH) {
         const float* cum = pdl_fresh((const float*)a.cum) + (size_t)h * dk;
-        ds_batches<8, DS_OUT_THREADS, float4>(DS_CHUNK, kq, [&](int r, int d) {
+        ds_batches<4, DS_OUT_THREADS, float4>(DS_CHUNK, kq, [&](int r, int d) {
             return *reinterpret_cast<const float4*>(qx + (size_t)(t0 + min(r, n - 1)) * a.xs + (d < dk ? d : 0));
         }, [&](int r, int d, const float4& q) {
             *reinterpret_cast<float4*>(qf + r * qs + d) = r < n && d < dk ? ds_turn(a, q, d, a.qmul) : ds_zero4();
         });
-        ds_batches<8, DS_OUT_THREADS, float4>(DS_CHUNK, kq, [&](int r, int d) {       // rows beyond n: the last token's
+        ds_batches<4, DS_OUT_THREADS, float4>(DS_CHUNK, kq, [&](int r, int d) {       // rows beyond n: the last token's
             return *reinterpret_cast<const float4*>(cum + (size_t)(t0 + min(r, n - 1)) * a.H * dk + (d < dk ? d : 0));
         }, [&](int r, int d, const float4& q) { *reinterpret_cast<float4*>(bf + r * qs + d) = d < dk ? q : ds_zero4(); });
     } else {
@@ -628,7 +676,7 @@ decay_chunk_out_kernel(const DecayChunks a) {
                 const int c = ks * 16 + (lane & 3) * 2 + (u >> 1) * 8, at = (row0 + (lane >> 2) + (u & 1) * 8) * qs + c;
                 const float2 q = *reinterpret_cast<const float2*>(qf + at), b = *reinterpret_cast<const float2*>(bf + at);
                 const float2 e = ref != nullptr ? *reinterpret_cast<const float2*>(ref + c) : make_float2(0.f, 0.f);
-                const float x0 = q.x * expf(b.x - e.x), x1 = q.y * expf(b.y - e.y);
+                const float x0 = q.x * ds_exp2(b.x - e.x), x1 = q.y * ds_exp2(b.y - e.y);
                 const __nv_bfloat162 hh = __floats2bfloat162_rn(x0, x1);
                 const float2 hf = __bfloat1622float2(hh);
                 ah[u] = *reinterpret_cast<const uint32_t*>(&hh);
@@ -650,7 +698,7 @@ decay_chunk_out_kernel(const DecayChunks a) {
 #pragma unroll
     for (int n0 = 0; n0 < DVP; n0 += SB) {
         if (n0 < dv) {
-            ds_batches<8, DS_OUT_THREADS, uint4>(SB, kq, [&](int r, int d) {
+            ds_batches<4, DS_OUT_THREADS, uint4>(SB, kq, [&](int r, int d) {
                 return *reinterpret_cast<const uint4*>(sin + (size_t)min(n0 + r, dv - 1) * dk + (d < dk ? d : 0));
             }, [&](int r, int d, uint4 v) {
                 if (n0 + r >= dv || d >= dk) v = make_uint4(0u, 0u, 0u, 0u);
@@ -659,7 +707,8 @@ decay_chunk_out_kernel(const DecayChunks a) {
             });
             __syncthreads();
             if (mine)
-                for (int ks = 0; ks < dkp / 16; ++ks) {
+#pragma unroll 1
+                for (int ks = grp; ks < dkp / 16; ks += 2) {
                     uint32_t ah[4], al[4];
                     q_frag(ks, nullptr, ah, al);
 #pragma unroll
@@ -688,7 +737,7 @@ decay_chunk_out_kernel(const DecayChunks a) {
     }
     // scores against the chunk's own keys, decayed by what lies between
     if constexpr (CH) {
-        ds_batches<8, DS_OUT_THREADS, float4>(DS_CHUNK, kq, [&](int r, int d) {
+        ds_batches<4, DS_OUT_THREADS, float4>(DS_CHUNK, kq, [&](int r, int d) {
             return *reinterpret_cast<const float4*>(kx + (size_t)(t0 + min(r, n - 1)) * a.xs + (d < dk ? d : 0));
         }, [&](int r, int d, const float4& q) {
             float4 v = ds_zero4();
@@ -696,7 +745,7 @@ decay_chunk_out_kernel(const DecayChunks a) {
                 const float4 b = *reinterpret_cast<const float4*>(bf + r * qs + d);
                 const float4 e = *reinterpret_cast<const float4*>(bf + (r | (DS_SUB - 1)) * qs + d);
                 v = ds_turn(a, q, d, a.kmul);
-                v = make_float4(v.x * expf(e.x - b.x), v.y * expf(e.y - b.y), v.z * expf(e.z - b.z), v.w * expf(e.w - b.w));
+                v = make_float4(v.x * ds_exp2(e.x - b.x), v.y * ds_exp2(e.y - b.y), v.z * ds_exp2(e.z - b.z), v.w * ds_exp2(e.w - b.w));
             }
             ds_split4(v, bh + r * qs + d, bl + r * qs + d);
         });
@@ -704,9 +753,10 @@ decay_chunk_out_kernel(const DecayChunks a) {
         load_rows(kx, a.kmul, bh, bl);
     }
     __syncthreads();
-    float s[DS_CHUNK / 8][4];
+    constexpr int PAIRS = DS_CHUNK / DS_SUB / 2;           // sub-chunks of keys a warp may have: 2 j + grp
+    float s[2 * PAIRS][4];
 #pragma unroll
-    for (int i = 0; i < DS_CHUNK / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+    for (int i = 0; i < 2 * PAIRS; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
     if constexpr (CH) {
         float span = 0.f;                                      // how far the log decays go inside this warp's sub-chunk
         for (int d = lane; d < dk; d += 32) span = fmaxf(span, bf[row0 * qs + d] - bf[(row0 + DS_SUB - 1) * qs + d]);
@@ -714,8 +764,9 @@ decay_chunk_out_kernel(const DecayChunks a) {
         if (mine) {
             const bool by_terms = span > DS_MAX_SPAN;
 #pragma unroll
-            for (int np = 0; np < DS_CHUNK / DS_SUB; ++np) {
-                if (np > warp || (np == warp && by_terms)) continue;
+            for (int j = 0; j < PAIRS; ++j) {
+                const int np = 2 * j + grp;
+                if (np > rw || (np == rw && by_terms)) continue;
                 const float* ref = bf + (np * DS_SUB + DS_SUB - 1) * qs;
                 for (int ks = 0; ks < dkp / 16; ++ks) {
                     uint32_t ah[4], al[4], xh[4], xl[4];
@@ -725,49 +776,55 @@ decay_chunk_out_kernel(const DecayChunks a) {
                     ldmatrix_x4(xl, bl + bt);
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
-                        mma_bf16_16816(s[2 * np + e], ah, xh[2 * e], xh[2 * e + 1]);
-                        mma_bf16_16816(s[2 * np + e], ah, xl[2 * e], xl[2 * e + 1]);
-                        mma_bf16_16816(s[2 * np + e], al, xh[2 * e], xh[2 * e + 1]);
+                        mma_bf16_16816(s[2 * j + e], ah, xh[2 * e], xh[2 * e + 1]);
+                        mma_bf16_16816(s[2 * j + e], ah, xl[2 * e], xl[2 * e + 1]);
+                        mma_bf16_16816(s[2 * j + e], al, xh[2 * e], xh[2 * e + 1]);
                     }
                 }
             }
             // the warp's own sub-chunk: by terms where it has to be, and only keys up to the query
 #pragma unroll
-            for (int np = 0; np < DS_CHUNK / DS_SUB; ++np) {
-                if (np != warp) continue;
-#pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                    const int r = (i & 2) ? r1 : r0, c = np * DS_SUB + (i >> 2) * 8 + (lane & 3) * 2 + (i & 1);
-                    float& x = s[2 * np + (i >> 2)][i & 3];
-                    if (c > r) {
-                        x = 0.f;
-                    } else if (by_terms && r < n) {
+            for (int j = 0; j < PAIRS; ++j) {
+                const int np = 2 * j + grp;
+                if (np != rw) continue;
+                auto key = [&](int i) { return np * DS_SUB + (i >> 2) * 8 + (lane & 3) * 2 + (i & 1); };
+                if (by_terms)
+#pragma unroll 1
+                    for (int i = 0; i < 8; ++i) {
+                        const int r = (i & 2) ? r1 : r0, c = min(key(i), n - 1);
                         const float* kr = kx + (size_t)(t0 + c) * a.xs;
                         float sum = 0.f;
-                        for (int d = 0; d < dk; ++d)
-                            sum += qf[r * qs + d] * ((a.act ? ds_silu(kr[d]) : kr[d]) * a.kmul) * expf(bf[r * qs + d] - bf[c * qs + d]);
-                        x = sum;
+#pragma unroll 1
+                        for (int d = 0; d < dk; ++d)          // c after r: masked below; the difference may then be large, capped
+                            sum += qf[r * qs + d] * ((a.act ? ds_silu(kr[d]) : kr[d]) * a.kmul) * ds_exp2(fminf(bf[r * qs + d] - bf[c * qs + d], 0.f));
+#pragma unroll
+                        for (int u = 0; u < 8; ++u)
+                            if (u == i) s[2 * j + (u >> 2)][u & 3] = sum;
                     }
-                }
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+                    if (key(i) > ((i & 2) ? r1 : r0)) s[2 * j + (i >> 2)][i & 3] = 0.f;
             }
         }
     } else {
         if (mine) {
+#pragma unroll 1
             for (int ks = 0; ks < dkp / 16; ++ks) {
                 uint32_t ah[4], al[4];
                 q_frag(ks, nullptr, ah, al);
 #pragma unroll
-                for (int np = 0; np < DS_CHUNK / 16; ++np) {
-                    if (np > warp) continue;                   // keys after this warp's last token
+                for (int j = 0; j < PAIRS; ++j) {
+                    const int np = 2 * j + grp;
+                    if (np > rw) continue;                     // keys after this warp's last token
                     uint32_t xh[4], xl[4];
                     const int bt = (np * 16 + (mat >> 1) * 8 + lr) * qs + ks * 16 + (mat & 1) * 8;
                     ldmatrix_x4(xh, bh + bt);
                     ldmatrix_x4(xl, bl + bt);
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
-                        mma_bf16_16816(s[2 * np + e], ah, xh[2 * e], xh[2 * e + 1]);
-                        mma_bf16_16816(s[2 * np + e], ah, xl[2 * e], xl[2 * e + 1]);
-                        mma_bf16_16816(s[2 * np + e], al, xh[2 * e], xh[2 * e + 1]);
+                        mma_bf16_16816(s[2 * j + e], ah, xh[2 * e], xh[2 * e + 1]);
+                        mma_bf16_16816(s[2 * j + e], ah, xl[2 * e], xl[2 * e + 1]);
+                        mma_bf16_16816(s[2 * j + e], al, xh[2 * e], xh[2 * e + 1]);
                     }
                 }
             }
@@ -775,29 +832,29 @@ decay_chunk_out_kernel(const DecayChunks a) {
     }
     if constexpr (!CH) {
 #pragma unroll
-        for (int nt = 0; nt < DS_CHUNK / 8; ++nt)
+        for (int nt = 0; nt < 2 * PAIRS; ++nt)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const int r = e < 2 ? r0 : r1, c = nt * 8 + (lane & 3) * 2 + (e & 1), back = r - c;
+                const int r = e < 2 ? r0 : r1, c = (nt & ~1) * 16 + grp * DS_SUB + (nt & 1) * 8 + (lane & 3) * 2 + (e & 1), back = r - c;
                 if (DECAY == PRISM_DS_HEAD) s[nt][e] = back >= 0 ? s[nt][e] * pw[back] : 0.f;
                 else s[nt][e] = back >= 0 ? s[nt][e] * (expf(s_b[r] - s_b[c]) * s_d[c]) : 0.f;
             }
     }
     __syncthreads();
-    ds_batches<8, DS_OUT_THREADS, float4>(DS_CHUNK, DVP / 4, [&](int r, int d) {
+    ds_batches<4, DS_OUT_THREADS, float4>(DS_CHUNK, DVP / 4, [&](int r, int d) {
         return *reinterpret_cast<const float4*>(vx + (size_t)(t0 + min(r, n - 1)) * a.xs + (d < dv ? d : 0));
     }, [&](int r, int d, float4 v) {
-        ds_split4(r < n && d < dv ? ds_turn(a, v, d, 1.f) : ds_zero4(), bh + r * VS + d, bl + r * VS + d);
+        ds_split4(r < n && d < dv ? (ROT ? v : ds_turn(a, v, d, 1.f)) : ds_zero4(), bh + r * VS + d, bl + r * VS + d);
     });
     __syncthreads();
-    if (!mine) return;
 #pragma unroll
-    for (int kk = 0; kk < DS_CHUNK / 16; ++kk) {
-        if (kk > warp) continue;
+    for (int j2 = 0; j2 < PAIRS; ++j2) {
+        const int kk = 2 * j2 + grp;
+        if (!mine || kk > rw) continue;
         uint32_t ph[4], pl[4];
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
-            const float x0 = s[2 * kk + (u >> 1)][(u & 1) * 2], x1 = s[2 * kk + (u >> 1)][(u & 1) * 2 + 1];
+            const float x0 = s[2 * j2 + (u >> 1)][(u & 1) * 2], x1 = s[2 * j2 + (u >> 1)][(u & 1) * 2 + 1];
             const __nv_bfloat162 hh = __floats2bfloat162_rn(x0, x1);
             const float2 hf = __bfloat1622float2(hh);
             ph[u] = *reinterpret_cast<const uint32_t*>(&hh);
@@ -817,7 +874,25 @@ decay_chunk_out_kernel(const DecayChunks a) {
             }
         }
     }
-    if (a.gate == nullptr) {           // the read-out itself, with the skip path where there is one
+    // the pair's sums come together through the buffer (64 rows of DVP + 8 floats)
+    __syncthreads();
+    float* sums = reinterpret_cast<float*>(bh);
+    if (grp == 1 && mine)
+#pragma unroll
+        for (int i = 0; i < DVP / 8; ++i) {
+            const int d = i * 8 + (lane & 3) * 2;
+            *reinterpret_cast<float2*>(sums + r0 * VS + d) = make_float2(o[i][0], o[i][1]);
+            *reinterpret_cast<float2*>(sums + r1 * VS + d) = make_float2(o[i][2], o[i][3]);
+        }
+    __syncthreads();
+    if (grp == 1 || !mine) return;
+#pragma unroll
+    for (int i = 0; i < DVP / 8; ++i) {
+        const int d = i * 8 + (lane & 3) * 2;
+        const float2 x = *reinterpret_cast<const float2*>(sums + r0 * VS + d), y = *reinterpret_cast<const float2*>(sums + r1 * VS + d);
+        o[i][0] += x.x; o[i][1] += x.y; o[i][2] += y.x; o[i][3] += y.y;
+    }
+    if (!ROT && a.gate == nullptr) {   // the read-out itself, with the skip path where there is one
         const float skip = DECAY == PRISM_DS_TOKEN && a.skip != nullptr ? load_param(a.skip, a.skip_bf16, h) : 0.f;
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
@@ -861,7 +936,7 @@ decay_chunk_out_kernel(const DecayChunks a) {
             if (d >= dv) continue;
             const float2 gz = *reinterpret_cast<const float2*>(gate + d);
             float2 y = make_float2(o[i][2 * e] * inv * ds_silu(gz.x), o[i][2 * e + 1] * inv * ds_silu(gz.y));
-            if (a.weight != nullptr) {
+            if (!ROT && a.weight != nullptr) {
                 y.x *= load_param(a.weight, a.weight_bf16, d);
                 y.y *= load_param(a.weight, a.weight_bf16, d + 1);
             }
@@ -941,6 +1016,7 @@ PRISM_EXPORT int prism_decay_step(int kind, const float* q, const float* k, cons
     do {                                           \
         if (dk <= 32) PRISM_DSTEP(TT, 8, 1, 4, D);    \
         if (dk <= 64) PRISM_DSTEP(TT, 16, 1, 8, D);   \
+        if (dk <= 128 && dv <= 64) PRISM_DSTEP(TT, 32, 1, 8, D); \
         if (dk <= 128) PRISM_DSTEP(TT, 32, 1, 16, D); \
         PRISM_DSTEP(TT, 32, 2, 8, D);                 \
     } while (0)
@@ -958,31 +1034,33 @@ PRISM_EXPORT int prism_decay_step(int kind, const float* q, const float* k, cons
 }
 
 // As above for segments of any length (q, k, v rows, strides and pointers in whole quads); table [T, rot / 2, 2] float32:
-// cosine and sine of position * frequency; pw [H, 65]: powers 0 .. 64 of the heads' decays; cum [T, H dk] float32: the log decays
-// of PRISM_DS_CHANNEL, overwritten; ws: (T / 64 + S) * H * dv * dk floats; fac: (T / 64 + S) * H floats.  out bf16 with a gate, else
+// cosine and sine of position * frequency; pw [H, 65]: powers 0 .. 64 of the heads' decays; cum [T, H dk] float32: scratch of
+// PRISM_DS_CHANNEL; ws: (T / 64 + S) * H * dv * dk floats; fac: (T / 64 + S) * H floats.  out bf16 with a gate, else
 // float32.
 PRISM_EXPORT int prism_decay_chunks(int kind, const float* q, const float* k, const float* v, long long xs, int T, int S, int H, int rep,
                                     int dk, int dv, int act, const float* table, int rot, int pairs, float amp, float qmul, float kmul,
                                     const float* pw, const float* dt, long long dts, const void* dt_bias, int dt_bias_dtype,
-                                    const void* a_log, int a_log_dtype, const void* skip, int skip_dtype, float* cum, float* state,
+                                    const void* a_log, int a_log_dtype, const void* skip, int skip_dtype, const float* low, long long ls,
+                                    int R, const float* a2t, const void* a2_bias, int a2_bias_dtype, float rate, float* cum, float* state,
                                     const int* seg_start, const int* slots, const float* gate, long long gs, const void* weight,
                                     int weight_dtype, float eps, float* ws, float* fac, void* out, long long os, cudaStream_t stream) {
     using namespace prism;
     if (T <= 0 || S <= 0) return 0;
     if (!prism_decay_chunks_supported(dk, dv, rot, pairs) || H < 1 || H > 65535 || S > 65535 || rep < 1 || H % rep || rot < 0 || rot > dk ||
-        (rot && (table == nullptr || kind != PRISM_DS_HEAD || act)) || xs % 4 || os % 2 || (uintptr_t)q % 16 || (uintptr_t)k % 16 ||
+        (rot && (table == nullptr || kind != PRISM_DS_HEAD || act || gate == nullptr || weight != nullptr)) || xs % 4 || os % 2 || (uintptr_t)q % 16 || (uintptr_t)k % 16 ||
         (uintptr_t)v % 16 || (uintptr_t)table % 16 || (uintptr_t)state % 16 || (uintptr_t)ws % 16 || (uintptr_t)cum % 16 ||
         (uintptr_t)out % (gate ? 4 : 8) || (gate && (gs % 2 || (uintptr_t)gate % 8)))
         return (int)cudaErrorInvalidValue;
     if ((kind == PRISM_DS_HEAD && pw == nullptr) ||
         (kind == PRISM_DS_TOKEN && (dt == nullptr || dt_bias == nullptr || a_log == nullptr || fac == nullptr || gate != nullptr || act)) ||
-        (kind == PRISM_DS_CHANNEL && cum == nullptr) || kind < 0 || kind > PRISM_DS_CHANNEL)
+        (kind == PRISM_DS_CHANNEL && (cum == nullptr || low == nullptr || a2t == nullptr || R < 1)) || kind < 0 || kind > PRISM_DS_CHANNEL)
         return (int)cudaErrorInvalidValue;
     const auto b16 = [](int d) { return d == PRISM_DTYPE_BF16 ? 1 : 0; };
     DecayChunks a;
     a.q = q; a.k = k; a.v = v; a.xs = xs; a.H = H; a.rep = rep; a.dk = dk; a.dv = dv; a.S = S; a.act = act;
     a.table = reinterpret_cast<const float2*>(table); a.rot = rot; a.pairs = pairs; a.amp = amp; a.qmul = qmul; a.kmul = kmul; a.pw = pw;
     a.dt = dt; a.dts = dts; a.dt_bias = dt_bias; a.dt_bias_bf16 = b16(dt_bias_dtype); a.a_log = a_log; a.a_log_bf16 = b16(a_log_dtype);
+    a.low = low; a.ls = ls; a.R = R; a.a2t = a2t; a.a2_bias = a2_bias; a.a2_bias_bf16 = b16(a2_bias_dtype); a.rate = rate;
     a.skip = skip; a.skip_bf16 = b16(skip_dtype); a.cum = cum; a.state = state; a.seg_start = seg_start; a.slots = slots; a.ws = ws;
     a.fac = fac; a.gate = gate; a.gs = gs; a.weight = weight; a.weight_bf16 = b16(weight_dtype); a.eps = eps; a.out = out; a.os = os;
     const int chunks = T / DS_CHUNK + S;

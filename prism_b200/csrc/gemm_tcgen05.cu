@@ -218,7 +218,7 @@ gemm_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                 }
             }
             if (finish && m < N) {
-                const float b = EPI != EPI_PARTIAL && bias != nullptr ? load_param(bias, bias_bf16, m) : 0.f;
+                const float b = bias != nullptr && (EPI != EPI_PARTIAL || blockIdx.y == 0) ? load_param(bias, bias_bf16, m) : 0.f;
                 const float bu = EPI == EPI_SWIGLU && bias != nullptr ? load_param(bias, bias_bf16, N + m) : 0.f;
 #pragma unroll
                 for (int n = 0; n < NTOK; ++n) {
@@ -230,7 +230,7 @@ gemm_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                         reinterpret_cast<__nv_bfloat16*>(y)[(size_t)n * ldy + m] =
                             __float2bfloat16_rn(glu_act == 2 ? clamped_glu(g, u, glu_limit) : a * u);
                     } else if (EPI == EPI_PARTIAL) {
-                        reinterpret_cast<float*>(y)[((size_t)blockIdx.y * M + n) * ldy + m] = acc[0][n];
+                        reinterpret_cast<float*>(y)[((size_t)blockIdx.y * M + n) * ldy + m] = acc[0][n] + b;
                     } else if (EPI == EPI_F32) {
                         reinterpret_cast<float*>(y)[(size_t)n * ldy + m] = acc[0][n] + b;
                     } else {
@@ -286,7 +286,7 @@ PRISM_EXPORT int prism_gemm_tcgen05_supported(int M, int N, int K) {
 }
 
 // epi: 0 bf16 (+bias), 1 float32 (+bias), 2 paired SwiGLU (W is [2N, K], bias [2N] or null; bf16 out [M, N]),
-// 3 partial sums: y is float32 [ksplit, M, N] (ldy = N), no bias; 4: as 2 with the gate through gelu_tanh instead of silu,
+// 3 partial sums: y is float32 [ksplit, M, N] (ldy = N), a bias joins the first; 4: as 2 with the gate through gelu_tanh instead of silu,
 // 5: as 2 in the clamped form with `glu_limit` (common.cuh: clamped_glu).
 // ksplit > 1 with epi 0 or 1 needs a workspace `ws` of ksplit * M * N floats and `counters`, one int per
 // 128-row tile of N, zero before the first launch (the kernel leaves them zero); the last CTA of each

@@ -38,9 +38,10 @@ __device__ __forceinline__ float moe_tc_act(float z, int act) {
     return act == 3 ? r * r : r;                                                                      // relu squared, relu
 }
 
-// an expert's hidden value from its gate and up values; act 4: the clamped form (common.cuh: clamped_glu)
-__device__ __forceinline__ float moe_tc_glu(float g, float u, int act, float limit) {
-    return act == 4 ? clamped_glu(g, u, limit) : moe_tc_act(g, act) * u;
+// an expert's hidden value from its gate and up values
+template <bool CLAMP> __device__ __forceinline__ float moe_tc_glu(float g, float u, int act, float limit) {
+    if constexpr (CLAMP) return clamped_glu(g, u, limit);
+    else return moe_tc_act(g, act) * u;
 }
 
 template <int NTOK, bool DUAL> struct MoeCfg {
@@ -63,7 +64,7 @@ struct MoeShared {
     long long ldy;
 };
 
-template <int NTOK, bool DUAL>
+template <int NTOK, bool DUAL, bool CLAMP>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                 const int* __restrict__ offs_in, const int* __restrict__ counts_in, const int* __restrict__ row_dst_in,
@@ -240,7 +241,7 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                         reinterpret_cast<float*>(y)[(size_t)p * ldy + m] = acc[0][n];
                     } else if (DUAL) {
                         reinterpret_cast<__nv_bfloat16*>(y)[(size_t)p * ldy + m] =
-                            __float2bfloat16_rn(moe_tc_glu(acc[0][n], acc[W_TILES - 1][n], act, limit));
+                            __float2bfloat16_rn(moe_tc_glu<CLAMP>(acc[0][n], acc[W_TILES - 1][n], act, limit));
                     } else if (row_dst == nullptr) {          // an expert without a gate: its hidden layer, act(up a_p)
                         reinterpret_cast<__nv_bfloat16*>(y)[(size_t)p * ldy + m] = __float2bfloat16_rn(moe_tc_act(acc[0][n], act));
                     } else {
@@ -260,7 +261,7 @@ moe_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
     }
 }
 
-template <int NTOK, bool DUAL>
+template <int NTOK, bool DUAL, bool CLAMP = false>
 int moe_launch(const void* x, long long ldx, long long x_rows, const void* W, const int* offs, const int* counts,
                const int* row_dst, const float* row_w, int token_tiles, int E, int N, int K, int act, void* y,
                long long ldy, int* err, const void* sw, const void* sx, long long ldsx, const MoeShared& sh, int ksplit, float* ws,
@@ -278,7 +279,7 @@ int moe_launch(const void* x, long long ldx, long long x_rows, const void* W, co
         rc = make_map(&msx, sx, sh.rows, sh.K, ldsx, NTOK);
         if (rc) return rc;
     }
-    auto kern = moe_swap_kernel<NTOK, DUAL>;
+    auto kern = moe_swap_kernel<NTOK, DUAL, CLAMP>;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM);
     const int widest = sh.tiles > 0 && sh.N > N ? sh.N : N;
     dim3 grid((widest + MOE_TILE_M - 1) / MOE_TILE_M, token_tiles + sh.tiles, ksplit);
@@ -371,6 +372,8 @@ PRISM_EXPORT int prism_moe_gemm_tcgen05(const void* a, long long lda, const void
     if (token_tiles + sh.tiles > 65535) return (int)cudaErrorInvalidValue;
     const long long x_rows = (long long)token_tiles * ntok;
 #define ARGS a, lda, x_rows, w, offs, counts, row_dst, row_w, token_tiles, E, N, K, act, out, ldo, err, sw, sx, ldsx, sh, ksplit, ws, counters, limit, stream
+    if (dual && act == 4)        // the clamped form (common.cuh: clamped_glu)
+        return ntok == 16 ? moe_launch<16, true, true>(ARGS) : ntok == 32 ? moe_launch<32, true, true>(ARGS) : moe_launch<64, true, true>(ARGS);
     if (dual) return ntok == 16 ? moe_launch<16, true>(ARGS) : ntok == 32 ? moe_launch<32, true>(ARGS) : moe_launch<64, true>(ARGS);
     return ntok == 16 ? moe_launch<16, false>(ARGS) : ntok == 32 ? moe_launch<32, false>(ARGS) : moe_launch<64, false>(ARGS);
 #undef ARGS

@@ -11,7 +11,8 @@
 // position p becomes (a cos t - b sin t, b cos t + a sin t), t = p * freq[i]; `freq` is a float32 table
 // of rot / 2 entries (any frequency scaling is in the table), the angle and sincosf are float32.  The slot of
 // position p of request seg is block_table[seg][p / page_size] * page_size + p % page_size.
-// One warp per (token, head); one more warp per token copies the values.
+// One warp per (token, head); one more warp per token copies the values.  With `whole` one CTA takes a token: it reads q and k
+// once into shared memory, sums both, and norms and turns them from there.
 #include "common.cuh"
 
 namespace prism {
@@ -90,6 +91,100 @@ __global__ void qk_norm_rope_store_kernel(const float* __restrict__ q_in, const 
     }
 }
 
+// The whole-projection form: dynamic shared memory [(nh + nkv) dk] floats, then cosines and sines [rot / 2] each.  VEC 4: q, k, v
+// rows and outputs are read and written four entries at a time.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) qk_norm_whole_kernel(
+    const float* __restrict__ q_in, const float* __restrict__ k_in, const float* __restrict__ v_in, long long ps,
+    const void* __restrict__ wq, int wq_bf16, const void* __restrict__ wk, int wk_bf16, float eps, const float* __restrict__ freq, int rot,
+    T* __restrict__ q_out, T* __restrict__ k_plane, T* __restrict__ v_plane, const int* __restrict__ block_table, int bt_width,
+    const int* __restrict__ positions, const int* __restrict__ tok_seg, int nh, int nkv, int dk, int dv, int page_size, int num_pages,
+    int max_pos, int* err, int halves, float v_scale) {
+    pdl_trigger();
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[33];
+    const bool own = k_plane != nullptr;
+    const int t = blockIdx.x, pos = positions[t], nq = nh * dk, nk = own ? nkv * dk : 0, half = rot >> 1;
+    float *cs = row + (nh + nkv) * dk, *sn = cs + half;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * freq[i], sn + i, cs + i);
+    if (pos < 0 || pos >= max_pos) {
+        if (threadIdx.x == 0) report_error(err, PRISM_ERR_POSITION_RANGE);
+        return;
+    }
+    const int page = own ? block_table[(size_t)tok_seg[t] * bt_width + pos / page_size] : 0;
+    const bool page_ok = page >= 0 && page < num_pages;
+    if (!page_ok && threadIdx.x == 0) report_error(err, PRISM_ERR_PAGE_RANGE);
+    const size_t slot = page_ok ? (size_t)page * page_size + pos % page_size : 0;
+    pdl_wait();
+    const float* q = pdl_fresh(q_in) + (size_t)t * ps;
+    const float* k = pdl_fresh(k_in) + (size_t)t * ps;
+    const float* v = pdl_fresh(v_in) + (size_t)t * ps;
+    auto load = [](const float* p, float (&x)[VEC]) {
+        if constexpr (VEC == 4) {
+            const float4 a = *reinterpret_cast<const float4*>(p);
+            x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w;
+        } else {
+            x[0] = *p;
+        }
+    };
+    auto store = [](T* p, const float (&x)[VEC]) {
+        if constexpr (VEC == 4 && sizeof(T) == 2) {
+            const __nv_bfloat162 a = __floats2bfloat162_rn(x[0], x[1]), b = __floats2bfloat162_rn(x[2], x[3]);
+            *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+        } else if constexpr (VEC == 4) {
+            *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+        } else {
+            *p = from_float<T>(x[0]);
+        }
+    };
+    float sq = 0.f, sk = 0.f;
+    for (int c = threadIdx.x * VEC; c < nq + nk; c += blockDim.x * VEC) {
+        float x[VEC];
+        load(c < nq ? q + c : k + (c - nq), x);
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            row[c + i] = x[i];
+            ss += x[i] * x[i];
+        }
+        if (c < nq) sq += ss; else sk += ss;
+    }
+    if (own && page_ok)
+        for (int c = threadIdx.x * VEC; c < nkv * dv; c += blockDim.x * VEC) {
+            float x[VEC];
+            load(v + c, x);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) x[i] *= v_scale;
+            store(v_plane + slot * nkv * dv + c, x);
+        }
+    sq = block_sum(sq, red);
+    sk = own ? block_sum(sk, red) : 0.f;
+    const float inv_q = 1.f / sqrtf(sq / (float)nq + eps), inv_k = own ? 1.f / sqrtf(sk / (float)nk + eps) : 0.f;
+    for (int c = threadIdx.x * VEC; c < nq + nk; c += blockDim.x * VEC) {
+        const bool is_q = c < nq;
+        if (!is_q && !page_ok) continue;
+        const int g = is_q ? c : c - nq;                       // place in its projection
+        const void* w = is_q ? wq : wk;
+        const int wb = is_q ? wq_bf16 : wk_bf16;
+        const float inv = is_q ? inv_q : inv_k;
+        float x[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            const int d = (g + i) % dk;
+            float a = row[c + i] * inv * load_param(w, wb, g + i);
+            if (d < rot) {
+                const int e = halves ? (d < half ? half : -half) : ((d & 1) ? -1 : 1);
+                const bool second = halves ? d >= half : (d & 1);
+                const int f = halves ? (second ? d - half : d) : d >> 1;
+                const float b = row[c + i + e] * inv * load_param(w, wb, g + i + e);
+                a = second ? a * cs[f] + b * sn[f] : a * cs[f] - b * sn[f];
+            }
+            x[i] = a;
+        }
+        store(is_q ? q_out + (size_t)t * nq + g : k_plane + slot * nk + g, x);
+    }
+}
+
 }  // namespace prism
 
 // q, k, v: float32 rows with one row stride `ps` (column blocks of one product); planes [slots, nkv, dk] and
@@ -108,6 +203,27 @@ PRISM_EXPORT int prism_qk_norm_rope_store(const float* q, const float* k, const 
     const dim3 grid(T, (units + threads / 32 - 1) / (threads / 32));
     if (T > 65535 * 32) return (int)cudaErrorInvalidValue;
     const int qb = wq_dtype == PRISM_DTYPE_BF16, kb = wk_dtype == PRISM_DTYPE_BF16;
+    const size_t row_bytes = ((size_t)(nh + nkv) * dk + rot) * sizeof(float);
+    if (whole && wq != nullptr && (wk != nullptr || k_plane == nullptr) && row_bytes <= 160 * 1024) {
+        const int esz = dtype == PRISM_DTYPE_BF16 ? 2 : 4;
+        const bool vec = dk % 4 == 0 && dv % 4 == 0 && ps % 4 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0 && (uintptr_t)v % 16 == 0 &&
+                         (uintptr_t)q_out % (4 * esz) == 0 && (uintptr_t)k_plane % (4 * esz) == 0 && (uintptr_t)v_plane % (4 * esz) == 0;
+#define PRISM_QW(TT, V)                                                                                                      \
+    do {                                                                                                                     \
+        auto kern = prism::qk_norm_whole_kernel<TT, V>;                                                                      \
+        if (row_bytes > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)row_bytes);  \
+        return (int)prism::launch_kernel(kern, dim3(T), dim3(256), row_bytes, stream, q, k, v, ps, wq, qb, wk, kb, eps, freq, rot, \
+                                         (TT*)q_out, (TT*)k_plane, (TT*)v_plane, block_table, bt_width, positions, tok_seg, nh, nkv, \
+                                         dk, dv, page_size, num_pages, max_pos, err, halves, v_scale);                       \
+    } while (0)
+        if (dtype == PRISM_DTYPE_BF16) {
+            if (vec) PRISM_QW(__nv_bfloat16, 4);
+            PRISM_QW(__nv_bfloat16, 1);
+        }
+        if (vec) PRISM_QW(float, 4);
+        PRISM_QW(float, 1);
+#undef PRISM_QW
+    }
     if (dtype == PRISM_DTYPE_BF16)
         return (int)prism::launch_kernel(prism::qk_norm_rope_store_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, q, k,
                                          v, ps, wq, qb, wk, kb, eps, freq, rot, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_plane,

@@ -164,7 +164,6 @@ __global__ void decay_from_exponent_kernel(float* __restrict__ w, long long ws, 
 //   PRISM_LR_SIGMOID   sigmoid(z)                            a gate
 //   PRISM_LR_EXPSIG    exp(-rate sigmoid(z))                 a per-channel decay kept inside (exp(-rate), 1), rate a constant
 //   PRISM_LR_SIGPOW    sigmoid(z)^rate                       a per-channel decay near one for a small constant rate
-//   PRISM_LR_LOGSIGPOW rate log sigmoid(z)                   its logarithm
 // b may be null.  A CTA takes 128 channels and sixteen tokens, so that every weight it reads serves sixteen tokens
 // (whose inner values sit side by side in shared memory: four 128-bit loads per weight); w2t is the second matrix
 // transposed, [R, N], so that neighbouring threads read neighbouring floats.
@@ -173,7 +172,6 @@ __global__ void decay_from_exponent_kernel(float* __restrict__ w, long long ws, 
 #define PRISM_LR_SIGMOID 2
 #define PRISM_LR_EXPSIG 3
 #define PRISM_LR_SIGPOW 4
-#define PRISM_LR_LOGSIGPOW 5
 constexpr int LRD_TOK = 16;
 __global__ void lowrank_decay_kernel(const float* __restrict__ low_in, long long ls, int R, const float* __restrict__ w2t,
                                      const void* __restrict__ w0, int w0_bf16, int N, int T, float* __restrict__ out,
@@ -214,8 +212,7 @@ __global__ void lowrank_decay_kernel(const float* __restrict__ low_in, long long
             out[(size_t)(t0 + j) * os + n] = epi == PRISM_LR_EXPEXP ? expf(-expf(z))
                                              : epi == PRISM_LR_SOFTPLUS ? expf(-rate * softplus_f(z))
                                              : epi == PRISM_LR_EXPSIG ? expf(-crate * sigmoid_f(z))
-                                             : epi == PRISM_LR_SIGPOW ? expf(-crate * softplus_f(-z))
-                                             : epi == PRISM_LR_LOGSIGPOW ? -crate * softplus_f(-z) : sigmoid_f(z);
+                                             : epi == PRISM_LR_SIGPOW ? expf(-crate * softplus_f(-z)) : sigmoid_f(z);
         }
 }
 

@@ -115,7 +115,7 @@ class _Sig:
     prism_decay_step = [_i, _p, _p, _p, _ll, _i, _i, _i, _i, _i, _i, _p, _i, _i, _f, _f, _f, _p, _p, _ll, _p, _i, _p, _i, _p, _i,
                         _p, _ll, _i, _p, _p, _i, _f, _p, _p, _p, _p, _ll, _p, _i, _f, _p, _i, _ll, _p]
     prism_decay_chunks = [_i, _p, _p, _p, _ll, _i, _i, _i, _i, _i, _i, _i, _p, _i, _i, _f, _f, _f, _p, _p, _ll, _p, _i, _p, _i, _p, _i,
-                          _p, _p, _p, _p, _p, _ll, _p, _i, _f, _p, _p, _p, _ll, _p]
+                          _p, _ll, _i, _p, _p, _i, _f, _p, _p, _p, _p, _p, _ll, _p, _i, _f, _p, _p, _p, _ll, _p]
     prism_unit_removal = [_p, _p, _ll, _p, _i, _f, _i, _i, _i, _p, _p]
     prism_decay_from_exponent = [_p, _ll, _p, _i, _i, _i, _p]
     prism_lowrank_decay = [_p, _ll, _i, _p, _p, _i, _i, _i, _p, _ll, _i, _i, _p, _i, _i, _f, _p]
@@ -334,7 +334,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out:
     """tcgen05 + TMA weight-streaming product for up to 64 tokens.  ``epi``:
     ``EPI_BF16`` / ``EPI_F32`` (``out [M, N]``, + bias), ``EPI_SWIGLU`` (``w`` is
     the fused ``[2N, K]`` gate/up weight), ``EPI_PARTIAL`` (``out`` float32
-    ``[ksplit, M, N]`` partial sums over K for the next kernel to add).  ``group_rows`` (a multiple of 128):
+    ``[ksplit, M, N]`` partial sums over K for the next kernel to add, a bias in the first).  ``group_rows`` (a multiple of 128):
     ``x`` is ``[groups, M, K]`` and the weight rows ``[g group_rows, (g + 1) group_rows)`` read ``x[g]``."""
     _cuda(x, w, bias, out)
     group_tokens = 0
@@ -348,7 +348,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out:
     assert x.stride(1) == 1 and w.stride(1) == 1 and out.is_contiguous()
     assert w.shape[0] == (2 * N if epi in _PAIRED else N) and (bias is None or bias.shape == (w.shape[0],))
     if epi == EPI_PARTIAL:
-        assert out.dtype == torch.float32 and out.shape == (ksplit, M, N) and bias is None
+        assert out.dtype == torch.float32 and out.shape == (ksplit, M, N)
     else:
         assert out.shape == (M, N)
         assert out.dtype == (torch.float32 if epi == EPI_F32 else torch.bfloat16)
@@ -436,12 +436,12 @@ def linear_delta(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] 
     next norm: like ``linear``, but it may return a float32 stack ``[k, M, N]``
     of partial sums over K, which the fused add + norm kernel adds up.  ``f32``: the
     result is float32 in any case (never rounded to 16 bits before the residual sum)."""
-    if bias is None and tc_gemm_ok(x, w):
+    if tc_gemm_ok(x, w):
         N, K = w.shape
         ks = tc_ksplit(N, K, M=x.shape[0])
         if ks > 1:
             out = torch.empty((ks, x.shape[0], N), dtype=torch.float32, device=x.device)
-            gemm_tc(x, w, None, out, EPI_PARTIAL, ksplit=ks)
+            gemm_tc(x, w, bias, out, EPI_PARTIAL, ksplit=ks)
             return out
     return linear(x, w, bias, out_dtype=torch.float32 if f32 else None)
 
@@ -2004,7 +2004,7 @@ class DecayedSum:
             return "step"
         ptrs = (self.q, self.k, self.v, self.out) + (() if self.gate is None else (self.gate,))
         if (ctx.max_q_len >= DECAY_CHUNKED_FROM and (self.out.dtype if self.gate is not None else ctx.dtype) == torch.bfloat16
-                and L.prism_decay_chunks_supported(self.dk, self.dv, self.rd, 1 if self.il else 0) and not (self.rd and self.silu)
+                and L.prism_decay_chunks_supported(self.dk, self.dv, self.rd, 1 if self.il else 0) and not (self.rd and (self.silu or self.gate is None or self.weight is not None))
                 and all(t.data_ptr() % 16 == 0 for t in ptrs) and (self.T == 1 or self.q.stride(0) % 4 == 0)
                 and self.out.stride(0) % 2 == 0 and (self.gate is None or self.gate.stride(0) % 2 == 0)):
             return "chunks"
@@ -2042,13 +2042,13 @@ class DecayedSum:
             fac = ctx.alloc((n * H,), torch.float32)
         elif self.kind == DECAY_CHANNEL:
             cum = ctx.alloc((T, H * self.dk), torch.float32)
-            lowrank_decay(self.low, self.a2t, self.a2_bias, cum, inner_tanh=False, epilogue=LR_LOGSIGPOW, rate=self.rate)
         st = lambda t: 0 if t is None else t.stride(0)
         _check(lib().prism_decay_chunks(
             self.kind, _ptr(self.q), _ptr(self.k), _ptr(self.v), self.q.stride(0), T, ctx.S, H, self.rep, self.dk, self.dv,
             1 if self.silu else 0, _ptr(table), self.rd, 1 if self.il else 0, float(self.amp), self.qmul, self.kmul, _ptr(self.powers),
             _ptr(self.dt), st(self.dt), _ptr(self.dt_bias), self._dt(self.dt_bias), _ptr(self.a_log), self._dt(self.a_log),
-            _ptr(self.skip), self._dt(self.skip), _ptr(cum), _ptr(self.state), _ptr(ctx.seg_start), _ptr(ctx.state_slots),
+            _ptr(self.skip), self._dt(self.skip), _ptr(self.low), st(self.low), 0 if self.a2t is None else self.a2t.shape[0], _ptr(self.a2t),
+            _ptr(self.a2_bias), self._dt(self.a2_bias), self.rate, _ptr(cum), _ptr(self.state), _ptr(ctx.seg_start), _ptr(ctx.state_slots),
             _ptr(self.gate), st(self.gate), _ptr(self.weight), self._dt(self.weight), self.eps, _ptr(ws), _ptr(fac), _ptr(self.out),
             self.out.stride(0), _stream()), "decay_chunks")
         launch_count += 2
@@ -2165,7 +2165,7 @@ def unit_removal(k: torch.Tensor, a: torch.Tensor, a_bias: Optional[torch.Tensor
                                     float(unit_eps), T, H, dk, _ptr(ex), _stream()), "unit_removal")
 
 
-LR_EXPEXP, LR_SOFTPLUS, LR_SIGMOID, LR_EXPSIG, LR_SIGPOW, LR_LOGSIGPOW = 0, 1, 2, 3, 4, 5      # csrc/recurrent.cu: PRISM_LR_*
+LR_EXPEXP, LR_SOFTPLUS, LR_SIGMOID, LR_EXPSIG, LR_SIGPOW = 0, 1, 2, 3, 4      # csrc/recurrent.cu: PRISM_LR_*
 
 
 def lowrank_decay(low: torch.Tensor, w2t: torch.Tensor, w0: Optional[torch.Tensor], out: torch.Tensor, inner_tanh: bool = True,
@@ -2174,7 +2174,7 @@ def lowrank_decay(low: torch.Tensor, w2t: torch.Tensor, w0: Optional[torch.Tenso
     and in float32 throughout.  ``inner``: tanh or nothing.  ``epilogue``: ``LR_EXPEXP`` ``exp(-exp(z))`` (a per-channel
     decay from its double exponent), ``LR_SOFTPLUS`` ``exp(-exp(rate_log[n // per]) softplus(z))`` (a per-channel decay
     with one rate per ``per`` channels), ``LR_SIGMOID`` (a gate), ``LR_EXPSIG`` ``exp(-rate sigmoid(z))`` (a per-channel
-    decay that stays above ``exp(-rate)``), ``LR_SIGPOW`` ``sigmoid(z)^rate`` and ``LR_LOGSIGPOW`` its logarithm.  ``low [T, R]`` float32 (row stride free), ``w2t [R,
+    decay that stays above ``exp(-rate)``), ``LR_SIGPOW`` ``sigmoid(z)^rate``.  ``low [T, R]`` float32 (row stride free), ``w2t [R,
     N]`` float32 (the second matrix, transposed), ``w0 [N]`` or None, ``out [T, N]`` float32."""
     _cuda(low, w2t, w0, out, rate_log)
     T, R = low.shape
