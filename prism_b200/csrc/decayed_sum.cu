@@ -44,6 +44,15 @@ __device__ __forceinline__ float ds_exp2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+// log2 of sigmoid(z), with e = 2^-|z|/ln 2: where e is small log2(1 + e) comes from the series of ln(1 + e), which keeps its
+// leading digits
+__device__ __forceinline__ float ds_log2_sigmoid(float z) {
+    const float y = -fabsf(z) * 1.44269504f, e = ds_exp2(y);
+    float l;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(l) : "f"(1.f + e));
+    const float series = e * (1.f - e * (0.5f - e * (0.33333333f - e * (0.25f - e * 0.2f)))) * 1.44269504f;
+    return (z < 0.f ? y : 0.f) - (e < 0.05f ? series : l);
+}
 __device__ __forceinline__ float ds_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // ---------------------------------------------------------------------------------------------------------
@@ -422,19 +431,24 @@ __global__ void __launch_bounds__(DS_STATE_THREADS) decay_chunk_state_kernel(con
             __syncthreads();
             const float* w2 = a.a2t + (size_t)h * dk + d;
             const float bias = on && a.a2_bias != nullptr ? load_param(a.a2_bias, a.a2_bias_bf16, (size_t)h * dk + d) : 0.f;
-            const float scale = -a.rate * 1.44269504f;
+            float wr[DS_STEP_RANK];
+#pragma unroll
+            for (int c = 0; c < DS_STEP_RANK; ++c) wr[c] = on && c < RT ? w2[(size_t)c * cs] : 0.f;
             if (on)
                 for (int r = r0; r < r1; r += U) {
                     float z[U];
 #pragma unroll
                     for (int u = 0; u < U; ++u) z[u] = bias;
-                    for (int c = 0; c < RT; ++c) {
-                        const float w = w2[(size_t)c * cs];
+                    auto add = [&](int c, float w) {
                         const float4 x0 = *reinterpret_cast<const float4*>(s_low + c * DS_CHUNK + r);
                         const float4 x1 = *reinterpret_cast<const float4*>(s_low + c * DS_CHUNK + r + 4);
                         z[0] += w * x0.x; z[1] += w * x0.y; z[2] += w * x0.z; z[3] += w * x0.w;
                         z[4] += w * x1.x; z[5] += w * x1.y; z[6] += w * x1.z; z[7] += w * x1.w;
-                    }
+                    };
+#pragma unroll
+                    for (int c = 0; c < DS_STEP_RANK; ++c)
+                        if (c < RT) add(c, wr[c]);
+                    for (int c = DS_STEP_RANK; c < RT; ++c) add(c, w2[(size_t)c * cs]);
                     for (int c = RT; c < a.R; ++c) {
                         const float w = w2[(size_t)c * cs];
 #pragma unroll
@@ -444,7 +458,7 @@ __global__ void __launch_bounds__(DS_STATE_THREADS) decay_chunk_state_kernel(con
 #pragma unroll
                     for (int u = 0; u < U; ++u)
                         if (r + u < r1) {
-                            sum += scale * ds_softplus(-z[u]);
+                            sum += a.rate * ds_log2_sigmoid(z[u]);
                             cum[(size_t)(r + u) * cs] = sum;                 // so far: from the run's first row on
                         }
                 }
