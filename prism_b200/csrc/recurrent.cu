@@ -244,7 +244,7 @@ __global__ void unit_removal_kernel(const float* __restrict__ k_in, const float*
 
 // out[t][h dv + c] = o[t][h][c] / sqrt(mean_c(o[t][h]^2) + eps) * weight[widx] * act(gate[t][h dv + c]) * scale,
 // act silu, or sigmoid (gate_sigmoid; the gate may then hold the sigmoid already: gate_sigmoid 2),
-// widx = c (one weight for all heads) or h dv + c (per_head_weight).  One warp per (token, head).
+// widx = c (one weight for all heads) or h dv + c (per_head_weight); weight null: ones.  One warp per (token, head).
 template <typename T>
 __global__ void headnorm_gate_kernel(const float* __restrict__ o_in, const float* __restrict__ gate_in, long long gs,
                                      const void* __restrict__ weight, int weight_bf16, int per_head_weight, float eps,
@@ -263,7 +263,7 @@ __global__ void headnorm_gate_kernel(const float* __restrict__ o_in, const float
     ss = warp_sum(ss);
     const float inv = 1.f / sqrtf(ss / (float)dv + eps);
     for (int c = lane; c < dv; c += 32) {
-        const float wv = load_param(weight, weight_bf16, per_head_weight ? (size_t)h * dv + c : (size_t)c);
+        const float wv = weight != nullptr ? load_param(weight, weight_bf16, per_head_weight ? (size_t)h * dv + c : (size_t)c) : 1.f;
         const float gz = gate[(size_t)t * gs + (size_t)h * dv + c];
         const float g = gate_sigmoid == 2 ? gz : (gate_sigmoid ? sigmoid_f(gz) : silu_f(gz));
         out[(size_t)t * os + (size_t)h * dv + c] = from_float<T>(row[c] * inv * wv * g * scale);

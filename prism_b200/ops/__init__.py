@@ -1845,19 +1845,19 @@ def shift_mix(x: torch.Tensor, prev: torch.Tensor, mu: torch.Tensor, ctx, out: t
            "shift_mix")
 
 
-def headnorm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, scale: float, out: torch.Tensor,
+def headnorm_gate(o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], eps: float, scale: float, out: torch.Tensor,
                   gate_act: str = "silu"):
     """``out[t, h] = o[t, h] / rms(o[t, h]) * weight * act(gate[t, h]) * scale``, ``gate_act``: ``silu``, ``sigmoid`` or
     ``none`` (the gate holds the factor itself); ``o [T, H, dv]`` float32, ``gate
     [T, H * dv]`` float32 and ``out [T, H * dv]`` (compute dtype) with row strides of their own; ``weight [dv]`` (one
-    for all heads) or ``[H * dv]``."""
+    for all heads), ``[H * dv]`` or None (ones)."""
     _cuda(o, gate, weight, out)
     T, H, dv = o.shape
     assert o.dtype == torch.float32 and o.is_contiguous() and gate.dtype == torch.float32 and gate.stride(1) == 1
-    assert gate.shape == (T, H * dv) and out.shape == (T, H * dv) and out.stride(1) == 1 and weight.is_contiguous()
-    assert weight.shape in ((dv,), (H * dv,))
-    per_head = 1 if (weight.shape[0] == H * dv and H > 1) else 0
-    _check(lib().prism_headnorm_gate(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _dt(weight), per_head, float(eps),
+    assert gate.shape == (T, H * dv) and out.shape == (T, H * dv) and out.stride(1) == 1
+    assert weight is None or (weight.shape in ((dv,), (H * dv,)) and weight.is_contiguous())
+    per_head = 1 if (weight is not None and weight.shape[0] == H * dv and H > 1) else 0
+    _check(lib().prism_headnorm_gate(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), F32 if weight is None else _dt(weight), per_head, float(eps),
                                      float(scale), T, H, dv, _ptr(out), _dt(out), out.stride(0),
                                      {"silu": 0, "sigmoid": 1, "none": 2}[gate_act], _stream()), "headnorm_gate")
 
@@ -2076,7 +2076,7 @@ class DecayedSum:
             lowrank_decay(self.low, self.a2t, self.a2_bias, ww, inner_tanh=False, epilogue=LR_SIGPOW, rate=self.rate)
             recurrent_scan(SCAN_GATED, q, k, v, self.state, ctx, H, 1, dk, dv, o, ww=ww)
         if self.gate is not None:
-            headnorm_gate(o, self.gate, self.weight if self.weight is not None else _ones(dv, q.device), self.eps, 1.0, self.out)
+            headnorm_gate(o, self.gate, self.weight, self.eps, 1.0, self.out)
         elif o.data_ptr() != self.out.data_ptr():
             self.out.copy_(o.view(T, H * dv))
 
@@ -2084,17 +2084,6 @@ class DecayedSum:
         """``path``: one of the three (tests and timing); None: chosen here."""
         path = path or self.path(ctx)
         {"step": self.step, "chunks": self.chunks, "scan": self.scan}[path](ctx)
-
-
-_ones_of = {}
-
-
-def _ones(n: int, device) -> torch.Tensor:
-    """A float32 vector of ones, made once per size and device."""
-    key = (n, str(device))
-    if key not in _ones_of:
-        _ones_of[key] = torch.ones(n, dtype=torch.float32, device=device)
-    return _ones_of[key]
 
 
 def retention(ctx, proj: torch.Tensor, H: int, dk: int, dv: int, rot, decay: torch.Tensor, powers: torch.Tensor,
