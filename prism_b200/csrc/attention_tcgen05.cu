@@ -17,7 +17,8 @@
 // S of tile j+1 is computed while the softmax of tile j runs; two CTAs share an SM (256 of the
 // 512 tensor-memory columns and 97 KB of shared memory each), so one CTA's prologue and
 // epilogue hide behind the other's loop.  Softmax, the running maximum and sum, and the
-// accumulators are float32; the scores never leave the SM.
+// accumulators are float32; the scores never leave the SM.  TWO: the probabilities enter P V as two bf16 terms (16
+// mantissa bits, for models whose attention weights are float32); the two take exactly the place of the 64 scores.
 //
 // Rows of V beyond the last visible key (or before the window) are zeroed in shared memory
 // before they are multiplied, so nothing unwritten in a page can reach the result.
@@ -44,7 +45,7 @@ template <int HD> struct ACfg {
     static constexpr size_t SMEM = (size_t)Q_BYTES + 2 * STAGES * KV_BYTES + 1024 /*alignment*/ + 256 /*barriers*/;
 };
 
-template <int HD>
+template <int HD, bool TWO>
 __global__ void __launch_bounds__(THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out, int out_stride,
@@ -205,6 +206,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                         const uint64_t db = umma_desc_mn(v_addr + s * C::KV_BYTES + k * (UMMA_K * 128), BK * 128);
                         umma_bf16_ts(tmem_base + C::O_COL, tmem_base + s * BK + k * (UMMA_K / 2), db, idesc_pv,
                                      (jj > 0 || k > 0) ? 1u : 0u);
+                        if (TWO) umma_bf16_ts(tmem_base + C::O_COL, tmem_base + s * BK + BK / 2 + k * (UMMA_K / 2), db, idesc_pv, 1u);
                     }
                     umma_commit(&v_empty[s]);
                     umma_commit(&pv_done[jj & 1]);
@@ -253,7 +255,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             const float m_new = move ? m_tile : m_run;
             const float mu = m_new == -INFINITY ? 0.f : m_new;
             const float corr = move ? ex2(m_run - mu) : 1.f;           // 0 for a row that saw nothing yet
-            uint32_t pr[32];
+            uint32_t pr[32], lw[TWO ? 32 : 1];
             const uint64_t scale2 = f2_pack(scale_log2, scale_log2), neg_mu2 = f2_pack(-mu, -mu);
             uint64_t sum_a = f2_pack(0.f, 0.f), sum_b = sum_a;
 #pragma unroll
@@ -266,6 +268,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 sum_b = f2_add(sum_b, f2_pack(p2, p3));
                 pr[i] = pack2(p0, p1);
                 pr[16 + i] = pack2(p2, p3);
+                if constexpr (TWO) {
+                    lw[i] = pack2(p0 - __uint_as_float(pr[i] << 16), p1 - __uint_as_float(pr[i] & 0xffff0000u));
+                    lw[16 + i] = pack2(p2 - __uint_as_float(pr[16 + i] << 16), p3 - __uint_as_float(pr[16 + i] & 0xffff0000u));
+                }
             }
             float l0, l1;
             f2_unpack(f2_add(sum_a, sum_b), l0, l1);
@@ -304,6 +310,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
             }
             tmem_st32(lane_base + s * BK, pr);                         // P over the first half of S
+            if constexpr (TWO) tmem_st32(lane_base + s * BK + BK / 2, lw);   // what rounding took from it over the second
             tmem_wait_st();
             tc_fence_before();
             mbar_arrive(&p_full[s]);
@@ -366,7 +373,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     }
 }
 
-template <int HD>
+template <int HD, bool TWO>
 int launch(const void* q, int q_stride, int T, void* out, int out_stride, const void* kc, const void* vc, int cache_pages,
            const int* bt, int bt_width, const int* seg_start, const int* cached_len, int S, int max_q_len, int nh, int nkv,
            int page_size, int num_pages, int window, float scale, int* err, int nsplit, float* part_o, float* part_ml,
@@ -379,7 +386,7 @@ int launch(const void* q, int q_stride, int T, void* out, int out_stride, const 
     if (rc) return rc;
     rc = make_map(&mv, vc, (long long)cache_pages * page_size, (long long)nkv * HD, (long long)nkv * HD, BK);
     if (rc) return rc;
-    auto kern = attn_prefill_tc_kernel<HD>;
+    auto kern = attn_prefill_tc_kernel<HD, TWO>;
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM);
     dim3 grid(nh, (max_q_len + BQ - 1) / BQ * nsplit, S);
     return (int)launch_kernel(kern, grid, dim3(THREADS), C::SMEM, stream, mq, mk, mv, (__nv_bfloat16*)out, out_stride, bt,
@@ -397,14 +404,14 @@ PRISM_EXPORT int prism_attention_prefill_tc_supported(int hd, int nh, int nkv, i
 
 // nsplit > 1: the key tiles of every query tile are shared among nsplit CTAs, which leave partial results in
 // part_o (float [T, nh, nsplit, hd]) and part_ml (float [T, nh, nsplit, 2]) for prism_attention_merge_bf16; `out`
-// is then not written here.
+// is then not written here.  two_terms 1: the softmax's weights keep 16 mantissa bits into the second product.
 // Prefill / portions: S segments; segment s has tokens seg_start[s] .. seg_start[s+1]-1 of q [T, nh, hd] at positions
 // cached_len[s] + i.  kc / vc: bf16 [cache_pages, page_size, nkv, hd]; block-table entries are < num_pages <= cache_pages.
 PRISM_EXPORT int prism_attention_prefill_tc(const void* q, int q_stride, int T, void* out, int out_stride, const void* kc,
                                             const void* vc, int cache_pages, const int* block_table, int bt_width,
                                             const int* seg_start, const int* cached_len, int S, int max_q_len, int nh,
                                             int nkv, int hd, int page_size, int num_pages, int window, float scale,
-                                            int* err, int nsplit, float* part_o, float* part_ml, cudaStream_t stream) {
+                                            int* err, int nsplit, float* part_o, float* part_ml, int two_terms, cudaStream_t stream) {
     if (S <= 0 || max_q_len <= 0 || T <= 0) return 0;
     if (nsplit < 1 || (nsplit > 1 && (part_o == nullptr || part_ml == nullptr || ((uintptr_t)part_o & 15))))
         return (int)cudaErrorInvalidValue;
@@ -415,6 +422,7 @@ PRISM_EXPORT int prism_attention_prefill_tc(const void* q, int q_stride, int T, 
         return (int)cudaErrorInvalidValue;
 #define ARGS q, q_stride, T, out, out_stride, kc, vc, cache_pages, block_table, bt_width, seg_start, cached_len, S, \
              max_q_len, nh, nkv, page_size, num_pages, window, scale, err, nsplit, part_o, part_ml, stream
-    return hd == 64 ? prism::tca::launch<64>(ARGS) : prism::tca::launch<128>(ARGS);
+    if (two_terms) return hd == 64 ? prism::tca::launch<64, true>(ARGS) : prism::tca::launch<128, true>(ARGS);
+    return hd == 64 ? prism::tca::launch<64, false>(ARGS) : prism::tca::launch<128, false>(ARGS);
 #undef ARGS
 }

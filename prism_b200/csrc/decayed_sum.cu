@@ -34,6 +34,8 @@ namespace prism {
 
 constexpr int DS_CHUNK = 64;
 constexpr int DS_SUB = 16;                 // a sub-chunk: the rows a pair of warps of the output kernel owns
+constexpr float DS_LEAST_LOG2 = -160.f;    // a decay below 2^-160 is zero in float32 (as is one below e^-160): its logarithm need not go lower,
+                                           // which keeps the sums, and so the digits of their differences, small
 constexpr float DS_MAX_SPAN = 80.f;        // the most a sub-chunk's log decays (in units of ln 2) may sum to before its scores are formed
                                            // term by term
 
@@ -345,7 +347,7 @@ __device__ __forceinline__ void ds_token_sums(const DecayChunks& a, int h, int t
         const int r = lane + 32 * i;
         const float s = r < n ? ds_softplus(dt[(size_t)(t0 + r) * a.dts + h] + bias) : 0.f;
         d[r] = s;
-        x[i] = -rate * s;
+        x[i] = fmaxf(-rate * s, DS_LEAST_LOG2);
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float y = __shfl_up_sync(0xffffffffu, x[i], o);
@@ -458,7 +460,7 @@ __global__ void __launch_bounds__(DS_STATE_THREADS) decay_chunk_state_kernel(con
 #pragma unroll
                     for (int u = 0; u < U; ++u)
                         if (r + u < r1) {
-                            sum += a.rate * ds_log2_sigmoid(z[u]);
+                            sum += fmaxf(a.rate * ds_log2_sigmoid(z[u]), DS_LEAST_LOG2);
                             cum[(size_t)(r + u) * cs] = sum;                 // so far: from the run's first row on
                         }
                 }
@@ -1010,7 +1012,7 @@ PRISM_EXPORT int prism_decay_step(int kind, const float* q, const float* k, cons
     if (!prism_decay_step_supported(dk, dv) || H < 1 || rep < 1 || H % rep || T > 65535 || rot < 0 || rot > dk || rot % 2 ||
         (rot && (freq == nullptr || kind != PRISM_DS_HEAD)) || (uintptr_t)state % 16 || (gate == nullptr && out_dtype == PRISM_DTYPE_BF16))
         return (int)cudaErrorInvalidValue;
-    if ((kind == PRISM_DS_HEAD && decay == nullptr) || (kind == PRISM_DS_TOKEN && (dt == nullptr || dt_bias == nullptr || a_log == nullptr)) ||
+    if ((kind == PRISM_DS_HEAD && decay == nullptr) || (kind == PRISM_DS_TOKEN && (dt == nullptr || dt_bias == nullptr || a_log == nullptr || gate)) ||
         (kind == PRISM_DS_CHANNEL && (low == nullptr || a2t == nullptr || R < 1)) || kind < 0 || kind > PRISM_DS_CHANNEL)
         return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)(3 * dk + 3 * dv) * sizeof(float);

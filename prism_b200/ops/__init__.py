@@ -154,7 +154,7 @@ class _Sig:
                                     _f, _p, _p]
     prism_attention_prefill_tc_supported = [_i, _i, _i, _i]
     prism_attention_prefill_tc = [_p, _i, _i, _p, _i, _p, _p, _i, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i,
-                                  _f, _p, _i, _p, _p, _p]
+                                  _f, _p, _i, _p, _p, _i, _p]
     prism_attention_merge_bf16 = [_p, _p, _i, _p, _i, _i, _i, _i, _p]
     prism_swiglu = [_p, _p, _i, _i, _i, _p]
     prism_sgemm_nt = [_p, _i, _p, _i, _p, _i, _p, _i, _i, _i, _i, _p]
@@ -829,11 +829,12 @@ def attention_merge(part_o: torch.Tensor, part_ml: torch.Tensor, out: torch.Tens
 
 
 def attention_prefill_tc(q, out, k_cache, v_cache, block_table, seg_start, cached_len, max_q_len,
-                         num_pages, window, scale, err, nsplit: int = 1, first_token: int = 0):
+                         num_pages, window, scale, err, nsplit: int = 1, first_token: int = 0, two_terms: bool = False):
     """The same on the 5th-generation tensor cores (tcgen05, TMA, tensor memory): 128 query
     rows per CTA.  Head size 64 or 128, pages of a multiple of 64 tokens.  ``nsplit`` > 1: that many
     CTAs share a query tile's keys and a second kernel merges their partial results (of the tokens
-    from ``first_token`` on: the segments given must cover exactly those)."""
+    from ``first_token`` on: the segments given must cover exactly those).  ``two_terms``: the softmax's weights enter
+    the second product as two bf16 terms instead of one."""
     _cuda(q, out, k_cache, v_cache, block_table, seg_start, cached_len)
     T, nh, hd = q.shape
     nkv, P = k_cache.shape[2], k_cache.shape[1]
@@ -849,7 +850,7 @@ def attention_prefill_tc(q, out, k_cache, v_cache, block_table, seg_start, cache
                                             _ptr(v_cache), k_cache.shape[0], _ptr(block_table), block_table.shape[1],
                                             _ptr(seg_start), _ptr(cached_len), S, int(max_q_len), nh, nkv, hd,
                                             P, num_pages, int(window or 0), float(scale), _ptr(err), int(nsplit),
-                                            _ptr(po), _ptr(pml), _stream()), "attention_prefill_tc")
+                                            _ptr(po), _ptr(pml), 1 if two_terms else 0, _stream()), "attention_prefill_tc")
     if nsplit > 1:
         attention_merge(po[first_token:], pml[first_token:], out[first_token:])
 
@@ -1501,6 +1502,10 @@ def masked_attention(ctx, q: torch.Tensor, out: torch.Tensor, k_plane: torch.Ten
     if (q.dtype == torch.bfloat16 and MASKED_TC and not FORCE_GENERIC_ATTENTION
             and attention_masked_tc_ok(q, k_plane, v_plane, nh, nkv, dk, dv)):
         few = ctx.decode_only
+        if sink is None and dist_bias is None and masked_prefill_tc_ok(ctx, q, out, k_plane, v_plane, mask, scale):
+            attention_prefill_tc(q, out, k_plane, v_plane, block_table, ctx.seg_start, ctx.cached_len, ctx.max_q_len, num_pages, mask.size,
+                                 scale, ctx.err, two_terms=True)
+            return
         if dist_bias is None and scale > 0 and attention_latent_tc_ok(q, out, k_plane, v_plane, mask):
             attention_latent_tc(q, out, k_plane, dv, block_table, ctx.seg_start, ctx.cached_len, ctx.S, ctx.max_q_len, num_pages, mask,
                                 scale, sink, ctx.err,
@@ -1512,6 +1517,16 @@ def masked_attention(ctx, q: torch.Tensor, out: torch.Tensor, k_plane: torch.Ten
         return
     attention_masked_generic(q, out, k_plane, v_plane, block_table, ctx.positions, ctx.tok_seg, num_pages, mask,
                              scale, sink, ctx.err, dist_bias)
+
+
+def masked_prefill_tc_ok(ctx, q, out, k_plane, v_plane, mask: KeyMask, scale: float) -> bool:
+    """Whether portions under this mask (no sink, no bias by distance) run on the tcgen05 kernel of equal key and value sizes,
+    with the softmax's weights as two terms."""
+    T, nh, hd = q.shape
+    return (ATTENTION_TC and ctx.max_q_len >= ATTENTION_TC_MIN_Q and mask.kind != MASK_CHUNK and mask.keep == 0 and scale > 0
+            and k_plane.shape == v_plane.shape and k_plane.is_contiguous() and v_plane.is_contiguous() and q.is_contiguous()
+            and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and not _values_in_keys(k_plane, v_plane)
+            and attention_prefill_tc_supported(hd, nh, k_plane.shape[2], k_plane.shape[1]))
 
 
 LATENT_MIN_TILES = 8            # 64-key tiles a CTA keeps at least when a row tile's keys are shared among CTAs ...

@@ -95,14 +95,15 @@ CONFIG_D = model(90, 48, [
     layer("gla", gla(1, 40, 16, 30.0, 8), dense(24)),
     layer("lightning", lightning(3, 16, 24, (0.7, 0.96, 0.9961)), moe(24, 2, 2, 1, limit=0.5)),
 ])
-# E: a few hundred wide; sixteen query heads on two key heads, values wider than keys, attention without a window; states of
+# E: a few hundred wide; sixteen query heads on two key heads, values wider than keys, attention without a window, and keys and
+# values of 64 (portions of prompts on tcgen05); states of
 # 128 x 64 and 96 x 128; more groups than one on the right; inner widths that are no multiple of a k-block
 CONFIG_E = model(500, 384, [
     layer("parallel", parallel(left(16, 2, 64, 96, None, scale=0.12, rot_dims=32, base=10000.0), right(6, 64, 128, 3, 4, 2), 0.9, 0.3),
           moe(72, 12, 4, 4, limit=1.5)),
     layer("gla", gla(4, 96, 128, 16.0, 24), dense(200)),
     layer("lightning", lightning(3, 128, 64, (0.97, 0.99, 0.998)), moe(40, 6, 3, 2)),
-    layer("parallel", parallel(left(6, 3, 48, 32, 100, scale=0.2), right(4, 48, 32, 4, 2, 1), 0.5, 0.8), dense(136)),
+    layer("parallel", parallel(left(6, 3, 64, 64, 100, scale=0.15), right(4, 48, 32, 4, 2, 1), 0.5, 0.8), dense(136)),
 ])
 CONFIGS = {"A": (CONFIG_A, 11, 8), "B": (CONFIG_B, 12, 64), "C": (CONFIG_C, 23, 16), "D": (CONFIG_D, 14, 16), "E": (CONFIG_E, 15, 64)}
 LENGTHS = {"A": (61, 9, 2, 34, 1, 27), "B": (150, 31, 77, 64, 3), "C": (40, 1, 17, 5), "D": (75, 3, 22, 1, 30), "E": (130, 40, 66, 7)}

@@ -155,9 +155,9 @@ def test_step_sizes_and_decays():
     assert torch.allclose(out.cpu().double(), torch.exp(-NP.softplus(-zz) / 16.0), rtol=1e-5, atol=1e-6)
 
 
-def decayed_case(kind, H, rep, dk, dv, lens, g, strength=1.0):
+def decayed_case(kind, H, rep, dk, dv, lens, g, strength=1.0, R=5):
     """Float32 rows of a product and the plain result per request: a dict of what the op gets beside them."""
-    A, B, R = (H // rep) * dk, H * dv, 5
+    A, B = (H // rep) * dk, H * dv
     xs = [torch.randn(n, 2 * A + B, generator=g) for n in lens]
     args, decays = {}, []
     if kind == "head":
@@ -169,7 +169,7 @@ def decayed_case(kind, H, rep, dk, dv, lens, g, strength=1.0):
         steps = [NP.softplus((d + args["dt_bias"]).double()) for d in args["dt"]]
         decays = [[torch.exp(-torch.exp(args["a_log"][i].double()) * s[:, i:i + 1]) for i in range(H)] for s in steps]
     else:
-        args.update(a2t=torch.randn(R, H * dk, generator=g), a2_bias=torch.randn(H * dk, generator=g) * 2, rate=strength / 8.0)
+        args.update(a2t=torch.randn(R, H * dk, generator=g) * (5.0 / R) ** 0.5, a2_bias=torch.randn(H * dk, generator=g) * 2, rate=strength / 8.0)
         args["low"] = [torch.randn(n, R, generator=g) * 1.5 for n in lens]
         w = [torch.exp(-NP.softplus(-(l.double() @ args["a2t"].double() + args["a2_bias"].double())) * args["rate"]) for l in args["low"]]
         decays = [[x[:, i * dk:(i + 1) * dk] for i in range(H)] for x in w]
@@ -274,6 +274,24 @@ def test_weak_and_strong_decays_in_chunks(kind, strength):
                 o += n
 
 
+@pytest.mark.parametrize("R", [1, 15, 16, 17, 40, 41, 130])
+def test_ranks_of_the_decays_low_rank_product(R):
+    """Below, at and above what the kernels keep in registers, and above what their tile of shared memory holds."""
+    g = torch.Generator().manual_seed(R)
+    H, dk, dv, lens = 2, 40, 8, (90, 1)
+    xs, args, refs = decayed_case("channel", H, 1, dk, dv, lens, g, R=R)
+    for path, sizes in (("chunks", (70, 20)), ("scan", (70, 20)), (None, (89, 1))):
+        state = torch.zeros(2, H, dv, dk, device=DEV)
+        for live in pieces(lens, sizes):
+            ctx = step_ctx([n for _, _, n in live], [s for s, _, _ in live], torch.bfloat16)
+            out = torch.empty(sum(n for _, _, n in live), H * dv, device=DEV)
+            decayed_sum("channel", ctx, torch.cat([xs[s][a:a + n] for s, a, n in live]).to(DEV), args, live, H, 1, dk, dv, state, out, path)
+            o = 0
+            for s, a, n in live:
+                assert float((out[o:o + n].cpu().double() - refs[s][a:a + n]).abs().max()) <= 1e-3 * float(refs[s].abs().max()), (path, s, a)
+                o += n
+
+
 @pytest.mark.parametrize("kind", ["head", "token", "channel"])
 def test_an_old_token_comes_back_through_the_state_of_many_chunks(kind):
     """Keys and queries are orthogonal but for token 3: with decays close to one, what the last tokens read is token 3's
@@ -340,6 +358,70 @@ def test_limited_experts_with_identity_experts(T, W, F, E, idle, top, dtype):
             ops.moe_tensor_cores = keep
         assert y.shape == (top, T, W)
         assert float((y.sum(0).cpu().double() - ref).abs().max()) <= tol * max(1.0, float(ref.abs().max())), tc
+    ops.check_tc_errors()
+
+
+@pytest.mark.parametrize("hd, nh, nkv", [(64, 4, 2), (128, 6, 1), (64, 3, 3)])
+@pytest.mark.parametrize("window", [None, 1, 30, 64, 65, 100, 500])
+def test_windowed_attention_of_portions_with_weights_as_two_terms(hd, nh, nkv, window):
+    """Portions that start and end around pages, tiles and windows, single tokens among them, NaN in the slots nothing was
+    stored in, and one key that stands out just inside and just outside the last query's window: on tcgen05 and on the
+    masked mma.sync kernel."""
+    from prism_b200 import ops
+    g = torch.Generator().manual_seed(hd + nh)
+    mask, P = ops.KeyMask.window(window), 64
+    segs = [(0, 3), (200, 70), (63, 2), (0, 130), (330, 128), (447, 1)]
+    per = [-(-(c + n) // P) for c, n in segs]
+    order = torch.randperm(sum(per), generator=g).tolist()
+    bt = torch.full((len(segs), max(per)), sum(per), dtype=torch.int32)
+    k, v = torch.randn(sum(per) + 1, P, nkv, hd, generator=g), torch.randn(sum(per) + 1, P, nkv, hd, generator=g)
+    T = sum(n for _, n in segs)
+    q, ids, o = torch.randn(T, nh, hd, generator=g), [], 0
+    for s, (c, n) in enumerate(segs):
+        ids.append(order[o:o + per[s]])
+        bt[s, :per[s]] = torch.tensor(ids[s], dtype=torch.int32)
+        o += per[s]
+        if (c + n) % P:
+            k[ids[s][-1], (c + n) % P:] = math.nan
+            v[ids[s][-1], (c + n) % P:] = math.nan
+    edge = 330 + 127 - (window or 10 ** 6) + 1                # the first key the fifth request's last query sees
+    for key in (edge - 1, edge):
+        if 0 <= key <= 457:
+            k[ids[4][key // P], key % P] = 0.0
+            k[ids[4][key // P], key % P, :, :8] = 8.0
+            v[ids[4][key // P], key % P] = 50.0 if key == edge else -300.0
+    last = sum(n for _, n in segs[:5]) - 1
+    q[last] = 0.0
+    q[last, :, :8] = 8.0
+    q, k, v = q.to(torch.bfloat16), k.to(torch.bfloat16), v.to(torch.bfloat16)
+    refs, t = [], 0
+    for s, (c, n) in enumerate(segs):
+        kk, vv = (x[ids[s]].reshape(-1, nkv, hd)[:c + n].double() for x in (k, v))
+        see = NP.visible(c + n, window)[c:]
+        row = torch.zeros(n, nh, hd, dtype=torch.float64)
+        for h in range(nh):
+            sc = (q[t:t + n, h].double() @ kk[:, h // (nh // nkv)].T * 0.1).masked_fill(~see, -math.inf)
+            row[:, h] = torch.softmax(sc, -1) @ vv[:, h // (nh // nkv)]
+        refs.append(row.reshape(n, nh * hd))
+        t += n
+    ref = torch.cat(refs)
+    i32 = lambda x: torch.as_tensor(x, dtype=torch.int32).to(DEV)
+    ctx = types.SimpleNamespace(S=len(segs), max_q_len=130, max_kv_len=458, decode_only=False, err=torch.zeros(1, dtype=torch.int32, device=DEV),
+                                seg_start=i32([0] + torch.tensor([n for _, n in segs]).cumsum(0).tolist()), cached_len=i32([c for c, _ in segs]))
+    qd, kd, vd, btd = q.to(DEV), k.to(DEV), v.to(DEV), bt.to(DEV)
+    keep = ops.ATTENTION_TC
+    for tc in (True, False):
+        ops.ATTENTION_TC = tc
+        try:
+            out = torch.zeros(T, nh * hd + 8, dtype=torch.bfloat16, device=DEV)[:, :nh * hd]
+            assert ops.masked_prefill_tc_ok(ctx, qd, out, kd, vd, mask, 0.1) == tc
+            ops.masked_attention(ctx, qd, out, kd, vd, btd, sum(per), mask, 0.1)
+        finally:
+            ops.ATTENTION_TC = keep
+        assert int(ctx.err.item()) == 0
+        err = (out.float().cpu().double() - ref).abs()
+        # the result is rounded to bfloat16 once; the weights are not
+        assert bool((err <= 2.0 ** -8 * ref.abs() + 2e-3).all()), (tc, float(err.max()))
     ops.check_tc_errors()
 
 
